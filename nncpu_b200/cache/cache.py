@@ -46,13 +46,15 @@ class KVRequest:
     they differ from a key head's (0: the same).  ``chunk`` n: queries see the keys of their own block of n positions
     only (blocks counted from position 0), so the blocks before the one that is being filled need not be kept.
     ``keys_only``: the mixer keeps one vector per position and head and reads it as key and as value; no value
-    pages are made, and the group's value pages are its key pages."""
+    pages are made, and the group's value pages are its key pages.  ``keep_first`` n (with a window): the first n
+    positions stay visible to every query, so their pages are kept."""
     n_kv_heads: int
     head_dim: int
     window: int = 0
     v_head_dim: int = 0
     chunk: int = 0
     keys_only: bool = False
+    keep_first: int = 0
 
 
 @dataclass(frozen=True)
@@ -78,13 +80,18 @@ class KVGroup:
 
     def first_needed_page(self, length: int) -> int:
         """Pages below this index hold no key that a query at position
-        ``length`` or later can see."""
+        ``length`` or later can see (but for the first ``kept_pages`` of them)."""
         w, c = self.request.window, self.request.chunk
         if c > 0:
             return (length // c * c) // PAGE        # the block that position ``length`` belongs to starts there
         if w <= 0 or length + 1 <= w:
             return 0
         return (length + 1 - w) // PAGE
+
+    @property
+    def kept_pages(self) -> int:
+        """Pages at a sequence's start that a window never gives back."""
+        return pages_for(self.request.keep_first) if self.request.window > 0 else 0
 
     def pages_missing(self, slot: int, new_len: int) -> int:
         return max(0, pages_for(new_len) - len(self.tables.get(slot, ())))
@@ -96,7 +103,7 @@ class KVGroup:
 
     def trim(self, slot: int, length: int) -> None:
         table = self.tables.get(slot, [])
-        for i in range(min(self.first_needed_page(length), len(table))):
+        for i in range(self.kept_pages, min(self.first_needed_page(length), len(table))):
             if table[i] >= 0:
                 self.pool.give_back(table[i])
                 table[i] = -1
@@ -201,7 +208,8 @@ class Cache:
             if any(s is not None for s in self.states) and length > 0:
                 raise InvalidArgument("a sequence with per-sequence state cannot be rewound, only restarted")
             for g in self.groups:
-                if g.first_needed_page(self.lengths[slot]) > g.first_needed_page(length):
+                first = max(g.first_needed_page(length), g.kept_pages)
+                if g.first_needed_page(self.lengths[slot]) > first:
                     raise InvalidArgument(f"slot {slot}: the window has already moved past position {length}")
         self.lengths[slot] = length
 

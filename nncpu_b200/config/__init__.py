@@ -4,12 +4,14 @@ from .registry import (architectures, config_class, config_from_dict, load_confi
 from .specs import (AttentionSpec, BlockSpec, DenseMlpSpec, EmbeddingSpec, FeedForwardSpec, GatedDeltaSpec,
                     GatedLinearAttentionSpec,
                     GatedMlpSpec, LatentAttentionSpec, MixerSpec, ModelSpec, NormSpec, OutputSpec, PositionSpec,
-                    RoutedExpertsSpec, ScheduleEntry, StreamInjection, MixerPairSpec, RetentionSpec, TokenSideSpec)
+                    RoutedExpertsSpec, ScheduleEntry, StreamInjection, MixerPairSpec, RetentionSpec, StateSpaceSpec,
+                    TokenSideSpec)
 from .qwen3 import Qwen3Config
 from .romepel import RomepelConfig
 from .zevivik import ZevivikConfig
 from .pikalorn import PikalornConfig
 from .vodalorn import VodalornConfig
+from .gekilix import GekilixConfig
 
 __all__ = [
     "architectures", "config_class", "config_from_dict", "load_config", "register_architecture",
@@ -17,5 +19,5 @@ __all__ = [
     "ModelSpec", "NormSpec", "OutputSpec", "PositionSpec", "ScheduleEntry", "Qwen3Config", "RomepelConfig",
     "DenseMlpSpec", "GatedLinearAttentionSpec", "LatentAttentionSpec", "RoutedExpertsSpec", "StreamInjection",
     "ZevivikConfig", "GatedDeltaSpec", "PikalornConfig", "MixerPairSpec", "RetentionSpec", "TokenSideSpec",
-    "VodalornConfig",
+    "VodalornConfig", "GekilixConfig", "StateSpaceSpec",
 ]

@@ -48,6 +48,10 @@ class PositionSpec:
     scaling_original: float = 0.0
     scaling_fast: float = 0.0
     scaling_slow: float = 0.0
+    # ``scaling_kind`` "bands": the limits are wavelengths instead.  With l = 2 pi / f_i the wavelength of pair i, it turns
+    # at f_i where l < original / fast, at f_i / factor where l > original / slow, and between the two at
+    # (1 - s) f_i / factor + s f_i with s = (original / l - slow) / (fast - slow); cos and sin are not stretched.
+    scaling_kind: str = "ramp"
 
 
 @dataclass(frozen=True)
@@ -69,7 +73,10 @@ class AttentionSpec(MixerSpec):
     out_bias_optional: bool = False  # accept "<name>.o_proj.bias" when the file has it
     scale: float = 0.0               # multiplies q.k after the dot product
     window: int = 0                  # 0: every earlier key; n: the last n keys up to the query
+    keep_first: int = 0              # with a window: the sequence's first n keys stay visible too
     qk_norm: Optional[NormSpec] = None   # per-head norm of q and k (names end in q_norm / k_norm)
+    qk_norm_whole: bool = False      # that norm runs over all the heads' lanes at once (one weight per lane of the
+                                     # projection), before the split into heads
     position: Optional[PositionSpec] = None
     v_head_dim: int = 0              # lanes of a value head (and of a head's output); 0: head_dim
     slope_base: float = 0.0          # b != 0: head h takes 2^(-b (h + 1) / n_heads) * (i - j) off its scaled scores
@@ -183,6 +190,25 @@ class GatedLinearAttentionSpec(MixerSpec):
 
 
 @dataclass(frozen=True)
+class StateSpaceSpec(MixerSpec):
+    """A state-space mixer with one decay per head and token (Mamba-2, "Transformers are SSMs", Dao and Gu): per head a
+    state S of ``state`` x ``value_dim`` 32-bit numbers.  W_in h holds, in this order, z and x (``n_heads`` x
+    ``value_dim`` each), B and C (``n_groups`` x ``state`` each; head h uses group h // (n_heads / n_groups)) and dt
+    (``n_heads``).  x, B and C pass a causal convolution of ``conv`` taps per channel with a bias, then SiLU;
+    dt <- softplus(dt + dt_bias); S <- exp(-exp(A_log) dt) S + dt B x^T; y = S^T C + D x.  The heads' y times silu(z) are
+    RMS-normed in ``norm_groups`` equal parts (``eps``), multiplied by a weight and projected back.  The convolutions'
+    last inputs are state too."""
+    hidden_size: int = 0
+    n_heads: int = 0
+    value_dim: int = 0
+    state: int = 0
+    n_groups: int = 1
+    conv: int = 0
+    norm_groups: int = 1
+    eps: float = 1e-6
+
+
+@dataclass(frozen=True)
 class FeedForwardSpec:
     """The part of a block that works on each position alone."""
     kind: str
@@ -210,7 +236,12 @@ class RoutedExpertsSpec(FeedForwardSpec):
     are chosen, and their weights are their scores divided by the sum of the chosen scores (+ 1e-20), times
     ``weight_scale``.  With ``n_groups`` > 1 the experts form that many equal groups of neighbours, a group's score is
     its largest score, and only experts of the ``keep_groups`` best groups can be chosen.  ``router_bias`` False: the
-    router has no bias tensor.  ``out_scale`` multiplies what the part adds to the stream."""
+    router has no bias tensor.  ``out_scale`` multiplies what the part adds to the stream.
+
+    ``scores`` "sigmoid": an expert's score is the sigmoid of its logit, and the chosen experts' weights are their scores
+    as they are.  ``weight_on`` "input": a weight multiplies the expert's input, expert(w x), instead of its output.
+    ``shared_gate``: the shared feed-forward's output is multiplied by sigmoid(w x), one number per token
+    (``<shared name>.sg`` [1, hidden])."""
     hidden_size: int = 0
     intermediate_size: int = 0
     n_experts: int = 0
@@ -224,6 +255,8 @@ class RoutedExpertsSpec(FeedForwardSpec):
     weight_scale: float = 1.0
     router_bias: bool = True
     out_scale: float = 1.0
+    weight_on: str = "output"
+    shared_gate: bool = False
 
 
 @dataclass(frozen=True)

@@ -1,5 +1,7 @@
 // bfloat16 attention over the paged cache on tensor cores (mma.sync m16n8k16),
-// for head sizes 64 and 128.  Softmax runs in 32-bit with the scale applied
+// for key rows of 64 and 128 lanes and value rows of 64 lanes or the keys' size
+// (HD and VD below; a head of another size lies in such rows with zeros behind
+// it, and `vo` is the number of lanes a head has in the output).  Softmax runs in 32-bit with the scale applied
 // after the dot product (crates/nncpu/src/kernels/scalar.rs:444-548), online
 // over blocks of keys, and partial results are merged in key order like the
 // reference's block partials (crates/nncpu/src/kernels/scalar.rs:521-548,
@@ -72,11 +74,11 @@ __device__ __forceinline__ float ld_cluster_(const float* local, uint32_t rank) 
     return v;
 }
 
-// Merges the splits of every (token, head) in split order.  grid = (n_heads, n_tok), HD threads.
-template <int HD>
+// Merges the splits of every (token, head) in split order.  grid = (n_heads, n_tok), VD threads.
+template <int VD>
 __global__ void merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                              __nv_bfloat16* __restrict__ out, int n_heads, int n_kv, int n_splits,
-                             const float* __restrict__ sinks, const float* __restrict__ gate, long gate_ld) {
+                             const float* __restrict__ sinks, const float* __restrict__ gate, long gate_ld, int vo) {
     const int h = blockIdx.x, t = blockIdx.y, d = threadIdx.x;
     const int G = n_heads / n_kv, kvh = h / G, head = h % G;
     const size_t pb = ((size_t)t * n_kv + kvh) * n_splits;
@@ -86,13 +88,14 @@ __global__ void merge_kernel(const float* __restrict__ part_o, const float* __re
     for (int s = 0; s < n_splits; ++s) {
         const float ms = part_ml[((pb + s) * G + head) * 2];
         const float c = ms == -INFINITY ? 0.0f : exp2f(ms - m);
-        o = fmaf(part_o[((pb + s) * G + head) * HD + d], c, o);
+        o = fmaf(part_o[((pb + s) * G + head) * VD + d], c, o);
         l = fmaf(part_ml[((pb + s) * G + head) * 2 + 1], c, l);
     }
     if (sinks != nullptr && l > 0.0f) l += exp2f(sinks[h] * kLog2e - m);
     float res = l > 0.0f ? o / l : 0.0f;
-    if (gate != nullptr) res *= 1.0f / (1.0f + expf(-gate[(size_t)t * gate_ld + (size_t)h * HD + d]));
-    out[((size_t)t * n_heads + h) * HD + d] = __float2bfloat16_rn(res);
+    if (d >= vo) return;
+    if (gate != nullptr) res *= 1.0f / (1.0f + expf(-gate[(size_t)t * gate_ld + (size_t)h * vo + d]));
+    out[((size_t)t * n_heads + h) * vo + d] = __float2bfloat16_rn(res);
 }
 
 // ---------------------------------------------------------------------------
@@ -125,15 +128,16 @@ __device__ __forceinline__ uint32_t tile_off(int row, int chunk) {
     return (uint32_t)(row * (HD * 2) + (((chunk & ~7) | ((chunk ^ row) & 7)) << 4));
 }
 
-template <int HD>
+template <int HD, int VD>
 __global__ void __launch_bounds__(128, 3)
 prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_pages,
                const __nv_bfloat16* __restrict__ v_pages, const int* __restrict__ block_table, int bt_stride,
                const int* __restrict__ cu_seqlens, const int* __restrict__ tok_pos, __nv_bfloat16* __restrict__ out,
-               int n_seqs, int n_heads, int n_kv, float scale2, int window, float slope_base,
-               const float* __restrict__ sinks) {
-    constexpr int kTileBytes = kPage * HD * 2;           // one page of K or of V for one head
-    constexpr int kChunks = HD / 8;                      // 16-byte chunks per row
+               int n_seqs, int n_heads, int n_kv, float scale2, int window, int keep, float slope_base,
+               const float* __restrict__ sinks, int vo) {
+    constexpr int kTileBytes = kPage * HD * 2;           // one page of K for one head
+    constexpr int kStageBytes = kPage * (HD + VD) * 2;   // and of V behind it
+    constexpr int kChunks = HD / 8, kVChunks = VD / 8;   // 16-byte chunks per row
     extern __shared__ __align__(128) uint8_t fa_smem[];  // [2 stages][K tile | V tile]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int c = lane & 3, r = lane >> 2;
@@ -157,7 +161,7 @@ prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restr
     const int pos0 = tok_pos[q0];                        // positions of a sequence's new tokens are consecutive
     const int key_hi = pos0 + n_rows - 1;                // the last row's last key
     const int key_lo = first_visible_key(pos0, window);
-    const int page_lo = key_lo / kPage, page_hi = key_hi / kPage;
+    const PageWalk walk(key_lo, key_hi, keep);           // the pages that hold keys these rows see
     const int* table = block_table + (size_t)seq * bt_stride;
     const int kvh = h / (n_heads / n_kv);
     // a distance bias: this head takes slope * (query position - key position) off its scaled scores (0: none);
@@ -191,35 +195,39 @@ prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restr
     }
 
     auto issue = [&](int page_idx, int stage) {
-        const size_t base = ((size_t)table[page_idx] * n_kv + kvh) * (size_t)(kPage * HD);
-        const uint32_t dst = smem_u32_(fa_smem) + stage * 2 * kTileBytes;
+        const size_t head_row = ((size_t)table[page_idx] * n_kv + kvh) * (size_t)kPage;     // its first row in the pages
+        const uint32_t dst = smem_u32_(fa_smem) + stage * kStageBytes;
 #pragma unroll
         for (int i = threadIdx.x; i < kPage * kChunks; i += 128) {
             const int row = i / kChunks, chunk = i % kChunks;
-            cp_async16(dst + tile_off<HD>(row, chunk), k_pages + base + (size_t)row * HD + chunk * 8);
-            cp_async16(dst + kTileBytes + tile_off<HD>(row, chunk), v_pages + base + (size_t)row * HD + chunk * 8);
+            cp_async16(dst + tile_off<HD>(row, chunk), k_pages + (head_row + row) * HD + chunk * 8);
+        }
+#pragma unroll
+        for (int i = threadIdx.x; i < kPage * kVChunks; i += 128) {
+            const int row = i / kVChunks, chunk = i % kVChunks;
+            cp_async16(dst + kTileBytes + tile_off<VD>(row, chunk), v_pages + (head_row + row) * VD + chunk * 8);
         }
         cp_async_commit();
     };
 
-    float o[HD / 8][4];
+    float o[VD / 8][4];
 #pragma unroll
-    for (int t = 0; t < HD / 8; ++t) o[t][0] = o[t][1] = o[t][2] = o[t][3] = 0.0f;
+    for (int t = 0; t < VD / 8; ++t) o[t][0] = o[t][1] = o[t][2] = o[t][3] = 0.0f;
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
 
-    issue(page_lo, 0);
-    for (int pg = page_lo; pg <= page_hi; ++pg) {
-        const int stage = (pg - page_lo) & 1;
-        if (pg + 1 <= page_hi) {
-            issue(pg + 1, stage ^ 1);
+    issue(walk.page(0), 0);
+    for (int i = 0; i < walk.n; ++i) {
+        const int stage = i & 1;
+        if (i + 1 < walk.n) {
+            issue(walk.page(i + 1), stage ^ 1);
             cp_async_wait<1>();
         } else {
             cp_async_wait<0>();
         }
         __syncthreads();
-        const int k_base = pg * kPage;
-        if (k_base <= warp_key_hi && k_base + kPage - 1 >= warp_key_lo) {
-            const uint32_t ks_addr = smem_u32_(fa_smem) + stage * 2 * kTileBytes;
+        const int k_base = walk.page(i) * kPage;
+        if (k_base <= warp_key_hi && (k_base + kPage - 1 >= warp_key_lo || k_base < keep)) {
+            const uint32_t ks_addr = smem_u32_(fa_smem) + stage * kStageBytes;
             const uint32_t vs_addr = ks_addr + kTileBytes;
             // scores of 16 rows x 64 keys
             float s[8][4];
@@ -249,7 +257,7 @@ prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restr
                     if (!full || slope2 != 0.0f) {
                         const int key = k_base + t * 8 + 2 * c + (e & 1);
                         v -= slope2 * (float)(lim_hi[row] - key);
-                        if (!full && (key < lim_lo[row] || key > lim_hi[row])) v = -INFINITY;
+                        if (!full && ((key < lim_lo[row] && key >= keep) || key > lim_hi[row])) v = -INFINITY;
                     }
                     s[t][e] = v;
                     mx[row] = fmaxf(mx[row], v);
@@ -277,7 +285,7 @@ prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restr
             l[1] = l[1] * corr[1] + sum[1];
             if (__any_sync(0xffffffffu, corr[0] != 1.0f || corr[1] != 1.0f)) {
 #pragma unroll
-                for (int t = 0; t < HD / 8; ++t) {
+                for (int t = 0; t < VD / 8; ++t) {
                     o[t][0] *= corr[0]; o[t][1] *= corr[0]; o[t][2] *= corr[1]; o[t][3] *= corr[1];
                 }
             }
@@ -288,11 +296,11 @@ prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restr
                 const uint32_t a2 = pack_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1]);
                 const uint32_t a3 = pack_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3]);
 #pragma unroll
-                for (int dp = 0; dp < HD / 16; ++dp) {   // pairs of 8-lane tiles of the head
+                for (int dp = 0; dp < VD / 16; ++dp) {   // pairs of 8-lane tiles of the head
                     uint32_t b[4];
                     const int key = kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7);
                     const int chunk = dp * 2 + (lane >> 4);
-                    ldmatrix_x4_trans(b, vs_addr + tile_off<HD>(key, chunk));
+                    ldmatrix_x4_trans(b, vs_addr + tile_off<VD>(key, chunk));
                     mma_bf16(o[2 * dp], a0, a1, a2, a3, b[0], b[1]);
                     mma_bf16(o[2 * dp + 1], a0, a1, a2, a3, b[2], b[3]);
                 }
@@ -308,10 +316,18 @@ prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restr
         // a sink: one more term of the denominator, with no key and no value (the softmax works in powers of two)
         if (sinks != nullptr && l[row] > 0.0f) l[row] += exp2f(sinks[h] * kLog2e - m[row]);
         const float inv = l[row] > 0.0f ? 1.0f / l[row] : 0.0f;
-        __nv_bfloat16* dst = out + (size_t)(q0 + (row == 0 ? row_lo : row_hi)) * n_heads * HD + (size_t)h * HD;
+        __nv_bfloat16* dst = out + ((size_t)(q0 + (row == 0 ? row_lo : row_hi)) * n_heads + h) * vo;
 #pragma unroll
-        for (int t = 0; t < HD / 8; ++t)
-            *reinterpret_cast<uint32_t*>(dst + t * 8 + 2 * c) = pack_bf16(o[t][2 * row] * inv, o[t][2 * row + 1] * inv);
+        for (int t = 0; t < VD / 8; ++t) {
+            const int d = t * 8 + 2 * c;
+            const float a = o[t][2 * row] * inv, b = o[t][2 * row + 1] * inv;
+            if (vo == VD || ((vo & 1) == 0 && d < vo)) {
+                *reinterpret_cast<uint32_t*>(dst + d) = pack_bf16(a, b);
+            } else {                       // a head with an odd number of lanes: its lanes one by one
+                if (d < vo) dst[d] = __float2bfloat16_rn(a);
+                if (d + 1 < vo) dst[d + 1] = __float2bfloat16_rn(b);
+            }
+        }
     }
 }
 
@@ -335,49 +351,77 @@ constexpr int kMaxClusterSplits = 8;   // splits that merge inside a thread-bloc
 // steps to come, and puts them into its copy of the page, where nobody else looks for them in this step.  The
 // arithmetic is that of the separate kernel for norm, rotation and append, operation for operation.
 struct FusedQK {
-    const float* qkv;         // [n_tok, per_tok * HD]: the heads of q, then (if appended here) of k, then of v
-    int per_tok;              // heads a token's row holds
-    const void* q_gamma;      // per-head norm weights [HD], or null
+    const float* qkv;         // [n_tok, ld]: the heads of q, then (if appended here) of k, then of v
+    int ld;                   // floats a token's row holds
+    int hd, vd;               // lanes of a query/key head and of a value head in it (the pages' rows hold zeros beyond)
+    int k_at, v_at;           // where the heads of k and of v start in it
+    int whole;                // the norm runs over all the heads' lanes at once (weights [n_heads hd] and [n_kv hd])
+    const void* q_gamma;      // per-head norm weights [hd], or null
     const void* k_gamma;
     int g_dt;
     float eps;
-    const float2* cs;         // [n_tok, HD / 2] (cos, sin) of the tokens' positions, or null: no rotation
+    const float2* cs;         // [n_tok, half] (cos, sin) of the tokens' positions, or null: no rotation
+    int half;                 // pairs that are rotated
+    int pairs;                // 1: pair i is lanes (2 i, 2 i + 1); 0: lanes (i, i + hd / 2), and the whole head turns
     __nv_bfloat16* k_pages;   // the cache, writable; null: the keys and values are another entry's, nothing is appended
     __nv_bfloat16* v_pages;
     float slope_base;         // not of the projections: b != 0 gives head h the distance bias 2^(-b (h + 1) / n_heads) * (pos - key)
     float temp_coef;          // c != 0: the query at position p is multiplied by 1 + c ln(floor((p + 1) / temp_every) + 1)
     int temp_every;
     int values_are_keys;      // the row holds no v heads: a token's value is its key as projected (before norm and rotation)
-    int gate_at;              // >= 0: the row's heads from gate_at on are logits, one a lane of the output: the output is
+    int gate_at;              // >= 0: the row's floats from gate_at on are logits, one a lane of the output: the output is
                               // multiplied by their sigmoid; < 0: no gate
 };
 
-// One head's HD float32 values through norm (if gamma) and rotation (if cs) to bfloat16; a warp's job.  A lane holds
-// HD / 32 neighbouring lanes of the head, so a rotation pair (i, i + HD / 2) sits in the lanes l and l ^ 16.
+// One head's float32 values (n of them, zeros up to HD) through norm (if gamma) and rotation (if cs) to bfloat16; a
+// warp's job.  A lane holds HD / 32 neighbouring lanes of the head, so a rotation pair (i, i + HD / 2) sits in the lanes
+// l and l ^ 16, and a pair (2 i, 2 i + 1) in one lane.  given_scale > 0: the norm's scale is known (it runs over more
+// than this head).
 template <int HD>
-__device__ __forceinline__ void finish_head(const float* __restrict__ src, const void* __restrict__ gamma, int g_dt, float eps,
-                                            const float2* __restrict__ cs_row, __nv_bfloat16* __restrict__ dst, int lane,
+__device__ __forceinline__ void finish_head(const float* __restrict__ src, int n, const void* __restrict__ gamma, int gamma_at,
+                                            int g_dt, float eps, float given_scale, const float2* __restrict__ cs_row,
+                                            int half, int pairs, __nv_bfloat16* __restrict__ dst, int lane,
                                             float times = 1.0f) {
     constexpr int EPL = HD / 32;
     float x[EPL];
-    if (EPL == 4) {
-        const float4 v = *reinterpret_cast<const float4*>(src + lane * EPL);
-        x[0] = v.x; x[1] = v.y; x[2 % EPL] = v.z; x[3 % EPL] = v.w;
+    if (n == HD && (reinterpret_cast<uintptr_t>(src) & 15) == 0) {
+        if (EPL == 4) {
+            const float4 v = *reinterpret_cast<const float4*>(src + lane * EPL);
+            x[0] = v.x; x[1] = v.y; x[2 % EPL] = v.z; x[3 % EPL] = v.w;
+        } else {
+            const float2 v = *reinterpret_cast<const float2*>(src + lane * EPL);
+            x[0] = v.x; x[1] = v.y;
+        }
     } else {
-        const float2 v = *reinterpret_cast<const float2*>(src + lane * EPL);
-        x[0] = v.x; x[1] = v.y;
+#pragma unroll
+        for (int e = 0; e < EPL; ++e) x[e] = lane * EPL + e < n ? src[lane * EPL + e] : 0.0f;
     }
     if (gamma) {
-        float ss = 0.0f;
+        float scale = given_scale;
+        if (given_scale <= 0.0f) {
+            float ss = 0.0f;
 #pragma unroll
-        for (int e = 0; e < EPL; ++e) ss = fmaf(x[e], x[e], ss);
+            for (int e = 0; e < EPL; ++e) ss = fmaf(x[e], x[e], ss);
 #pragma unroll
-        for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-        const float scale = 1.0f / sqrtf(ss * (1.0f / (float)HD) + eps);
+            for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+            scale = 1.0f / sqrtf(ss * (1.0f / (float)n) + eps);
+        }
 #pragma unroll
-        for (int e = 0; e < EPL; ++e) x[e] = (x[e] * scale) * ld_f(gamma, lane * EPL + e, g_dt);
+        for (int e = 0; e < EPL; ++e)
+            x[e] = lane * EPL + e < n ? (x[e] * scale) * ld_f(gamma, gamma_at + lane * EPL + e, g_dt) : 0.0f;
     }
-    if (cs_row != nullptr) {
+    if (cs_row != nullptr && pairs) {
+#pragma unroll
+        for (int e = 0; e < EPL; e += 2) {
+            const int i = (lane * EPL + e) >> 1;
+            if (i < half) {
+                const float2 c = cs_row[i];
+                const float u = x[e], v = x[e + 1];
+                x[e] = c.x * u - c.y * v;
+                x[e + 1] = c.y * u + c.x * v;
+            }
+        }
+    } else if (cs_row != nullptr) {
         const int i0 = (lane & 15) * EPL;
 #pragma unroll
         for (int e = 0; e < EPL; ++e) {
@@ -398,50 +442,77 @@ __device__ __forceinline__ void finish_head(const float* __restrict__ src, const
     }
 }
 
-template <int HD, int NT, bool kCluster, bool kFused>
+// The sum of squares of n floats, by a block of 128 threads; every thread gets it.  `scratch` holds 4 floats.
+__device__ __forceinline__ float row_squares(const float* __restrict__ src, int n, float* scratch) {
+    float ss = 0.0f;
+    if ((n & 3) == 0 && (reinterpret_cast<uintptr_t>(src) & 15) == 0) {
+        for (int i = threadIdx.x; i < (n >> 2); i += 128) {
+            const float4 v = reinterpret_cast<const float4*>(src)[i];
+            ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
+        }
+    } else {
+        for (int i = threadIdx.x; i < n; i += 128) ss = fmaf(src[i], src[i], ss);
+    }
+    ss = warp_sum(ss);
+    if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    ss = (scratch[0] + scratch[1]) + (scratch[2] + scratch[3]);
+    __syncthreads();
+    return ss;
+}
+
+template <int HD, int VD, int NT, bool kCluster, bool kFused>
 __global__ void __launch_bounds__(128, 2)
 decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_pages,
                    const __nv_bfloat16* __restrict__ v_pages, const int* __restrict__ block_table, int bt_stride,
                    const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, __nv_bfloat16* __restrict__ out,
                    float* __restrict__ part_o, float* __restrict__ part_ml, int n_heads, int n_kv, float scale2,
-                   int window, const FusedQK f, const float* __restrict__ sinks, int kv_rep) {
-    constexpr int kTileBytes = kPage * HD * 2;
-    constexpr int kChunks = HD / 8;
-    constexpr int W = HD + 2;
+                   int window, int keep, const FusedQK f, const float* __restrict__ sinks, int kv_rep, int vo) {
+    constexpr int kTileBytes = kPage * HD * 2, kStageBytes = kPage * (HD + VD) * 2;
+    constexpr int kChunks = HD / 8, kVChunks = VD / 8;
+    constexpr int W = VD + 2;
     extern __shared__ __align__(128) uint8_t dsm[];  // stages of [K page | V page]; afterwards the merge buffers
     const int split = blockIdx.x, n_splits = gridDim.x, kvh = blockIdx.y, t = blockIdx.z;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int c = lane & 3, r = lane >> 2;
     const int G = n_heads / n_kv;
     const int seq = tok_seq[t];
-    const size_t out_row = (size_t)t * n_heads * HD + (size_t)kvh * G * HD;
+    const size_t out_row = ((size_t)t * n_heads + (size_t)kvh * G) * vo;
     if (seq < 0) {  // padding: zeros (every block of a cluster takes this way out together)
         if (n_splits == 1 || split == 0)
-            for (int i = threadIdx.x; i < G * HD; i += 128) out[out_row + i] = __float2bfloat16_rn(0.0f);
+            for (int i = threadIdx.x; i < G * vo; i += 128) out[out_row + i] = __float2bfloat16_rn(0.0f);
         if (n_splits > 1 && !kCluster) {
             const size_t pb = ((size_t)t * n_kv + kvh) * n_splits + split;
-            for (int i = threadIdx.x; i < G * HD; i += 128) part_o[pb * G * HD + i] = 0.0f;
+            for (int i = threadIdx.x; i < G * VD; i += 128) part_o[pb * G * VD + i] = 0.0f;
             for (int i = threadIdx.x; i < G * 2; i += 128) part_ml[pb * G * 2 + i] = (i & 1) ? 0.0f : -INFINITY;
         }
         return;
     }
     const int pos = tok_pos[t];
     const int first = first_visible_key(pos, window);
-    const int p_first = first / kPage, p_last = pos / kPage;
-    const int per = (p_last - p_first + n_splits) / n_splits;      // pages per split, rounded up
-    const int p0 = p_first + split * per, p1 = min(p_last, p0 + per - 1);
+    const PageWalk walk(first, pos, keep);
+    const int p_last = pos / kPage;
+    const int per = (walk.n + n_splits - 1) / n_splits;            // pages per split, rounded up
+    const int p0 = split * per, p1 = min(walk.n - 1, p0 + per - 1);   // this split's part of the walk
     const int* table = block_table + (size_t)seq * bt_stride;
 
     auto issue = [&](int page_idx, int stage) {
         // kv_rep > 1: more than 16 heads share a key/value head, and kv_rep blocks each serve a part of them from
         // the same pages (n_kv counts those blocks; the pages hold n_kv / kv_rep heads)
-        const size_t base = ((size_t)table[page_idx] * (n_kv / kv_rep) + kvh / kv_rep) * (size_t)(kPage * HD);
-        const uint32_t dst = smem_u32_(dsm) + stage * 2 * kTileBytes;
+        const size_t head_row = ((size_t)table[walk.page(page_idx)] * (n_kv / kv_rep) + kvh / kv_rep) * (size_t)kPage;
+        const uint32_t dst = smem_u32_(dsm) + stage * kStageBytes;
 #pragma unroll
         for (int i = threadIdx.x; i < kPage * kChunks; i += 128) {
             const int row = i / kChunks, chunk = i % kChunks;
-            cp_async16(dst + tile_off<HD>(row, chunk), k_pages + base + (size_t)row * HD + chunk * 8);
-            cp_async16(dst + kTileBytes + tile_off<HD>(row, chunk), v_pages + base + (size_t)row * HD + chunk * 8);
+            cp_async16(dst + tile_off<HD>(row, chunk), k_pages + (head_row + row) * HD + chunk * 8);
+            if (VD == HD) cp_async16(dst + kTileBytes + tile_off<VD>(row, chunk), v_pages + (head_row + row) * VD + chunk * 8);
+        }
+        if (VD != HD) {
+#pragma unroll
+            for (int i = threadIdx.x; i < kPage * kVChunks; i += 128) {
+                const int row = i / kVChunks, chunk = i % kVChunks;
+                cp_async16(dst + kTileBytes + tile_off<VD>(row, chunk), v_pages + (head_row + row) * VD + chunk * 8);
+            }
         }
     };
     // two pages ahead; an empty commit keeps the group count in step when there is nothing to fetch
@@ -454,27 +525,35 @@ decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restri
     // position, the token's key and value (appended to the cache for later steps; for this step they are put into
     // the block's copy of the page when that has arrived).
     __shared__ __align__(16) __nv_bfloat16 q_s[kFused ? 16 * HD : 8];
-    __shared__ __align__(16) __nv_bfloat16 kv_s[kFused ? 2 * HD : 8];
-    const bool owner = kFused && f.k_pages != nullptr && p0 <= p_last && p_last <= p1;
+    __shared__ __align__(16) __nv_bfloat16 kv_s[kFused ? HD + VD : 8];
+    __shared__ float sq_s[4];
+    const bool owner = kFused && f.k_pages != nullptr && p0 <= walk.n - 1 && walk.n - 1 <= p1;
     if constexpr (kFused) {
-        const float* row = f.qkv + (size_t)t * f.per_tok * HD;
-        const float2* cs_row = f.cs ? f.cs + (size_t)t * (HD / 2) : nullptr;
+        const float* row = f.qkv + (size_t)t * f.ld;
+        const float2* cs_row = f.cs ? f.cs + (size_t)t * f.half : nullptr;
+        float q_scale = 0.0f, k_scale = 0.0f;      // a norm over all the heads: its scale is the same for every block
+        if (f.whole) {
+            if (f.q_gamma) q_scale = 1.0f / sqrtf(row_squares(row, n_heads * f.hd, sq_s) * (1.0f / (float)(n_heads * f.hd)) + f.eps);
+            if (f.k_gamma && owner) k_scale = 1.0f / sqrtf(row_squares(row + f.k_at, n_kv * f.hd, sq_s) * (1.0f / (float)(n_kv * f.hd)) + f.eps);
+        }
         const float temp = f.temp_coef != 0.0f ? 1.0f + f.temp_coef * logf((float)((pos + 1) / f.temp_every) + 1.0f) : 1.0f;
         for (int g = warp; g < G; g += 4)
-            finish_head<HD>(row + (size_t)(kvh * G + g) * HD, f.q_gamma, f.g_dt, f.eps, cs_row, q_s + g * HD, lane, temp);
+            finish_head<HD>(row + (size_t)(kvh * G + g) * f.hd, f.hd, f.q_gamma, f.whole ? (kvh * G + g) * f.hd : 0, f.g_dt,
+                            f.eps, q_scale, cs_row, f.half, f.pairs, q_s + g * HD, lane, temp);
         if (owner) {
             if (warp == 0)
-                finish_head<HD>(row + (size_t)(n_heads + kvh) * HD, f.k_gamma, f.g_dt, f.eps, cs_row, kv_s, lane);
+                finish_head<HD>(row + f.k_at + (size_t)kvh * f.hd, f.hd, f.k_gamma, f.whole ? kvh * f.hd : 0, f.g_dt, f.eps,
+                                k_scale, cs_row, f.half, f.pairs, kv_s, lane);
             if (warp == 1)
-                finish_head<HD>(row + (size_t)(n_heads + (f.values_are_keys ? 0 : n_kv) + kvh) * HD, nullptr, 0, 0.0f, nullptr,
-                                kv_s + HD, lane);
+                finish_head<VD>(row + f.v_at + (size_t)kvh * f.vd, f.vd, nullptr, 0, 0, 0.0f, 0.0f, nullptr, 0, 0, kv_s + HD, lane);
         }
         __syncthreads();
-        if (owner && threadIdx.x < 2 * kChunks) {
-            const int which = threadIdx.x / kChunks, chunk = threadIdx.x % kChunks;
-            __nv_bfloat16* page = (which ? f.v_pages : f.k_pages) +
-                                  (((size_t)table[p_last] * n_kv + kvh) * kPage + pos % kPage) * (size_t)HD;
-            *reinterpret_cast<uint4*>(page + chunk * 8) = *reinterpret_cast<const uint4*>(kv_s + which * HD + chunk * 8);
+        if (owner && threadIdx.x < kChunks + kVChunks) {
+            const bool is_v = threadIdx.x >= kChunks;
+            const int chunk = is_v ? threadIdx.x - kChunks : threadIdx.x;
+            const size_t page_row = ((size_t)table[p_last] * n_kv + kvh) * kPage + pos % kPage;
+            __nv_bfloat16* page = is_v ? f.v_pages + page_row * VD : f.k_pages + page_row * HD;
+            *reinterpret_cast<uint4*>(page + chunk * 8) = *reinterpret_cast<const uint4*>(kv_s + (is_v ? HD : 0) + chunk * 8);
         }
     }
     // queries of the heads 8 * tt + r as right-hand operands: (lanes 2c, 2c + 1) and (2c + 8, 2c + 9) of each 16
@@ -482,19 +561,20 @@ decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restri
 #pragma unroll
     for (int tt = 0; tt < NT; ++tt) {
         const bool ok = 8 * tt + r < G;
-        const __nv_bfloat16* qrow = kFused ? q_s + (size_t)(8 * tt + r) * HD : q + out_row + (size_t)(8 * tt + r) * HD;
+        const __nv_bfloat16* qrow = kFused ? q_s + (size_t)(8 * tt + r) * HD
+                                           : q + ((size_t)t * n_heads + (size_t)kvh * G + 8 * tt + r) * HD;
 #pragma unroll
         for (int ks = 0; ks < HD / 16; ++ks) {
             qb[tt][ks][0] = ok ? *reinterpret_cast<const uint32_t*>(qrow + ks * 16 + 2 * c) : 0u;
             qb[tt][ks][1] = ok ? *reinterpret_cast<const uint32_t*>(qrow + ks * 16 + 8 + 2 * c) : 0u;
         }
     }
-    float o[NT][HD / 16][4];
+    float o[NT][VD / 16][4];
     float m[NT][2], l[NT][2];
 #pragma unroll
     for (int tt = 0; tt < NT; ++tt) {
 #pragma unroll
-        for (int i = 0; i < HD / 16; ++i) o[tt][i][0] = o[tt][i][1] = o[tt][i][2] = o[tt][i][3] = 0.0f;
+        for (int i = 0; i < VD / 16; ++i) o[tt][i][0] = o[tt][i][1] = o[tt][i][2] = o[tt][i][3] = 0.0f;
         m[tt][0] = m[tt][1] = -INFINITY;
         l[tt][0] = l[tt][1] = 0.0f;
     }
@@ -505,22 +585,24 @@ decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restri
         __syncthreads();           // everybody's have, and everybody is done with the stage refilled next
         if (pg + 2 <= p1) issue(pg + 2, (pg + 2 - p0) % kDecodeStages);
         cp_async_commit();
-        if (kFused && owner && pg == p_last) {
+        if (kFused && owner && pg == walk.n - 1) {
             // the token's own key and value take their row of the page that has just arrived
-            if (threadIdx.x < 2 * kChunks) {
-                const int which = threadIdx.x / kChunks, chunk = threadIdx.x % kChunks;
-                *reinterpret_cast<uint4*>(dsm + stage * 2 * kTileBytes + which * kTileBytes + tile_off<HD>(pos % kPage, chunk)) =
-                    *reinterpret_cast<const uint4*>(kv_s + which * HD + chunk * 8);
+            if (threadIdx.x < kChunks + kVChunks) {
+                const bool is_v = threadIdx.x >= kChunks;
+                const int chunk = is_v ? threadIdx.x - kChunks : threadIdx.x;
+                const uint32_t at = is_v ? kTileBytes + tile_off<VD>(pos % kPage, chunk) : tile_off<HD>(pos % kPage, chunk);
+                *reinterpret_cast<uint4*>(dsm + stage * kStageBytes + at) =
+                    *reinterpret_cast<const uint4*>(kv_s + (is_v ? HD : 0) + chunk * 8);
             }
             __syncthreads();
         }
-        const int k0 = pg * kPage + 16 * warp;             // this warp's 16 keys of the page
-        if (k0 > pos || k0 + 15 < first) continue;
-        const uint32_t ks_addr = smem_u32_(dsm) + stage * 2 * kTileBytes;
+        const int k0 = walk.page(pg) * kPage + 16 * warp;  // this warp's 16 keys of the page
+        if (k0 > pos || (k0 + 15 < first && k0 >= keep)) continue;
+        const uint32_t ks_addr = smem_u32_(dsm) + stage * kStageBytes;
         const uint32_t vs_addr = ks_addr + kTileBytes;
         const bool inside = k0 >= first && k0 + 15 <= pos;
-        const bool lo_ok = inside || (k0 + r >= first && k0 + r <= pos);
-        const bool hi_ok = inside || (k0 + r + 8 >= first && k0 + r + 8 <= pos);
+        const bool lo_ok = inside || ((k0 + r >= first || k0 + r < keep) && k0 + r <= pos);
+        const bool hi_ok = inside || ((k0 + r + 8 >= first || k0 + r + 8 < keep) && k0 + r + 8 <= pos);
         // S^T = K . Q^T : 16 keys x 8 heads per column tile
         float s[NT][4];
 #pragma unroll
@@ -576,17 +658,17 @@ decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restri
 #pragma unroll
             for (int tt = 0; tt < NT; ++tt)
 #pragma unroll
-                for (int i = 0; i < HD / 16; ++i) {
+                for (int i = 0; i < VD / 16; ++i) {
                     o[tt][i][0] *= corr[tt][0]; o[tt][i][1] *= corr[tt][1];
                     o[tt][i][2] *= corr[tt][0]; o[tt][i][3] *= corr[tt][1];
                 }
         }
         // O^T += V^T . P^T : 16 head lanes per row tile
 #pragma unroll
-        for (int dt = 0; dt < HD / 16; ++dt) {
+        for (int dt = 0; dt < VD / 16; ++dt) {
             uint32_t a[4];
             const int key = 16 * warp + (lane >> 4) * 8 + (lane & 7);
-            ldmatrix_x4_trans(a, vs_addr + tile_off<HD>(key, dt * 2 + ((lane >> 3) & 1)));
+            ldmatrix_x4_trans(a, vs_addr + tile_off<VD>(key, dt * 2 + ((lane >> 3) & 1)));
 #pragma unroll
             for (int tt = 0; tt < NT; ++tt) mma_bf16(o[tt][dt], a[0], a[1], a[2], a[3], pb[tt][0], pb[tt][1]);
         }
@@ -608,46 +690,46 @@ decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restri
             const int head = 8 * tt + 2 * c + e;
             if (head < G) {
 #pragma unroll
-                for (int i = 0; i < HD / 16; ++i) {
+                for (int i = 0; i < VD / 16; ++i) {
                     mine[head * W + i * 16 + r] = o[tt][i][e];
                     mine[head * W + i * 16 + r + 8] = o[tt][i][2 + e];
                 }
                 if (r == 0) {
-                    mine[head * W + HD] = m[tt][e];
-                    mine[head * W + HD + 1] = l[tt][e];
+                    mine[head * W + VD] = m[tt][e];
+                    mine[head * W + VD + 1] = l[tt][e];
                 }
             }
         }
     __syncthreads();
     const size_t pbase = ((size_t)t * n_kv + kvh) * n_splits + split;
     float* merged = sm + (size_t)4 * G * W;
-    for (int i = threadIdx.x; i < G * HD; i += 128) {
-        const int head = i / HD, d = i % HD;
+    for (int i = threadIdx.x; i < G * VD; i += 128) {
+        const int head = i / VD, d = i % VD;
         float mm = -INFINITY;
 #pragma unroll
-        for (int w = 0; w < 4; ++w) mm = fmaxf(mm, sm[(w * G + head) * W + HD]);
+        for (int w = 0; w < 4; ++w) mm = fmaxf(mm, sm[(w * G + head) * W + VD]);
         float oo = 0.0f, ll = 0.0f;
 #pragma unroll
         for (int w = 0; w < 4; ++w) {
-            const float mw = sm[(w * G + head) * W + HD];
+            const float mw = sm[(w * G + head) * W + VD];
             const float cw = mw == -INFINITY ? 0.0f : exp2f(mw - mm);
             oo = fmaf(sm[(w * G + head) * W + d], cw, oo);
-            ll = fmaf(sm[(w * G + head) * W + HD + 1], cw, ll);
+            ll = fmaf(sm[(w * G + head) * W + VD + 1], cw, ll);
         }
         if (n_splits == 1) {
             if (sinks != nullptr && ll > 0.0f) ll += exp2f(sinks[kvh * G + head] * kLog2e - mm);
             float res = ll > 0.0f ? oo / ll : 0.0f;
             if (kFused && f.gate_at >= 0)
-                res *= 1.0f / (1.0f + expf(-f.qkv[((size_t)t * f.per_tok + f.gate_at + kvh * G + head) * HD + d]));
-            out[out_row + i] = __float2bfloat16_rn(res);
+                res *= 1.0f / (1.0f + expf(-f.qkv[(size_t)t * f.ld + f.gate_at + (size_t)(kvh * G + head) * vo + min(d, vo - 1)]));
+            if (d < vo) out[out_row + (size_t)head * vo + d] = __float2bfloat16_rn(res);
         } else if (kCluster) {
             merged[head * W + d] = oo;
             if (d == 0) {
-                merged[head * W + HD] = mm;
-                merged[head * W + HD + 1] = ll;
+                merged[head * W + VD] = mm;
+                merged[head * W + VD + 1] = ll;
             }
         } else {
-            part_o[pbase * G * HD + i] = oo;
+            part_o[pbase * G * VD + i] = oo;
             if (d == 0) {
                 part_ml[(pbase * G + head) * 2] = mm;
                 part_ml[(pbase * G + head) * 2 + 1] = ll;
@@ -656,19 +738,19 @@ decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restri
     }
     if (kCluster && n_splits > 1) {
         cluster_barrier_();   // every split's result is in its block's shared memory
-        const int total = G * HD, share = (total + n_splits - 1) / n_splits;
+        const int total = G * VD, share = (total + n_splits - 1) / n_splits;
         const int rank = (int)cluster_rank_();
         for (int i = rank * share + threadIdx.x; i < min(total, (rank + 1) * share); i += 128) {
-            const int head = i / HD, d = i % HD;
+            const int head = i / VD, d = i % VD;
             // all the loads from the other blocks' shared memory are issued before the first is used: one trip
             // through the cluster, not one per split
             float ms[kMaxClusterSplits], os[kMaxClusterSplits], ls[kMaxClusterSplits];
 #pragma unroll
             for (int sp = 0; sp < kMaxClusterSplits; ++sp) {
                 if (sp < n_splits) {
-                    ms[sp] = ld_cluster_(merged + head * W + HD, sp);
+                    ms[sp] = ld_cluster_(merged + head * W + VD, sp);
                     os[sp] = ld_cluster_(merged + head * W + d, sp);
-                    ls[sp] = ld_cluster_(merged + head * W + HD + 1, sp);
+                    ls[sp] = ld_cluster_(merged + head * W + VD + 1, sp);
                 }
             }
             float mm = -INFINITY;
@@ -687,43 +769,44 @@ decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restri
             if (sinks != nullptr && ll > 0.0f) ll += exp2f(sinks[kvh * G + head] * kLog2e - mm);
             float res = ll > 0.0f ? oo / ll : 0.0f;
             if (kFused && f.gate_at >= 0)
-                res *= 1.0f / (1.0f + expf(-f.qkv[((size_t)t * f.per_tok + f.gate_at + kvh * G + head) * HD + d]));
-            out[out_row + i] = __float2bfloat16_rn(res);
+                res *= 1.0f / (1.0f + expf(-f.qkv[(size_t)t * f.ld + f.gate_at + (size_t)(kvh * G + head) * vo + min(d, vo - 1)]));
+            if (d < vo) out[out_row + (size_t)head * vo + d] = __float2bfloat16_rn(res);
         }
         cluster_barrier_();   // no block leaves while its result may still be read
     }
 }
 
-template <int HD>
+template <int HD, int VD>
 int launch_decode(const void* q, const void* k_pages, const void* v_pages, const int* block_table, int bt_stride,
                   const int* tok_seq, const int* tok_pos, void* out, float* scratch, int n_tok, int n_heads, int n_kv,
-                  float scale, int window, int n_splits, cudaStream_t stream, const FusedQK* fused = nullptr,
+                  float scale, int window, int keep, int vo, int n_splits, cudaStream_t stream, const FusedQK* fused = nullptr,
                   float slope_base = 0.0f, const float* sinks = nullptr) {
     using Kernel = void (*)(const __nv_bfloat16*, const __nv_bfloat16*, const __nv_bfloat16*, const int*, int, const int*,
-                            const int*, __nv_bfloat16*, float*, float*, int, int, float, int, const FusedQK, const float*, int);
+                            const int*, __nv_bfloat16*, float*, float*, int, int, float, int, int, const FusedQK, const float*,
+                            int, int);
     // a block serves at most 16 heads of a key/value head: where more share one, kv_rep blocks take a part each
     int kv_rep = 1;
     while ((n_heads / n_kv) % kv_rep != 0 || n_heads / n_kv / kv_rep > 16) ++kv_rep;
     n_kv *= kv_rep;
     const int G = n_heads / n_kv;
     float* part_o = scratch;
-    float* part_ml = scratch ? scratch + (size_t)n_tok * n_kv * n_splits * G * HD : nullptr;
+    float* part_ml = scratch ? scratch + (size_t)n_tok * n_kv * n_splits * G * VD : nullptr;
     // without scratch the splits merge inside a cluster (the caller checked n_splits <= 8)
     const bool cluster = scratch == nullptr && n_splits > 1;
-    const Kernel plain = cluster ? (G <= 8 ? (Kernel)decode_kernel<HD, 1, true, false> : (Kernel)decode_kernel<HD, 2, true, false>)
-                                 : (G <= 8 ? (Kernel)decode_kernel<HD, 1, false, false> : (Kernel)decode_kernel<HD, 2, false, false>);
-    const Kernel from_qkv = cluster ? (G <= 8 ? (Kernel)decode_kernel<HD, 1, true, true> : (Kernel)decode_kernel<HD, 2, true, true>)
-                                    : (G <= 8 ? (Kernel)decode_kernel<HD, 1, false, true> : (Kernel)decode_kernel<HD, 2, false, true>);
+    const Kernel plain = cluster ? (G <= 8 ? (Kernel)decode_kernel<HD, VD, 1, true, false> : (Kernel)decode_kernel<HD, VD, 2, true, false>)
+                                 : (G <= 8 ? (Kernel)decode_kernel<HD, VD, 1, false, false> : (Kernel)decode_kernel<HD, VD, 2, false, false>);
+    const Kernel from_qkv = cluster ? (G <= 8 ? (Kernel)decode_kernel<HD, VD, 1, true, true> : (Kernel)decode_kernel<HD, VD, 2, true, true>)
+                                    : (G <= 8 ? (Kernel)decode_kernel<HD, VD, 1, false, true> : (Kernel)decode_kernel<HD, VD, 2, false, true>);
     const Kernel kernel = fused ? from_qkv : plain;
     FusedQK f = fused ? *fused : FusedQK{};
     if (!fused) f.slope_base = slope_base;
-    const size_t stages = (size_t)kDecodeStages * 2 * kPage * HD * 2;
-    const size_t merge = (size_t)5 * G * (HD + 2) * sizeof(float);
+    const size_t stages = (size_t)kDecodeStages * kPage * (HD + VD) * 2;
+    const size_t merge = (size_t)5 * G * (VD + 2) * sizeof(float);
     const size_t smem = stages > merge ? stages : merge;
     static bool configured[8][64] = {};
     if (first_use_on_this_device(configured[(fused ? 4 : 0) + (cluster ? 2 : 0) + (G <= 8 ? 0 : 1)])) {
         const cudaError_t e = cudaFuncSetAttribute((const void*)kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                                   (int)(stages > (size_t)5 * 16 * (HD + 2) * 4 ? stages : (size_t)5 * 16 * (HD + 2) * 4));
+                                                   (int)(stages > (size_t)5 * 16 * (VD + 2) * 4 ? stages : (size_t)5 * 16 * (VD + 2) * 4));
         NN_CHECK(e == cudaSuccess, "attention decode: cannot reserve shared memory: %s", cudaGetErrorString(e));
     }
     cudaLaunchConfig_t cfg = {};
@@ -740,36 +823,36 @@ int launch_decode(const void* q, const void* k_pages, const void* v_pages, const
     cfg.numAttrs = cluster ? 1 : 0;
     const cudaError_t e = cudaLaunchKernelEx(&cfg, kernel, (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pages,
                                              (const __nv_bfloat16*)v_pages, block_table, bt_stride, tok_seq, tok_pos,
-                                             (__nv_bfloat16*)out, part_o, part_ml, n_heads, n_kv, scale * kLog2e, window, f,
-                                             sinks, kv_rep);
+                                             (__nv_bfloat16*)out, part_o, part_ml, n_heads, n_kv, scale * kLog2e, window, keep, f,
+                                             sinks, kv_rep, vo);
     NN_CHECK(e == cudaSuccess, "attention decode (%d splits%s): launch failed: %s", n_splits, cluster ? ", cluster" : "",
              cudaGetErrorString(e));
     if (n_splits > 1 && !cluster) {
         const bool gated = fused && fused->gate_at >= 0;
-        merge_kernel<HD><<<dim3(n_heads, n_tok), HD, 0, stream>>>(
+        merge_kernel<VD><<<dim3(n_heads, n_tok), VD, 0, stream>>>(
             part_o, part_ml, (__nv_bfloat16*)out, n_heads, n_kv, n_splits, sinks,
-            gated ? f.qkv + (size_t)f.gate_at * HD : nullptr, gated ? (long)f.per_tok * HD : 0l);
+            gated ? f.qkv + f.gate_at : nullptr, gated ? (long)f.ld : 0l, vo);
         NN_LAUNCH_OK("attention merge");
     }
     return 0;
 }
 
-template <int HD>
+template <int HD, int VD>
 int launch_prefill(const void* q, const void* k_pages, const void* v_pages, const int* block_table, int bt_stride,
                    const int* cu_seqlens, const int* tok_pos, void* out, int n_tok, int n_seqs, int n_heads, int n_kv,
-                   float scale, int window, float slope_base, const float* sinks, cudaStream_t stream) {
+                   float scale, int window, int keep, int vo, float slope_base, const float* sinks, cudaStream_t stream) {
     const int max_tiles = n_tok / 64 + n_seqs;
-    constexpr int smem = 2 * 2 * kPage * HD * 2;
+    constexpr int smem = 2 * kPage * (HD + VD) * 2;
     static bool configured[64] = {};
     if (first_use_on_this_device(configured)) {
-        const cudaError_t e = cudaFuncSetAttribute(prefill_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        const cudaError_t e = cudaFuncSetAttribute(prefill_kernel<HD, VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         NN_CHECK(e == cudaSuccess, "attention prefill: cannot reserve shared memory: %s", cudaGetErrorString(e));
     }
     dim3 grid(max_tiles, n_heads);
-    prefill_kernel<HD><<<grid, 128, smem, stream>>>((const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pages,
+    prefill_kernel<HD, VD><<<grid, 128, smem, stream>>>((const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pages,
                                                  (const __nv_bfloat16*)v_pages, block_table, bt_stride, cu_seqlens,
                                                  tok_pos, (__nv_bfloat16*)out, n_seqs, n_heads, n_kv, scale * kLog2e,
-                                                 window, slope_base, sinks);
+                                                 window, keep, slope_base, sinks, vo);
     NN_LAUNCH_OK("attention prefill");
     return 0;
 }
@@ -781,11 +864,15 @@ extern "C" int nncpu_attention_mma_supported(int n_heads, int n_kv, int hd) {
     return (hd == 64 || hd == 128) && n_kv > 0 && n_heads % n_kv == 0;
 }
 
+// Lanes of the pages' value rows and of a value head in the output: rows as long as the keys' or of 64 lanes, heads
+// that fit them.
+static bool value_size_ok(int hd, int vp, int vo) { return (vp == hd || vp == 64) && vo > 0 && vo <= vp; }
+
 // Floats of scratch the decode kernel needs for n_tok tokens cut into n_splits splits (0 for one split).
-extern "C" long nncpu_attention_decode_scratch_floats(int n_tok, int n_heads, int n_kv, int hd, int n_splits) {
+extern "C" long nncpu_attention_decode_scratch_floats(int n_tok, int n_heads, int n_kv, int vp, int n_splits) {
     if (n_splits <= 1) return 0;
     const long G = n_heads / n_kv;
-    return (long)n_tok * n_kv * n_splits * G * (hd + 2);
+    return (long)n_tok * n_kv * n_splits * G * (vp + 2);
 }
 
 // One token per sequence: token t belongs to sequence tok_seq[t] (negative: padding) and sits at
@@ -793,8 +880,10 @@ extern "C" long nncpu_attention_decode_scratch_floats(int n_tok, int n_heads, in
 extern "C" int nncpu_attention_decode_mma(const void* q, const void* k_pages, const void* v_pages,
                                           const int* block_table, int bt_stride, const int* tok_seq,
                                           const int* tok_pos, void* out, float* scratch, long scratch_floats,
-                                          int n_tok, int n_heads, int n_kv, int hd, float scale, int window,
-                                          int n_splits, float slope_base, const float* sinks, void* stream) {
+                                          int n_tok, int n_heads, int n_kv, int hd, int vp, int vo, float scale, int window,
+                                          int keep, int n_splits, float slope_base, const float* sinks, void* stream) {
+    // pages of keys have rows of hd lanes, pages of values rows of vp; a head's output has vo lanes.  keep: with a
+    // window, the sequence's first keys that stay visible.
     NN_CHECK(nncpu_attention_mma_supported(n_heads, n_kv, hd),
              "attention (tensor cores): %d heads over %d key/value heads of size %d is not supported "
              "(head size 64 or 128, heads a multiple of key/value heads)", n_heads, n_kv, hd);
@@ -803,28 +892,35 @@ extern "C" int nncpu_attention_decode_mma(const void* q, const void* k_pages, co
     if (scratch == nullptr && n_splits > 1)
         NN_CHECK(n_splits <= 8, "attention decode: %d splits without scratch (a cluster merges at most 8)", n_splits);
     else
-        NN_CHECK(scratch_floats >= nncpu_attention_decode_scratch_floats(n_tok, n_heads, n_kv, hd, n_splits),
+        NN_CHECK(scratch_floats >= nncpu_attention_decode_scratch_floats(n_tok, n_heads, n_kv, vp, n_splits),
                  "attention decode: %ld floats of scratch, %ld needed", scratch_floats,
-                 nncpu_attention_decode_scratch_floats(n_tok, n_heads, n_kv, hd, n_splits));
+                 nncpu_attention_decode_scratch_floats(n_tok, n_heads, n_kv, vp, n_splits));
+    NN_CHECK(value_size_ok(hd, vp, vo) && keep >= 0, "attention decode: value rows of %d lanes, %d of them used", vp, vo);
     if (n_tok == 0) return 0;
-    if (hd == 64)
-        return launch_decode<64>(q, k_pages, v_pages, block_table, bt_stride, tok_seq, tok_pos, out, scratch, n_tok,
-                                 n_heads, n_kv, scale, window, n_splits, (cudaStream_t)stream, nullptr, slope_base, sinks);
-    return launch_decode<128>(q, k_pages, v_pages, block_table, bt_stride, tok_seq, tok_pos, out, scratch, n_tok,
-                              n_heads, n_kv, scale, window, n_splits, (cudaStream_t)stream, nullptr, slope_base, sinks);
+#define NN_DECODE(HD_, VD_)                                                                                                 \
+    return launch_decode<HD_, VD_>(q, k_pages, v_pages, block_table, bt_stride, tok_seq, tok_pos, out, scratch, n_tok,      \
+                                   n_heads, n_kv, scale, window, keep, vo, n_splits, (cudaStream_t)stream, nullptr, slope_base, sinks)
+    if (hd == 64) NN_DECODE(64, 64);
+    if (vp == 64) NN_DECODE(128, 64);
+    NN_DECODE(128, 128);
+#undef NN_DECODE
 }
 
 // The same from the float32 projections: qkv [n_tok, per_tok * hd] holds, per token, the heads of q and, if `append`,
 // of k and v after them (per_tok = n_heads + 2 n_kv, else n_heads).  Every block makes its queries itself (per-head RMS
 // norm with q_gamma if given, rotation by cos_sin [n_tok, hd / 2, 2] if given); with `append` the token's key (k_gamma,
 // rotation) and value are made too, written to their row of the cache pages and used in this step.  Replaces the
-// separate kernel for norm, rotation and append in a decode step; the arithmetic is the same.
+// separate kernel for norm, rotation and append in a decode step; the arithmetic is the same.  A head has head_dim
+// lanes in the rows of qkv (value heads v_head_dim) and hd (vp) in the pages' rows, zeros behind it.  whole_norm: the norm
+// runs over all of a token's query (key) lanes at once, with as many weights.  rot_pairs: neighbouring lanes are the
+// pairs, and rot_half of them turn (otherwise lanes (i, i + hd / 2) of the whole head).
 extern "C" int nncpu_attention_decode_mma_from_qkv(const float* qkv, const void* q_gamma, const void* k_gamma, int g_dt,
                                                    float eps, const float* cos_sin, void* k_pages, void* v_pages,
                                                    int append, const int* block_table, int bt_stride,
                                                    const int* tok_seq, const int* tok_pos, void* out, float* scratch,
-                                                   long scratch_floats, int n_tok, int n_heads, int n_kv, int hd,
-                                                   float scale, int window, int n_splits, float slope_base,
+                                                   long scratch_floats, int n_tok, int n_heads, int n_kv, int hd, int vp,
+                                                   int head_dim, int v_head_dim, int whole_norm, int rot_half,
+                                                   int rot_pairs, float scale, int window, int keep, int n_splits, float slope_base,
                                                    float temp_coef, int temp_every, const float* sinks,
                                                    int values_are_keys, int gated, void* stream) {
     NN_CHECK(nncpu_attention_mma_supported(n_heads, n_kv, hd),
@@ -841,18 +937,29 @@ extern "C" int nncpu_attention_decode_mma_from_qkv(const float* qkv, const void*
     if (scratch == nullptr && n_splits > 1)
         NN_CHECK(n_splits <= 8, "attention decode: %d splits without scratch (a cluster merges at most 8)", n_splits);
     else
-        NN_CHECK(scratch_floats >= nncpu_attention_decode_scratch_floats(n_tok, n_heads, n_kv, hd, n_splits),
+        NN_CHECK(scratch_floats >= nncpu_attention_decode_scratch_floats(n_tok, n_heads, n_kv, vp, n_splits),
                  "attention decode: %ld floats of scratch, %ld needed", scratch_floats,
-                 nncpu_attention_decode_scratch_floats(n_tok, n_heads, n_kv, hd, n_splits));
+                 nncpu_attention_decode_scratch_floats(n_tok, n_heads, n_kv, vp, n_splits));
     if (n_tok == 0) return 0;
     FusedQK f{};
     f.qkv = qkv;
+    NN_CHECK(value_size_ok(hd, vp, v_head_dim) && keep >= 0 && head_dim > 0 && head_dim <= hd && (!values_are_keys || v_head_dim == head_dim),
+             "attention decode (from projections): heads of %d and %d lanes in rows of %d and %d", head_dim, v_head_dim, hd, vp);
+    NN_CHECK(cos_sin == nullptr || (rot_pairs ? 2 * rot_half <= head_dim : (2 * rot_half == hd && head_dim == hd)),
+             "attention decode (from projections): %d rotated pairs of a head of %d lanes", rot_half, head_dim);
     // a token's row: the heads of q, then (if appended here) of k and, unless the values are the keys, of v, then
-    // (if gated) as many heads of gate logits as of q
-    const int kv_heads_in_row = append ? (values_are_keys ? n_kv : 2 * n_kv) : 0;
-    f.per_tok = n_heads + kv_heads_in_row + (gated ? n_heads : 0);
+    // (if gated) a gate logit for every lane of the output
+    f.hd = head_dim;
+    f.vd = v_head_dim;
+    f.k_at = n_heads * head_dim;
+    f.v_at = values_are_keys ? f.k_at : f.k_at + n_kv * head_dim;
+    const int gate_at = n_heads * head_dim + (append ? n_kv * head_dim + (values_are_keys ? 0 : n_kv * v_head_dim) : 0);
+    f.ld = gate_at + (gated ? n_heads * v_head_dim : 0);
+    f.whole = whole_norm;
+    f.half = rot_half;
+    f.pairs = rot_pairs;
     f.values_are_keys = values_are_keys;
-    f.gate_at = gated ? n_heads + kv_heads_in_row : -1;
+    f.gate_at = gated ? gate_at : -1;
     f.q_gamma = q_gamma; f.k_gamma = k_gamma; f.g_dt = g_dt; f.eps = eps;
     f.cs = (const float2*)cos_sin;
     f.k_pages = append ? (__nv_bfloat16*)k_pages : nullptr;
@@ -861,11 +968,13 @@ extern "C" int nncpu_attention_decode_mma_from_qkv(const float* qkv, const void*
     f.slope_base = slope_base;
     f.temp_coef = temp_coef;
     f.temp_every = temp_every;
-    if (hd == 64)
-        return launch_decode<64>(nullptr, k_pages, v_pages, block_table, bt_stride, tok_seq, tok_pos, out, scratch, n_tok,
-                                 n_heads, n_kv, scale, window, n_splits, (cudaStream_t)stream, &f, 0.0f, sinks);
-    return launch_decode<128>(nullptr, k_pages, v_pages, block_table, bt_stride, tok_seq, tok_pos, out, scratch, n_tok,
-                              n_heads, n_kv, scale, window, n_splits, (cudaStream_t)stream, &f, 0.0f, sinks);
+#define NN_DECODE(HD_, VD_)                                                                                                 \
+    return launch_decode<HD_, VD_>(nullptr, k_pages, v_pages, block_table, bt_stride, tok_seq, tok_pos, out, scratch, n_tok, \
+                                   n_heads, n_kv, scale, window, keep, v_head_dim, n_splits, (cudaStream_t)stream, &f, 0.0f, sinks)
+    if (hd == 64) NN_DECODE(64, 64);
+    if (vp == 64) NN_DECODE(128, 64);
+    NN_DECODE(128, 128);
+#undef NN_DECODE
 }
 
 // Any mix of new tokens per sequence: sequence b brings the flat tokens cu_seqlens[b] .. cu_seqlens[b + 1] - 1
@@ -873,18 +982,21 @@ extern "C" int nncpu_attention_decode_mma_from_qkv(const float* qkv, const void*
 extern "C" int nncpu_attention_prefill_mma(const void* q, const void* k_pages, const void* v_pages,
                                            const int* block_table, int bt_stride, const int* cu_seqlens,
                                            const int* tok_pos, void* out, int n_tok, int n_seqs, int n_heads,
-                                           int n_kv, int hd, float scale, int window, float slope_base, const float* sinks,
-                                           void* stream) {
+                                           int n_kv, int hd, int vp, int vo, float scale, int window, int keep,
+                                           float slope_base, const float* sinks, void* stream) {
     NN_CHECK(nncpu_attention_mma_supported(n_heads, n_kv, hd),
              "attention (tensor cores): %d heads over %d key/value heads of size %d is not supported "
              "(head size 64 or 128, heads a multiple of key/value heads)", n_heads, n_kv, hd);
     NN_CHECK(n_tok >= 0 && n_seqs >= 0, "attention prefill: %d tokens of %d sequences", n_tok, n_seqs);
+    NN_CHECK(value_size_ok(hd, vp, vo) && keep >= 0, "attention prefill: value rows of %d lanes, %d of them used", vp, vo);
     if (n_tok == 0 || n_seqs == 0) return 0;
-    if (hd == 64)
-        return launch_prefill<64>(q, k_pages, v_pages, block_table, bt_stride, cu_seqlens, tok_pos, out, n_tok, n_seqs,
-                                  n_heads, n_kv, scale, window, slope_base, sinks, (cudaStream_t)stream);
-    return launch_prefill<128>(q, k_pages, v_pages, block_table, bt_stride, cu_seqlens, tok_pos, out, n_tok, n_seqs,
-                               n_heads, n_kv, scale, window, slope_base, sinks, (cudaStream_t)stream);
+#define NN_PREFILL(HD_, VD_)                                                                                                \
+    return launch_prefill<HD_, VD_>(q, k_pages, v_pages, block_table, bt_stride, cu_seqlens, tok_pos, out, n_tok, n_seqs,   \
+                                    n_heads, n_kv, scale, window, keep, vo, slope_base, sinks, (cudaStream_t)stream)
+    if (hd == 64) NN_PREFILL(64, 64);
+    if (vp == 64) NN_PREFILL(128, 64);
+    NN_PREFILL(128, 128);
+#undef NN_PREFILL
 }
 
 // ---------------------------------------------------------------------------
@@ -964,5 +1076,5 @@ extern "C" int nncpu_attention_decode_mma_static(const void* q, const void* k_pa
     float* scratch = nullptr;
     if (int e = static_scratch(&scratch)) return e;
     return nncpu_attention_decode_mma(q, k_pages, v_pages, block_table, bt_stride, tok_seq, tok_pos, out, scratch,
-                                      kStaticScratchFloats, n_tok, n_heads, n_kv, hd, scale, window, n_splits, 0.0f, nullptr, stream);
+                                      kStaticScratchFloats, n_tok, n_heads, n_kv, hd, hd, hd, scale, window, 0, n_splits, 0.0f, nullptr, stream);
 }

@@ -1,5 +1,7 @@
 // Prefill attention over the paged cache on the 5th-generation tensor cores
-// (bfloat16, head size 64 or 128, causal with an optional window).
+// (bfloat16, key rows of 64 or 128 lanes, value rows of 64 lanes or the keys'
+// size, causal with an optional window that may keep the sequence's first keys
+// visible; a head of another size lies in such rows with zeros behind it).
 //
 // A block owns 128 consecutive new tokens of one sequence and one or two query
 // heads that share a key/value head.  It walks the pages of keys those tokens
@@ -60,6 +62,8 @@ struct AttnParams {
     int n_seqs, n_heads, n_kv;
     float scale2;   // softmax scale times log2(e)
     int window;
+    int keep;       // with a window: the sequence's first keys that stay visible
+    int vo;         // lanes of a head in the output (at most the value rows' VD)
     float slope_base;   // b != 0: head h takes 2^(-b (h + 1) / n_heads) * (query position - key position) off its scaled scores
     const float* sinks; // float32 [n_heads] or null: exp(sinks[h]) joins the denominator of head h's softmax, with no key and no value
     int* status;
@@ -109,26 +113,29 @@ __device__ __forceinline__ void umma_bf16_ts(uint32_t tmem_d, uint32_t tmem_a, u
 }
 
 // Threads: warp 0 producer, warp 1 tensor-core issue and tensor memory, then one warpgroup per head.
-template <int HD, int kStreams>
+template <int HD, int VD, int kStreams>
 __global__ void __launch_bounds__(64 + 128 * kStreams, 1)
 prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                   const __grid_constant__ CUtensorMap map_v, const AttnParams p) {
-    constexpr int kSlabs = HD / 64;                 // 64-element (128-byte) column blocks of a head
+    constexpr int kSlabs = HD / 64, kVSlabs = VD / 64;   // 64-element (128-byte) column blocks of a head
     constexpr int kQBytes = kQRows * HD * 2;        // one head's query tile
     constexpr int kQSlab = kQRows * 128;
-    constexpr int kPageBytes = kPage * HD * 2;      // one page of K or of V for one head
+    constexpr int kPageBytes = kPage * HD * 2;      // one page of K for one head
+    constexpr int kVPageBytes = kPage * VD * 2;     // and of V
     constexpr int kKvSlab = kKeys * 128;            // a stage holds kKeys rows of 128 bytes per column block
-    constexpr int kKvBytes = kSlabs * kKvSlab;      // one stage of K or of V
+    constexpr int kKBytes = kSlabs * kKvSlab;       // one stage of K
+    constexpr int kVBytes = kVSlabs * kKvSlab;      // and of V
     constexpr int kTmemCols = kStreams * kStreamCols;
     static_assert(HD == 64 || HD == 128, "head size 64 or 128");
-    static_assert(kKeys + HD <= kStreamCols, "S (with P over its second half) and O fit a head's columns");
+    static_assert(VD == 64 || VD == HD, "value rows of 64 lanes or the keys' size");
+    static_assert(kKeys + VD <= kStreamCols, "S (with P over its second half) and O fit a head's columns");
 
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     uint8_t* smem_q = smem;                                   // [kStreams][kSlabs][128 rows][128 B]
     uint8_t* smem_k = smem_q + kStreams * kQBytes;            // [kStages][kSlabs][128 keys][128 B]
-    uint8_t* smem_v = smem_k + kStages * kKvBytes;            // the same
-    uint64_t* q_full = (uint64_t*)(smem_v + kStages * kKvBytes);
+    uint8_t* smem_v = smem_k + kStages * kKBytes;             // [kStages][kVSlabs][128 keys][128 B]
+    uint64_t* q_full = (uint64_t*)(smem_v + kStages * kVBytes);
     uint64_t* k_full = q_full + 1;                            // [kStages]
     uint64_t* v_full = k_full + kStages;                      // [kStages]
     uint64_t* k_empty = v_full + kStages;                     // [kStages]
@@ -162,8 +169,8 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
     const int pos0 = p.tok_pos[q0];                  // positions of a sequence's new tokens are consecutive
     const int key_hi = pos0 + n_rows - 1;
     const int key_lo = first_visible_key(pos0, p.window);
-    const int page_lo = key_lo / kPage, page_hi = key_hi / kPage;
-    const int n_pages = page_hi - page_lo + 1;
+    const PageWalk walk(key_lo, key_hi, p.keep);     // the pages that hold keys these rows see
+    const int n_pages = walk.n;
     const int n_steps = (n_pages + 1) / 2;           // two pages a step; the last step may hold one
     // the heads of a key/value head are dealt out two to a block; an odd group's last block has one
     const int group = p.n_heads / p.n_kv;
@@ -220,19 +227,19 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
                     mbar_expect_tx(&k_full[st], pages * kPageBytes);
                     for (int pg = 0; pg < pages; ++pg)
                         for (int s = 0; s < kSlabs; ++s)
-                            tma_load_4d(smem_k + st * kKvBytes + s * kKvSlab + pg * (kPage * 128), &map_k, &k_full[st],
-                                        64 * s, 0, kvh, table[page_lo + 2 * jk + pg]);
+                            tma_load_4d(smem_k + st * kKBytes + s * kKvSlab + pg * (kPage * 128), &map_k, &k_full[st],
+                                        64 * s, 0, kvh, table[walk.page(2 * jk + pg)]);
                     ++jk;
                     moved = true;
                 }
                 if (jv < jk && mbar_test_wait(&v_empty[jv % kStages], ((jv / kStages) & 1) ^ 1)) {
                     const int st = jv % kStages;
                     const int pages = min(2, n_pages - 2 * jv);
-                    mbar_expect_tx(&v_full[st], pages * kPageBytes);
+                    mbar_expect_tx(&v_full[st], pages * kVPageBytes);
                     for (int pg = 0; pg < pages; ++pg)
-                        for (int s = 0; s < kSlabs; ++s)
-                            tma_load_4d(smem_v + st * kKvBytes + s * kKvSlab + pg * (kPage * 128), &map_v, &v_full[st],
-                                        64 * s, 0, kvh, table[page_lo + 2 * jv + pg]);
+                        for (int s = 0; s < kVSlabs; ++s)
+                            tma_load_4d(smem_v + st * kVBytes + s * kKvSlab + pg * (kPage * 128), &map_v, &v_full[st],
+                                        64 * s, 0, kvh, table[walk.page(2 * jv + pg)]);
                     ++jv;
                     moved = true;
                 }
@@ -254,13 +261,13 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
     } else if (warp == 1) {
         if (lane == 0) {
             constexpr uint32_t idesc_s128 = instr_desc_bf16(kQRows, 128), idesc_s64 = instr_desc_bf16(kQRows, 64);
-            constexpr uint32_t idesc_o = instr_desc_bf16(kQRows, HD) | (1u << 16);   // B (V) is MN-major
+            constexpr uint32_t idesc_o = instr_desc_bf16(kQRows, VD) | (1u << 16);   // B (V) is MN-major
             bool ok = mbar_wait(q_full, 0);
             if (!ok) atomicExch(p.status, kTimeoutQ);
             // S_t(i) = Q_t . K(i)^T into the head's S columns; K(i) has landed
             auto issue_scores = [&](int t, int i) {
                 const int keys = min(2, n_pages - 2 * i) * kPage;
-                const uint32_t k_addr = smem_u32(smem_k + (i % kStages) * kKvBytes);
+                const uint32_t k_addr = smem_u32(smem_k + (i % kStages) * kKBytes);
                 const uint32_t q_addr = smem_u32(smem_q + t * kQBytes);
                 const uint32_t tmem_s = tmem_base + (uint32_t)(t * kStreamCols);
                 const uint32_t idesc = keys == 128 ? idesc_s128 : idesc_s64;
@@ -307,7 +314,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
                         }
                     }
                     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                    const uint32_t v_addr = smem_u32(smem_v + st * kKvBytes);
+                    const uint32_t v_addr = smem_u32(smem_v + st * kVBytes);
                     const uint32_t tmem_p = tmem_base + (uint32_t)(t * kStreamCols + kPOffset);
                     const uint32_t tmem_o = tmem_base + (uint32_t)(t * kStreamCols + kKeys);
                     const uint64_t v_desc = smem_desc_sw128_mn(v_addr, kKvSlab);   // 16 keys on: 2048 bytes, 128 in the field
@@ -350,7 +357,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
             }
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             const int halves = min(2, n_pages - 2 * i);
-            const int k_base = (page_lo + 2 * i) * kPage;
+            const int k_base[2] = {walk.page(2 * i) * kPage, walk.page(2 * i + 1) * kPage};
             // A step costs one pass over the row's scores: weights against the reference maximum as it stands (as
             // bfloat16 pairs) and their sum.  The largest score is not looked for: a sum of at most 2^8 proves that
             // no weight is above 2^8.  Only when a row's sum says otherwise (or the row has seen no key yet) is the
@@ -361,18 +368,18 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
             uint32_t w[2][32];   // P of the two pages, stored once the reference maximum is settled: P overwrites S
             auto load_half = [&](int hf, uint32_t (&u)[64]) {
                 tmem_ld64(tmem_row + (uint32_t)(64 * hf), u);
-                const int kb = k_base + 64 * hf;
+                const int kb = k_base[hf];
                 if (bias_per_key != 0.0f) {
                     const float far = (float)(lim_hi - kb);     // the distance of the page's first key
 #pragma unroll
                     for (int c = 0; c < 64; ++c)
                         u[c] = __float_as_uint(fmaf(bias_per_key, (float)c - far, __uint_as_float(u[c])));
                 }
-                if (!(kb >= lim_lo && kb + 63 <= lim_hi)) {
+                if (!((kb >= lim_lo || kb + 63 < p.keep) && kb + 63 <= lim_hi)) {
                     // the page crosses this row's limits
 #pragma unroll
                     for (int c = 0; c < 64; ++c)
-                        if (kb + c < lim_lo || kb + c > lim_hi) u[c] = 0xff800000u;   // -inf
+                        if ((kb + c < lim_lo && kb + c >= p.keep) || kb + c > lim_hi) u[c] = 0xff800000u;   // -inf
                 }
             };
             auto weights = [&]() {
@@ -417,7 +424,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
                 }
                 if (i > 0) {
 #pragma unroll 1
-                    for (int c0 = 0; c0 < HD; c0 += 32) {
+                    for (int c0 = 0; c0 < VD; c0 += 32) {
                         uint32_t o[32];
                         tmem_ld32(tmem_row + (uint32_t)(kKeys + c0), o);
 #pragma unroll
@@ -443,14 +450,19 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
             // the sink's term, in the unit of the row's sums: powers of two relative to the reference maximum
             if (p.sinks != nullptr && l > 0.0f) l += exp2f(p.sinks[h] * 1.4426950408889634f - m_ref);
             const float inv = l > 0.0f ? 1.0f / l : 0.0f;
-            __nv_bfloat16* dst = p.out + (size_t)(q0 + row) * ((size_t)p.n_heads * HD) + (size_t)h * HD;
+            __nv_bfloat16* dst = p.out + ((size_t)(q0 + row) * p.n_heads + h) * p.vo;
 #pragma unroll 1
-            for (int c0 = 0; c0 < HD; c0 += 32) {
+            for (int c0 = 0; c0 < VD; c0 += 32) {
                 uint32_t o[32];
                 tmem_ld32(tmem_row + (uint32_t)(kKeys + c0), o);
-                if (row < n_rows) {
+                if (row < n_rows && (p.vo & 7) != 0) {      // rows of another size: not 16-byte aligned
+#pragma unroll
+                    for (int c = 0; c < 32; ++c)
+                        if (c0 + c < p.vo) dst[c0 + c] = __float2bfloat16_rn(__uint_as_float(o[c]) * inv);
+                } else if (row < n_rows) {
 #pragma unroll
                     for (int c = 0; c < 32; c += 8) {
+                        if (c0 + c >= p.vo) break;
                         uint4 w;
                         w.x = pack_bf16(__uint_as_float(o[c]) * inv, __uint_as_float(o[c + 1]) * inv);
                         w.y = pack_bf16(__uint_as_float(o[c + 2]) * inv, __uint_as_float(o[c + 3]) * inv);
@@ -521,13 +533,13 @@ struct MapCache {
 
 MapCache g_maps;
 
-template <int HD, int kStreams>
+template <int HD, int VD, int kStreams>
 int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const AttnParams& p, int n_tok,
            cudaStream_t stream) {
-    constexpr int smem = kStreams * kQRows * HD * 2 + 2 * kStages * kKeys * HD * 2 + 256 + 1024;
+    constexpr int smem = kStreams * kQRows * HD * 2 + kStages * kKeys * (HD + VD) * 2 + 256 + 1024;
     static bool configured[64] = {};
     if (first_use_on_this_device(configured)) {
-        const cudaError_t e = cudaFuncSetAttribute(prefill_tc_kernel<HD, kStreams>,
+        const cudaError_t e = cudaFuncSetAttribute(prefill_tc_kernel<HD, VD, kStreams>,
                                                    cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         NN_CHECK(e == cudaSuccess, "attention (tensor cores): %d bytes of shared memory refused: %s", smem,
                  cudaGetErrorString(e));
@@ -543,7 +555,7 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, 
     cudaLaunchAttribute attr[1];
     cfg.attrs = attr;
     cfg.numAttrs = overlap_attribute(attr);
-    const cudaError_t e = cudaLaunchKernelEx(&cfg, prefill_tc_kernel<HD, kStreams>, mq, mk, mv, p);
+    const cudaError_t e = cudaLaunchKernelEx(&cfg, prefill_tc_kernel<HD, VD, kStreams>, mq, mk, mv, p);
     NN_CHECK(e == cudaSuccess, "attention prefill (tensor cores): launch failed: %s", cudaGetErrorString(e));
     return 0;
 }
@@ -554,17 +566,20 @@ extern "C" int nncpu_attention_prefill_tc_supported(int n_heads, int n_kv, int h
     return (head_dim == 64 || head_dim == 128) && n_kv > 0 && n_heads > 0 && n_heads % n_kv == 0;
 }
 
-// q and out: bfloat16 [n_tok, n_heads * head_dim]; K and V pages: bfloat16 [n_pages, n_kv, 64, head_dim] holding
-// every key the new tokens may see, their own included; cu_seqlens [n_seqs + 1] row ranges of the sequences;
+// q: bfloat16 [n_tok, n_heads * head_dim], out: bfloat16 [n_tok, n_heads * vo]; K and V pages: bfloat16 [n_pages, n_kv,
+// 64, head_dim] and [n_pages, n_kv, 64, vp] holding every key the new tokens may see, their own included; keep: with a
+// window, the sequence's first keys that stay visible; cu_seqlens [n_seqs + 1] row ranges of the sequences;
 // tok_pos [n_tok] positions (consecutive within a sequence).  *status receives a code if a wait runs out.
 extern "C" int nncpu_attention_prefill_tc(const void* q, const void* k_pages, const void* v_pages, int n_pages,
                                           const int* block_table, int bt_stride, const int* cu_seqlens,
                                           const int* tok_pos, void* out, int n_tok, int n_seqs, int n_heads, int n_kv,
-                                          int head_dim, float scale, int window, float slope_base, const float* sinks,
-                                          int* status, void* stream_) {
+                                          int head_dim, int vp, int vo, float scale, int window, int keep,
+                                          float slope_base, const float* sinks, int* status, void* stream_) {
     NN_CHECK(nncpu_attention_prefill_tc_supported(n_heads, n_kv, head_dim),
              "attention (tensor cores): head size %d with %d heads over %d key/value heads is not supported "
              "(head size 64 or 128, heads a multiple of key/value heads)", head_dim, n_heads, n_kv);
+    NN_CHECK((vp == head_dim || vp == 64) && vo > 0 && vo <= vp && keep >= 0,
+             "attention (tensor cores): value rows of %d lanes, %d of them used", vp, vo);
     NN_CHECK(n_tok >= 0 && n_seqs >= 0 && n_pages > 0, "attention (tensor cores): %d tokens of %d sequences, %d pages",
              n_tok, n_seqs, n_pages);
     NN_CHECK(((uintptr_t)q % 16) == 0 && ((uintptr_t)k_pages % 16) == 0 && ((uintptr_t)v_pages % 16) == 0 &&
@@ -574,7 +589,7 @@ extern "C" int nncpu_attention_prefill_tc(const void* q, const void* k_pages, co
     CUtensorMap mq, mk, mv;
     if (int e = g_maps.get(&mq, q, n_tok, (long)n_heads * head_dim, 0, 0)) return e;
     if (int e = g_maps.get(&mk, k_pages, n_pages, n_kv, head_dim, 1)) return e;
-    if (int e = g_maps.get(&mv, v_pages, n_pages, n_kv, head_dim, 1)) return e;
+    if (int e = g_maps.get(&mv, v_pages, n_pages, n_kv, vp, 1)) return e;
     AttnParams p;
     p.block_table = block_table;
     p.bt_stride = bt_stride;
@@ -586,12 +601,15 @@ extern "C" int nncpu_attention_prefill_tc(const void* q, const void* k_pages, co
     p.n_kv = n_kv;
     p.scale2 = scale * 1.4426950408889634f;
     p.window = window;
+    p.keep = keep;
+    p.vo = vo;
     p.slope_base = slope_base;
     p.sinks = sinks;
     p.status = status;
     cudaStream_t stream = (cudaStream_t)stream_;
     // two heads to a block where a key/value head has two to give; one head per block otherwise
-    if (n_heads == n_kv)
-        return head_dim == 64 ? launch<64, 1>(mq, mk, mv, p, n_tok, stream) : launch<128, 1>(mq, mk, mv, p, n_tok, stream);
-    return head_dim == 64 ? launch<64, 2>(mq, mk, mv, p, n_tok, stream) : launch<128, 2>(mq, mk, mv, p, n_tok, stream);
+    const bool one = n_heads == n_kv;
+    if (head_dim == 64) return one ? launch<64, 64, 1>(mq, mk, mv, p, n_tok, stream) : launch<64, 64, 2>(mq, mk, mv, p, n_tok, stream);
+    if (vp == 64) return one ? launch<128, 64, 1>(mq, mk, mv, p, n_tok, stream) : launch<128, 64, 2>(mq, mk, mv, p, n_tok, stream);
+    return one ? launch<128, 128, 1>(mq, mk, mv, p, n_tok, stream) : launch<128, 128, 2>(mq, mk, mv, p, n_tok, stream);
 }

@@ -178,6 +178,19 @@ __device__ __forceinline__ int first_visible_key(int pos, int span) {
     return 0;
 }
 
+// The pages that hold the keys which queries with first visible key `lo` and last key `hi` see, in order: those of the
+// sequence's first `keep` keys that lie before the window's, then the window's own.  Which keys of a page a query
+// sees is a matter of masks: (key >= its first visible key || key < keep) && key <= its position.
+struct PageWalk {
+    int n_kept, lo, n;
+    __device__ __forceinline__ PageWalk(int key_lo, int key_hi, int keep) {
+        lo = key_lo / kPage;
+        n_kept = keep > 0 ? min((keep + kPage - 1) / kPage, lo) : 0;
+        n = n_kept + key_hi / kPage - lo + 1;
+    }
+    __device__ __forceinline__ int page(int i) const { return i < n_kept ? i : lo + i - n_kept; }
+};
+
 // Gated activations act(gate) * up of the feed-forwards, on 32-bit values.  kGateSilu: silu(g) u.  kGateGeluTanh: the
 // tanh form of GELU, g/2 (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))) u.  kGateSwishClamp: with g' = min(g, limit) and
 // u' = clamp(u, -limit, limit): g' sigmoid(1.702 g') (u' + 1).

@@ -550,13 +550,104 @@ extern "C" int nncpu_qk_norm_rope_append(const void* qkv, int in_dt, const void*
 }
 
 // ---------------------------------------------------------------------------
+// The same step for mixers whose query and key norm runs over ALL of a token's query (key) lanes at once, before they are
+// split into heads, and / or that rotate neighbouring lanes (2 i, 2 i + 1): qkv float32 [n_tok, ld] holds the heads of q
+// (hd lanes each), of k (hd) and of v (vd).  A head lies in q_out and in the pages in rows of qp (queries, keys) and
+// vp (values) lanes, zeros behind its own.  One block per token: the row's two sums of squares first, then its items of
+// four lanes.  norm: 0 none, 1 over the whole row (weights [n_heads hd] and [n_kv hd]).  The first `half` pairs of a head
+// turn.
+// ---------------------------------------------------------------------------
+__global__ void __launch_bounds__(256)
+qk_whole_norm_append_kernel(const float* __restrict__ qkv, int ld, const void* __restrict__ q_gamma,
+                            const void* __restrict__ k_gamma, int g_dt, float eps, const float2* __restrict__ cs, int half,
+                            const int* __restrict__ tok_seq, const int* __restrict__ tok_pos,
+                            const int* __restrict__ block_table, int bt_stride, void* __restrict__ k_pages,
+                            void* __restrict__ v_pages, int kv_dt, void* __restrict__ q_out, int q_dt, int n_heads, int n_kv,
+                            int hd, int vd, int qp, int vp) {
+    __shared__ float scratch[33];
+    const int t = blockIdx.x, tid = threadIdx.x;
+    const float* row = qkv + (size_t)t * ld;
+    const int nq = n_heads * hd, nk = n_kv * hd;
+    float q_scale = 1.0f, k_scale = 1.0f;
+    if (q_gamma != nullptr) {
+        float ss = 0.0f;
+        for (int i = tid; i < nq; i += 256) ss = fmaf(row[i], row[i], ss);
+        q_scale = 1.0f / sqrtf(block_sum(ss, scratch) * (1.0f / (float)nq) + eps);
+    }
+    if (k_gamma != nullptr && n_kv > 0) {
+        float ss = 0.0f;
+        for (int i = tid; i < nk; i += 256) ss = fmaf(row[nq + i], row[nq + i], ss);
+        k_scale = 1.0f / sqrtf(block_sum(ss, scratch) * (1.0f / (float)nk) + eps);
+    }
+    const int seq = tok_seq[t], pos = tok_pos[t];
+    const int page = (seq >= 0 && n_kv > 0) ? block_table[(size_t)seq * bt_stride + pos / kPage] : -1;
+    // items of two neighbouring lanes of a head's row: queries, then (if this token has a place in the cache) keys, values
+    const int pq = (qp + 1) >> 1, pv = (vp + 1) >> 1;
+    const int items_q = n_heads * pq, items_k = page >= 0 ? n_kv * pq : 0, items_v = page >= 0 ? n_kv * pv : 0;
+    for (int it = tid; it < items_q + items_k + items_v; it += 256) {
+        if (it >= items_q + items_k) {
+            const int j = it - items_q - items_k, h = j / pv, d = (j % pv) * 2;
+            const float* src = row + nq + nk + (size_t)h * vd;
+            const size_t at = (((size_t)page * n_kv + h) * kPage + pos % kPage) * vp + d;
+            st_f(v_pages, at, kv_dt, d < vd ? src[d] : 0.0f);
+            if (d + 1 < vp) st_f(v_pages, at + 1, kv_dt, d + 1 < vd ? src[d + 1] : 0.0f);
+            continue;
+        }
+        const bool is_q = it < items_q;
+        const int j = is_q ? it : it - items_q, h = j / pq, d = (j % pq) * 2;
+        const int lane0 = h * hd + d;                              // its place among the query (key) lanes
+        const float* src = row + (is_q ? 0 : nq) + lane0;
+        const void* gamma = is_q ? q_gamma : k_gamma;
+        const float scale = is_q ? q_scale : k_scale;
+        float u = d < hd ? src[0] : 0.0f, v = d + 1 < hd ? src[1] : 0.0f;
+        if (gamma != nullptr) {
+            u = d < hd ? (u * scale) * ld_f(gamma, lane0, g_dt) : 0.0f;
+            v = d + 1 < hd ? (v * scale) * ld_f(gamma, lane0 + 1, g_dt) : 0.0f;
+        }
+        if (cs != nullptr && (d >> 1) < half) {
+            const float2 c = cs[(size_t)t * half + (d >> 1)];
+            const float a = u;
+            u = c.x * a - c.y * v;
+            v = c.y * a + c.x * v;
+        }
+        void* dst = is_q ? q_out : k_pages;
+        const int dt = is_q ? q_dt : kv_dt;
+        const size_t at = is_q ? ((size_t)t * n_heads + h) * qp + d : (((size_t)page * n_kv + h) * kPage + pos % kPage) * qp + d;
+        if (dt == DT_BF16 && (qp & 1) == 0) {
+            *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<__nv_bfloat16*>(dst) + at) = __floats2bfloat162_rn(u, v);
+        } else {
+            st_f(dst, at, dt, u);
+            if (d + 1 < qp) st_f(dst, at + 1, dt, v);
+        }
+    }
+}
+
+extern "C" int nncpu_qk_whole_norm_append(const float* qkv, int ld, const void* q_gamma, const void* k_gamma, int g_dt,
+                                          float eps, const float* cs, int half, const int* tok_seq, const int* tok_pos,
+                                          const int* block_table, int bt_stride, void* k_pages, void* v_pages, int kv_dt,
+                                          void* q_out, int q_dt, int n_tok, int n_heads, int n_kv, int hd, int vd, int qp,
+                                          int vp, void* stream) {
+    NN_CHECK(n_tok >= 0 && n_heads > 0 && n_kv >= 0 && hd > 0 && vd > 0 && qp >= hd && vp >= vd,
+             "q/k norm and append: %d and %d heads of %d and %d lanes in rows of %d and %d", n_heads, n_kv, hd, vd, qp, vp);
+    NN_CHECK(ld >= (n_heads + n_kv) * hd + n_kv * vd, "q/k norm and append: rows of %d elements", ld);
+    NN_CHECK(cs == nullptr || 2 * half <= hd, "q/k norm and append: %d rotated pairs of a head of %d lanes", half, hd);
+    NN_CHECK((uintptr_t)cs % 8 == 0, "q/k norm and append: the rotation table must be 8-byte aligned (cos/sin pairs)");
+    if (n_tok == 0) return 0;
+    qk_whole_norm_append_kernel<<<n_tok, 256, 0, (cudaStream_t)stream>>>(
+        qkv, ld, q_gamma, k_gamma, g_dt, eps, (const float2*)cs, half, tok_seq, tok_pos, block_table, bt_stride, k_pages,
+        v_pages, kv_dt, q_out, q_dt, n_heads, n_kv, hd, vd, qp, vp);
+    NN_LAUNCH_OK("q/k norm and append");
+    return 0;
+}
+
+// ---------------------------------------------------------------------------
 // Attention of every (token, head) over the cache of the token's sequence:
 // keys first..pos with first = first_visible_key(pos, window): a sliding window (window > 0), blocks of
-// -window positions (window < 0) or every earlier key (0).
+// -window positions (window < 0) or every earlier key (0); with a window the sequence's first `keep` keys too.
 // One block per (token, head) walks the span in chunks of 128 keys with an
 // online softmax; the chunk boundaries are fixed by the span alone, so the
 // result does not depend on the batch or on how tokens were cut into steps.
-// Values have vd lanes a head (the output too).  With slope_base != 0 head h
+// Values have vd lanes a head in their pages and vo (at most vd) in the output.  With slope_base != 0 head h
 // takes slope_h * (pos - key) off its scaled scores, slope_h = 2^(-slope_base (h + 1) / n_heads).
 // With sinks (float32 [n_heads]) the softmax's denominator of head h also holds exp(sinks[h]): a term without
 // key or value, not scaled, counted once.
@@ -567,8 +658,8 @@ __global__ void __launch_bounds__(kAttnThreads)
 attention_kernel(const void* __restrict__ q, int q_dt, const void* __restrict__ k_pages,
                  const void* __restrict__ v_pages, int kv_dt, const int* __restrict__ block_table, int bt_stride,
                  const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, void* __restrict__ out,
-                 int out_dt, int n_heads, int n_kv, int hd, int vd, float scale, int window, float slope_base,
-                 const float* __restrict__ sinks) {
+                 int out_dt, int n_heads, int n_kv, int hd, int vd, int vo, float scale, int window, int keep,
+                 float slope_base, const float* __restrict__ sinks) {
     extern __shared__ float smem[];
     float* qs = smem;                       // hd
     float* p = smem + hd;                   // kAttnThreads
@@ -578,14 +669,16 @@ attention_kernel(const void* __restrict__ q, int q_dt, const void* __restrict__ 
     const int t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
     const int seq = tok_seq[t];
     const size_t q_base = (size_t)t * n_heads * hd + (size_t)h * hd;
-    const size_t out_base = (size_t)t * n_heads * vd + (size_t)h * vd;
+    const size_t out_base = ((size_t)t * n_heads + h) * vo;
     if (seq < 0) {
-        for (int d = tid; d < vd; d += kAttnThreads) st_f(out, out_base + d, out_dt, 0.0f);
+        for (int d = tid; d < vo; d += kAttnThreads) st_f(out, out_base + d, out_dt, 0.0f);
         return;
     }
     const float slope = slope_base != 0.0f ? exp2f(-slope_base * (float)(h + 1) / (float)n_heads) : 0.0f;
     const int pos = tok_pos[t];
     const int first = first_visible_key(pos, window);
+    // the visible keys in order: those of the first `keep` that lie before the window's, then first .. pos
+    const int n_kept = min(keep, first), n_visible = n_kept + pos - first + 1;
     const int kvh = h / (n_heads / n_kv);
     for (int d = tid; d < hd; d += kAttnThreads) qs[d] = ld_f(q, q_base + d, q_dt);
     __syncthreads();
@@ -595,11 +688,12 @@ attention_kernel(const void* __restrict__ q, int q_dt, const void* __restrict__ 
 #pragma unroll
     for (int j = 0; j < 8; ++j) acc[j] = 0.0f;
 
-    for (int k0 = first; k0 <= pos; k0 += kAttnThreads) {
-        const int key = k0 + tid;
+    for (int k0 = 0; k0 < n_visible; k0 += kAttnThreads) {
+        const bool has_key = k0 + tid < n_visible;
+        const int key = k0 + tid < n_kept ? k0 + tid : first + k0 + tid - n_kept;
         float s = -INFINITY;
         long long off = -1;
-        if (key <= pos) {
+        if (has_key) {
             const int page = block_table[(size_t)seq * bt_stride + key / kPage];
             off = ((long long)page * n_kv + kvh) * kPage + key % kPage;      // the key's row in its pages
             float dot = 0.0f;
@@ -607,14 +701,14 @@ attention_kernel(const void* __restrict__ q, int q_dt, const void* __restrict__ 
             s = dot * scale - slope * (float)(pos - key);
         }
         const float m_new = fmaxf(m, block_max(s, scratch));
-        const float w = key <= pos ? expf(s - m_new) : 0.0f;
+        const float w = has_key ? expf(s - m_new) : 0.0f;
         const float corr = expf(m - m_new);  // 0 on the first chunk
         l = l * corr + block_sum(w, scratch);
         m = m_new;
         p[tid] = w;
         row[tid] = off;
         __syncthreads();
-        const int n_keys = min(kAttnThreads, pos + 1 - k0);
+        const int n_keys = min(kAttnThreads, n_visible - k0);
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
             const int d = tid + kAttnThreads * j;
@@ -631,25 +725,26 @@ attention_kernel(const void* __restrict__ q, int q_dt, const void* __restrict__ 
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
         const int d = tid + kAttnThreads * j;
-        if (d < vd) st_f(out, out_base + d, out_dt, acc[j] * inv);
+        if (d < vo) st_f(out, out_base + d, out_dt, acc[j] * inv);
     }
 }
 
 extern "C" int nncpu_attention(const void* q, int q_dt, const void* k_pages, const void* v_pages, int kv_dt,
                                const int* block_table, int bt_stride, const int* tok_seq, const int* tok_pos,
-                               void* out, int out_dt, int n_tok, int n_heads, int n_kv, int hd, int vd, float scale,
-                               int window, float slope_base, const float* sinks, void* stream) {
+                               void* out, int out_dt, int n_tok, int n_heads, int n_kv, int hd, int vd, int vo, float scale,
+                               int window, int keep, float slope_base, const float* sinks, void* stream) {
     NN_CHECK(n_tok >= 0 && n_heads > 0 && n_kv > 0 && n_heads % n_kv == 0,
              "attention: %d heads over %d key/value heads", n_heads, n_kv);
     NN_CHECK(hd > 0 && hd <= 1024, "attention: head size %d must be positive and at most 1024", hd);
     NN_CHECK(vd > 0 && vd <= 1024, "attention: value size %d must be positive and at most 1024", vd);
+    NN_CHECK(vo > 0 && vo <= vd && keep >= 0, "attention: %d lanes of values of %d, %d kept keys", vo, vd, keep);
     if (n_tok == 0) return 0;
     const size_t smem = (hd + kAttnThreads) * sizeof(float) + kAttnThreads * sizeof(long long) + 8;
     dim3 grid(n_tok, n_heads);
     attention_kernel<<<grid, kAttnThreads, smem, (cudaStream_t)stream>>>(q, q_dt, k_pages, v_pages, kv_dt,
                                                                          block_table, bt_stride, tok_seq, tok_pos,
-                                                                         out, out_dt, n_heads, n_kv, hd, vd, scale,
-                                                                         window, slope_base, sinks);
+                                                                         out, out_dt, n_heads, n_kv, hd, vd, vo, scale,
+                                                                         window, keep, slope_base, sinks);
     NN_LAUNCH_OK("attention");
     return 0;
 }
@@ -1994,21 +2089,57 @@ __device__ __forceinline__ void route_top_all(float* z, float* gbuf, int n_exper
     for (int c = lane; c < top; c += 32) weights[c] *= inv;
 }
 
+// Scores by the sigmoid: the `top` largest logits, weighted by their sigmoids as they are.  One warp; z is overwritten.
+__device__ __forceinline__ void route_top_sigmoid(float* z, int n_experts, int top, int* __restrict__ ids,
+                                                  float* __restrict__ weights, int lane) {
+    for (int c = 0; c < top; ++c) {
+        float best = -INFINITY;
+        int at = n_experts;
+        for (int e = lane; e < n_experts; e += 32) {
+            const float v = z[e];
+            if (v > best || (v == best && e < at)) { best = v; at = e; }
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+            const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+            if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
+        }
+        if (at >= n_experts) at = 0;
+        if (lane == 0) {
+            ids[c] = at;
+            weights[c] = 1.0f / (1.0f + expf(0.0f - best));
+            z[at] = __int_as_float(0x7FC00000);
+        }
+        __syncwarp();
+    }
+}
+
+constexpr int kScoresChosen = 0, kScoresAll = 1, kScoresSigmoid = 2;
+
+__device__ __forceinline__ void route_one(float* z, float* gbuf, int n_experts, int top, int scores, int n_groups, int keep,
+                                          float scale, int* __restrict__ ids, float* __restrict__ weights, int lane) {
+    if (scores == kScoresAll) route_top_all(z, gbuf, n_experts, top, n_groups, keep, scale, ids, weights, lane);
+    else if (scores == kScoresSigmoid) route_top_sigmoid(z, n_experts, top, ids, weights, lane);
+    else route_top(z, n_experts, top, ids, weights, lane);
+}
+
+// With `gate` (float [n_tok]) one more logit follows the experts' in a row: its sigmoid is the token's gate of a shared
+// feed-forward.
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const float* __restrict__ logits, int n_tok, int n_experts, int top, int* __restrict__ ids,
-                 float* __restrict__ weights, int all_scores, int n_groups, int keep, float scale) {
+                 float* __restrict__ weights, int all_scores, int n_groups, int keep, float scale, int ld,
+                 float* __restrict__ gate) {
     extern __shared__ float smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x * (blockDim.x >> 5) + warp;
     if (t >= n_tok) return;
     float* z = smem + (size_t)warp * (n_experts + n_groups);
-    for (int e = lane; e < n_experts; e += 32) z[e] = logits[(size_t)t * n_experts + e];
+    for (int e = lane; e < n_experts; e += 32) z[e] = logits[(size_t)t * ld + e];
+    if (gate != nullptr && lane == 0) gate[t] = 1.0f / (1.0f + expf(0.0f - logits[(size_t)t * ld + n_experts]));
     __syncwarp();
-    if (all_scores)
-        route_top_all(z, z + n_experts, n_experts, top, n_groups, keep, scale, ids + (size_t)t * top,
-                      weights + (size_t)t * top, lane);
-    else
-        route_top(z, n_experts, top, ids + (size_t)t * top, weights + (size_t)t * top, lane);
+    route_one(z, z + n_experts, n_experts, top, all_scores, n_groups, keep, scale, ids + (size_t)t * top,
+              weights + (size_t)t * top, lane);
 }
 
 // Whether a choice among groups can be made: equal groups, and the kept ones hold enough experts.
@@ -2018,16 +2149,19 @@ static bool route_groups_ok(int n_experts, int top, int n_groups, int keep) {
 }
 
 extern "C" int nncpu_moe_route(const float* logits, int n_tok, int n_experts, int top, int* ids, float* weights,
-                               int all_scores, int n_groups, int keep, float scale, void* stream) {
+                               int all_scores, int n_groups, int keep, float scale, int ld, float* gate, void* stream) {
+    // all_scores: 0 the softmax over the chosen logits, 1 over all (with groups and a scale), 2 sigmoids; ld: floats a row
+    // of logits (with `gate`, the gate's logit follows the experts')
     NN_CHECK(n_tok >= 0 && n_experts > 0 && n_experts <= kRouteMaxExperts && top > 0 && top <= n_experts,
              "router: %d tokens, the top %d of %d experts (at most %d)", n_tok, top, n_experts, kRouteMaxExperts);
-    NN_CHECK(all_scores ? route_groups_ok(n_experts, top, n_groups, keep) : n_groups <= 1,
+    NN_CHECK(all_scores == kScoresAll ? route_groups_ok(n_experts, top, n_groups, keep) : n_groups <= 1,
              "router: the %d best of %d groups of %d experts for the top %d", keep, n_groups, n_experts, top);
+    NN_CHECK(ld >= n_experts + (gate != nullptr ? 1 : 0), "router: rows of %d logits for %d experts", ld, n_experts);
     if (n_tok == 0) return 0;
     if (n_groups < 1) n_groups = 1;
     const size_t smem = (size_t)4 * (n_experts + n_groups) * sizeof(float);
     moe_route_kernel<<<(n_tok + 3) / 4, 128, smem, (cudaStream_t)stream>>>(logits, n_tok, n_experts, top, ids, weights,
-                                                                          all_scores, n_groups, keep, scale);
+                                                                          all_scores, n_groups, keep, scale, ld, gate);
     NN_LAUNCH_OK("router");
     return 0;
 }
@@ -2068,7 +2202,8 @@ __device__ __forceinline__ float warp_dot(const void* __restrict__ w, size_t row
 __global__ void __launch_bounds__(256)
 moe_router_kernel(const void* __restrict__ x, int x_dt, const void* __restrict__ w, int w_dt, const void* __restrict__ bias,
                   int b_dt, int n_tok, int per_block, int n_experts, int top, int width, int* __restrict__ ids,
-                  float* __restrict__ weights, int all_scores, int n_groups, int keep, float scale) {
+                  float* __restrict__ weights, int all_scores, int n_groups, int keep, float scale,
+                  float* __restrict__ gate) {
     extern __shared__ float smem[];          // a token's input, then its logits
     float* z = smem + width;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
@@ -2076,18 +2211,15 @@ moe_router_kernel(const void* __restrict__ x, int x_dt, const void* __restrict__
     for (int t = blockIdx.x * per_block; t < min(n_tok, (int)(blockIdx.x + 1) * per_block); ++t) {
         for (int i = threadIdx.x; i < width; i += blockDim.x) smem[i] = ld_f(x, (size_t)t * width + i, x_dt);
         __syncthreads();
-        for (int e = warp; e < n_experts; e += n_warps) {
+        for (int e = warp; e < n_experts + (gate != nullptr ? 1 : 0); e += n_warps) {
             const float d = warp_dot(w, (size_t)e * width, w_dt, smem, width, lane);
-            if (lane == 0) z[e] = d + (bias ? ld_f(bias, e, b_dt) : 0.0f);
+            if (lane == 0 && e == n_experts) gate[t] = 1.0f / (1.0f + expf(0.0f - d));     // the last row is the gate's
+            else if (lane == 0) z[e] = d + (bias ? ld_f(bias, e, b_dt) : 0.0f);
         }
         __syncthreads();
-        if (warp == 0) {
-            if (all_scores)
-                route_top_all(z, z + n_experts, n_experts, top, n_groups, keep, scale, ids + (size_t)t * top,
-                              weights + (size_t)t * top, lane);
-            else
-                route_top(z, n_experts, top, ids + (size_t)t * top, weights + (size_t)t * top, lane);
-        }
+        if (warp == 0)
+            route_one(z, z + n_experts, n_experts, top, all_scores, n_groups, keep, scale, ids + (size_t)t * top,
+                      weights + (size_t)t * top, lane);
         __syncthreads();
     }
 }
@@ -2098,10 +2230,11 @@ extern "C" int nncpu_moe_router_fits(int n_experts, int width) {
 
 extern "C" int nncpu_moe_router(const void* x, int x_dt, const void* w, int w_dt, const void* bias, int b_dt, int n_tok,
                                 int n_experts, int top, int width, int* ids, float* weights, int all_scores, int n_groups,
-                                int keep, float scale, void* stream) {
+                                int keep, float scale, float* gate, void* stream) {
+    // gate (optional, float [n_tok]): w has one row more, whose product's sigmoid is left there
     NN_CHECK(n_tok >= 0 && width > 0 && top > 0 && top <= n_experts && nncpu_moe_router_fits(n_experts, width),
              "router: %d tokens of %d, the top %d of %d experts", n_tok, width, top, n_experts);
-    NN_CHECK(all_scores ? route_groups_ok(n_experts, top, n_groups, keep) : n_groups <= 1,
+    NN_CHECK(all_scores == kScoresAll ? route_groups_ok(n_experts, top, n_groups, keep) : n_groups <= 1,
              "router: the %d best of %d groups of %d experts for the top %d", keep, n_groups, n_experts, top);
     if (n_tok == 0) return 0;
     if (n_groups < 1) n_groups = 1;
@@ -2109,7 +2242,7 @@ extern "C" int nncpu_moe_router(const void* x, int x_dt, const void* w, int w_dt
     // (2 048 tokens of 4 096 lanes, 16 experts: 88 us a launch with one token a block, 124 us with eight).
     const int per_block = 1;
     moe_router_kernel<<<(n_tok + per_block - 1) / per_block, 256, (size_t)(width + n_experts + n_groups) * 4, (cudaStream_t)stream>>>(
-        x, x_dt, w, w_dt, bias, b_dt, n_tok, per_block, n_experts, top, width, ids, weights, all_scores, n_groups, keep, scale);
+        x, x_dt, w, w_dt, bias, b_dt, n_tok, per_block, n_experts, top, width, ids, weights, all_scores, n_groups, keep, scale, gate);
     NN_LAUNCH_OK("router");
     return 0;
 }
@@ -2119,14 +2252,20 @@ constexpr int kMoeWarps = 8;
 __global__ void __launch_bounds__(kMoeWarps * 32)
 moe_gate_up_kernel(const void* __restrict__ x, int x_dt, const void* __restrict__ wg, const void* __restrict__ wu,
                    int w_dt, const int* __restrict__ ids, void* __restrict__ act, int act_dt, int top, int width, int ff,
-                   int n_experts, int kind, float limit) {
+                   int n_experts, int kind, float limit, const float* __restrict__ in_weights, int n_slots,
+                   const void* __restrict__ sh_g, const void* __restrict__ sh_u, int sh_ff, void* __restrict__ sh_act) {
+    // in_weights (optional, [n_slots]): a slot's weight multiplies its expert's input.  sh_act (optional): the blocks
+    // beyond the slots are the shared feed-forward's, one per token, with matrices of sh_ff rows in either layout.
     // wu null: wg holds [n_experts, 2 ff, width] with an expert's gate and up rows interleaved in blocks of 8 (the
     // layout of the tensor-core products' gated epilogue): gate row j is row 16 (j / 8) + j % 8, up row j eight below
     extern __shared__ float smem[];          // the token's input as floats
-    const int s = blockIdx.x, t = s / top;
+    const bool shared = (int)blockIdx.x >= n_slots;
+    const int s = shared ? (int)blockIdx.x - n_slots : (int)blockIdx.x, t = shared ? s : s / top;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int e = ids[s];
-    for (int i = threadIdx.x; i < width; i += blockDim.x) smem[i] = ld_f(x, (size_t)t * width + i, x_dt);
+    const int e = shared ? 0 : ids[s];
+    const float in_w = (!shared && in_weights != nullptr) ? in_weights[s] : 1.0f;
+    if (shared) { wg = sh_g; wu = sh_u; ff = sh_ff; act = sh_act; n_experts = 1; }
+    for (int i = threadIdx.x; i < width; i += blockDim.x) smem[i] = ld_f(x, (size_t)t * width + i, x_dt) * in_w;
     __syncthreads();
     if (e < 0 || e >= n_experts) return;
     const bool mixed = wu == nullptr;
@@ -2143,9 +2282,14 @@ moe_gate_up_kernel(const void* __restrict__ x, int x_dt, const void* __restrict_
 __global__ void __launch_bounds__(kMoeWarps * 32)
 moe_down_kernel(const void* __restrict__ act, int act_dt, const void* __restrict__ wd, int w_dt,
                 const int* __restrict__ ids, const float* __restrict__ weights, float* __restrict__ out, int top,
-                int width, int ff, int n_experts) {
-    extern __shared__ float smem[];          // the token's top * ff activations as floats
+                int width, int ff, int n_experts, const void* __restrict__ sh_act, const void* __restrict__ sh_wd, int sh_ff,
+                const float* __restrict__ sh_gate) {
+    // weights null: ones.  sh_act (optional) [n_tok, sh_ff]: the shared feed-forward's part, times the token's gate.
+    extern __shared__ float smem[];          // the token's top * ff activations as floats, then the shared ones
     const int t = blockIdx.x;
+    float* sh_smem = smem + (size_t)top * ff;
+    if (sh_act != nullptr)
+        for (int i = threadIdx.x; i < sh_ff; i += blockDim.x) sh_smem[i] = ld_f(sh_act, (size_t)t * sh_ff + i, act_dt);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     for (int i = threadIdx.x; i < top * ff; i += blockDim.x) smem[i] = ld_f(act, (size_t)t * top * ff + i, act_dt);
     __syncthreads();
@@ -2155,21 +2299,31 @@ moe_down_kernel(const void* __restrict__ act, int act_dt, const void* __restrict
             const int e = ids[(size_t)t * top + c];
             if (e < 0 || e >= n_experts) continue;
             const float d = warp_dot(wd, ((size_t)e * width + i) * ff, w_dt, smem + (size_t)c * ff, ff, lane);
-            sum = fmaf(weights[(size_t)t * top + c], d, sum);
+            sum = weights != nullptr ? fmaf(weights[(size_t)t * top + c], d, sum) : sum + d;
         }
+        if (sh_act != nullptr) sum = fmaf(sh_gate[t], warp_dot(sh_wd, (size_t)i * sh_ff, w_dt, sh_smem, sh_ff, lane), sum);
         if (lane == 0) out[(size_t)t * width + i] += sum;
     }
 }
 
 extern "C" int nncpu_moe_experts(const void* x, int x_dt, const void* wg, const void* wu, const void* wd, int w_dt,
                                  const int* ids, const float* weights, void* act, int act_dt, float* out, int n_tok,
-                                 int top, int width, int ff, int n_experts, int kind, float limit, void* stream) {
+                                 int top, int width, int ff, int n_experts, int kind, float limit, int weight_on_input,
+                                 const void* sh_g, const void* sh_u, const void* sh_wd, int sh_ff, void* sh_act,
+                                 const float* sh_gate, void* stream) {
+    // weight_on_input: the weights multiply the experts' inputs instead of their outputs.  sh_wd (optional): a shared
+    // feed-forward in the same launches (its gate/up rows interleaved like the experts' when sh_u is null), its output
+    // times sh_gate [n_tok]; sh_act [n_tok, sh_ff] is scratch.
     NN_CHECK(n_tok >= 0 && top > 0 && width > 0 && ff > 0 && n_experts > 0, "experts: %d tokens, top %d, %d x %d, %d experts",
              n_tok, top, width, ff, n_experts);
     NN_CHECK(kind >= kGateSilu && kind <= kGateSwishClamp, "experts: activation kind %d", kind);
     NN_CHECK(wu != nullptr || ff % 8 == 0, "experts: interleaved gate and up rows need a multiple of 8 of them (%d)", ff);
     constexpr size_t kMost = 200 * 1024;
-    NN_CHECK((size_t)width * 4 <= kMost && (size_t)top * ff * 4 <= kMost,
+    const bool with_shared = sh_wd != nullptr;
+    NN_CHECK(!with_shared || (sh_g != nullptr && sh_act != nullptr && sh_gate != nullptr && sh_ff > 0 && (sh_u != nullptr || sh_ff % 8 == 0)),
+             "experts: a shared feed-forward of %d rows", sh_ff);
+    if (!with_shared) { sh_ff = 0; sh_act = nullptr; }
+    NN_CHECK((size_t)width * 4 <= kMost && ((size_t)top * ff + sh_ff) * 4 <= kMost,
              "experts: a token's %d inputs or %d x %d activations do not fit the shared memory of this kernel", width, top, ff);
     if (n_tok == 0) return 0;
     static bool configured[64] = {};
@@ -2181,13 +2335,16 @@ extern "C" int nncpu_moe_experts(const void* x, int x_dt, const void* wg, const 
     const long slots = (long)n_tok * top;
     NN_CHECK(slots < (1l << 31), "experts: %ld token slots", slots);
     // few tokens: more blocks per token, so that the weights' stream is spread over the SMs
-    const int split_up = (int)max(1l, min((long)(ff + kMoeWarps - 1) / kMoeWarps, 1024 / max(1l, slots)));
+    const long blocks = slots + (with_shared ? n_tok : 0);
+    const int split_up = (int)max(1l, min((long)(max(ff, sh_ff) + kMoeWarps - 1) / kMoeWarps, 1024 / max(1l, blocks)));
     const int split_down = (int)max(1l, min((long)(width + kMoeWarps - 1) / kMoeWarps, 1024 / max(1l, (long)n_tok)));
-    moe_gate_up_kernel<<<dim3((unsigned)slots, split_up), kMoeWarps * 32, (size_t)width * 4, (cudaStream_t)stream>>>(
-        x, x_dt, wg, wu, w_dt, ids, act, act_dt, top, width, ff, n_experts, kind, limit);
+    moe_gate_up_kernel<<<dim3((unsigned)blocks, split_up), kMoeWarps * 32, (size_t)width * 4, (cudaStream_t)stream>>>(
+        x, x_dt, wg, wu, w_dt, ids, act, act_dt, top, width, ff, n_experts, kind, limit, weight_on_input ? weights : nullptr,
+        (int)slots, sh_g, sh_u, sh_ff, sh_act);
     NN_LAUNCH_OK("experts (gate and up)");
-    moe_down_kernel<<<dim3(n_tok, split_down), kMoeWarps * 32, (size_t)top * ff * 4, (cudaStream_t)stream>>>(
-        act, act_dt, wd, w_dt, ids, weights, out, top, width, ff, n_experts);
+    moe_down_kernel<<<dim3(n_tok, split_down), kMoeWarps * 32, ((size_t)top * ff + sh_ff) * 4, (cudaStream_t)stream>>>(
+        act, act_dt, wd, w_dt, ids, weight_on_input ? nullptr : weights, out, top, width, ff, n_experts, sh_act, sh_wd, sh_ff,
+        sh_gate);
     NN_LAUNCH_OK("experts (down)");
     return 0;
 }
@@ -2198,8 +2355,10 @@ extern "C" int nncpu_moe_experts(const void* x, int x_dt, const void* wg, const 
 //   plan: counts the slots of every expert, gives every slot a row (its expert's rows follow one another; the order
 //     inside an expert is whatever the atomics give, which changes no result: a row's product does not depend on its
 //     place), and lists the 128-row tiles of the grouped product.  One block.
-//   gather: xs[row] = x[slot_of_row[row] / top].
-//   combine: out[t] += sum_c weight[t, c] * y[row_of_slot[t * top + c]], choices in their order.
+//   gather: xs[row] = x[slot_of_row[row] / top] (times the slot's weight, where that multiplies the experts' input).
+//   combine: out[t] += sum_c weight[t, c] * y[row_of_slot[t * top + c]], choices in their order; with a shared
+//     feed-forward's branch also + gate[t] * branch[t]; and it can leave the RMS norm that reads the stream next, since it
+//     holds the stream's new row.
 // ---------------------------------------------------------------------------
 __global__ void __launch_bounds__(1024)
 moe_plan_kernel(const int* __restrict__ ids, int n_slots, int n_experts, int* __restrict__ row_of_slot,
@@ -2254,9 +2413,30 @@ extern "C" int nncpu_moe_plan(const int* ids, int n_slots, int n_experts, int* r
 
 __global__ void __launch_bounds__(256)
 moe_gather_kernel(const void* __restrict__ x, int x_dt, const int* __restrict__ slot_of_row, int top,
-                  __nv_bfloat16* __restrict__ xs, int width) {
+                  const float* __restrict__ weights, __nv_bfloat16* __restrict__ xs, int width) {
     const int row = blockIdx.x;
     const int t = slot_of_row[row] / top;
+    if (weights != nullptr) {
+        const float w = weights[slot_of_row[row]];
+        if (x_dt == DT_BF16 && (width & 7) == 0) {
+            const uint4* src = reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(x) + (size_t)t * width);
+            uint4* dst = reinterpret_cast<uint4*>(xs + (size_t)row * width);
+            for (int i = threadIdx.x; i < (width >> 3); i += blockDim.x) {
+                uint4 v = src[i];
+                __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const float2 f = __bfloat1622float2(h[j]);
+                    h[j] = __floats2bfloat162_rn(f.x * w, f.y * w);
+                }
+                dst[i] = v;
+            }
+        } else {
+            for (int i = threadIdx.x; i < width; i += blockDim.x)
+                xs[(size_t)row * width + i] = __float2bfloat16_rn(ld_f(x, (size_t)t * width + i, x_dt) * w);
+        }
+        return;
+    }
     if (x_dt == DT_BF16 && (width & 7) == 0) {
         const uint4* src = reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(x) + (size_t)t * width);
         uint4* dst = reinterpret_cast<uint4*>(xs + (size_t)row * width);
@@ -2267,10 +2447,10 @@ moe_gather_kernel(const void* __restrict__ x, int x_dt, const int* __restrict__ 
     }
 }
 
-extern "C" int nncpu_moe_gather(const void* x, int x_dt, const int* slot_of_row, int top, void* xs, int n_slots,
-                                int width, void* stream) {
+extern "C" int nncpu_moe_gather(const void* x, int x_dt, const int* slot_of_row, int top, const float* weights, void* xs,
+                                int n_slots, int width, void* stream) {
     NN_CHECK(n_slots > 0 && top > 0 && width > 0, "experts (gather): %d slots of %d", n_slots, width);
-    moe_gather_kernel<<<n_slots, 256, 0, (cudaStream_t)stream>>>(x, x_dt, slot_of_row, top, (__nv_bfloat16*)xs, width);
+    moe_gather_kernel<<<n_slots, 256, 0, (cudaStream_t)stream>>>(x, x_dt, slot_of_row, top, weights, (__nv_bfloat16*)xs, width);
     NN_LAUNCH_OK("experts (gather)");
     return 0;
 }
@@ -2309,10 +2489,87 @@ moe_combine_kernel(const void* __restrict__ y, int y_dt, const int* __restrict__
     }
 }
 
+// The same for float32 y and rows that a block holds in registers (width a multiple of 4, at most 256 * 4 * kVec): the
+// shared branch, and the norm of the new row.
+template <int kVec>
+__global__ void __launch_bounds__(256)
+moe_combine_close_kernel(const float* __restrict__ y, const int* __restrict__ row_of_slot, const float* __restrict__ weights,
+                         float* __restrict__ out, int top, int width, const float* __restrict__ branch,
+                         const float* __restrict__ gate, const void* __restrict__ gamma, int g_dt, float gamma_offset,
+                         float eps, void* __restrict__ norm_out, int norm_dt) {
+    __shared__ float scratch[33];
+    const int t = blockIdx.x, n4 = width >> 2;
+    const float g = branch != nullptr ? (gate != nullptr ? gate[t] : 1.0f) : 0.0f;
+    float4* o4 = reinterpret_cast<float4*>(out + (size_t)t * width);
+    float4 v[kVec];
+    float ss = 0.0f;
+#pragma unroll
+    for (int j = 0; j < kVec; ++j) {
+        const int i = threadIdx.x + j * 256;
+        v[j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (i >= n4) continue;
+        float4 sum = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        const float4 was = o4[i];
+        if (branch != nullptr) {
+            const float4 b = reinterpret_cast<const float4*>(branch + (size_t)t * width)[i];
+            sum = make_float4(g * b.x, g * b.y, g * b.z, g * b.w);
+        }
+        for (int c = 0; c < top; ++c) {
+            const int row = row_of_slot[(size_t)t * top + c];
+            if (row < 0) continue;
+            const float w = weights != nullptr ? weights[(size_t)t * top + c] : 1.0f;
+            const float4 q = reinterpret_cast<const float4*>(y + (size_t)row * width)[i];
+            sum.x = fmaf(w, q.x, sum.x); sum.y = fmaf(w, q.y, sum.y);
+            sum.z = fmaf(w, q.z, sum.z); sum.w = fmaf(w, q.w, sum.w);
+        }
+        v[j] = make_float4(was.x + sum.x, was.y + sum.y, was.z + sum.z, was.w + sum.w);
+        o4[i] = v[j];
+        ss = fmaf(v[j].x, v[j].x, ss); ss = fmaf(v[j].y, v[j].y, ss);
+        ss = fmaf(v[j].z, v[j].z, ss); ss = fmaf(v[j].w, v[j].w, ss);
+    }
+    if (norm_out == nullptr) return;
+    ss = block_sum(ss, scratch);
+    const float scale = 1.0f / sqrtf(ss * (1.0f / (float)width) + eps);
+#pragma unroll
+    for (int j = 0; j < kVec; ++j) {
+        const int i = threadIdx.x + j * 256;
+        if (i >= n4) continue;
+        float o[4] = {v[j].x * scale, v[j].y * scale, v[j].z * scale, v[j].w * scale};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[e] *= ld_f(gamma, 4 * i + e, g_dt) + gamma_offset;
+        const size_t at = (size_t)t * width + 4 * i;
+        if (norm_dt == DT_BF16) {
+            __nv_bfloat162 h[2] = {__floats2bfloat162_rn(o[0], o[1]), __floats2bfloat162_rn(o[2], o[3])};
+            *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(norm_out) + at) = *reinterpret_cast<uint2*>(h);
+        } else {
+            *reinterpret_cast<float4*>(reinterpret_cast<float*>(norm_out) + at) = make_float4(o[0], o[1], o[2], o[3]);
+        }
+    }
+}
+
+// Whether moe_combine takes a shared branch or leaves the norm that follows, for rows of `width` lanes.
+extern "C" int nncpu_moe_combine_closes(int width) { return width > 0 && width % 4 == 0 && width <= 256 * 4 * 8; }
+
 extern "C" int nncpu_moe_combine(const void* y, int y_dt, const int* row_of_slot, const float* weights, float* out,
-                                 int n_tok, int top, int width, void* stream) {
+                                 int n_tok, int top, int width, const float* branch, const float* gate, const void* gamma,
+                                 int g_dt, float gamma_offset, float eps, void* norm_out, int norm_dt, void* stream) {
     NN_CHECK(n_tok > 0 && top > 0 && width > 0, "experts (combine): %d tokens of %d", n_tok, width);
-    moe_combine_kernel<<<n_tok, 256, 0, (cudaStream_t)stream>>>(y, y_dt, row_of_slot, weights, out, top, width);
+    if (branch == nullptr && norm_out == nullptr && weights != nullptr) {
+        moe_combine_kernel<<<n_tok, 256, 0, (cudaStream_t)stream>>>(y, y_dt, row_of_slot, weights, out, top, width);
+        NN_LAUNCH_OK("experts (combine)");
+        return 0;
+    }
+    NN_CHECK(y_dt == DT_F32 && nncpu_moe_combine_closes(width), "experts (combine): rows of %d lanes cannot be closed", width);
+    NN_CHECK(((uintptr_t)y | (uintptr_t)out | (uintptr_t)branch | (uintptr_t)norm_out) % 16 == 0,
+             "experts (combine): rows must be 16-byte aligned");
+#define NN_CLOSE(V)                                                                                                     \
+    moe_combine_close_kernel<V><<<n_tok, 256, 0, (cudaStream_t)stream>>>((const float*)y, row_of_slot, weights, out, top, \
+                                                                         width, branch, gate, gamma, g_dt, gamma_offset, eps, norm_out, norm_dt)
+    if (width <= 256 * 4) NN_CLOSE(1);
+    else if (width <= 256 * 4 * 2) NN_CLOSE(2);
+    else if (width <= 256 * 4 * 4) NN_CLOSE(4);
+    else NN_CLOSE(8);
+#undef NN_CLOSE
     NN_LAUNCH_OK("experts (combine)");
     return 0;
 }

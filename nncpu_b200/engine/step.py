@@ -48,17 +48,18 @@ class StepContext:
     branch_is_fresh: bool = False         # the "residual" a part was given is an uninitialised branch: its last product writes, not adds
     out_scale: float = 1.0                # a part that says ``scales_output`` multiplies what it adds to the stream by this
 
-    def span_sum(self, window: int = 0, chunk: int = 0) -> int:
+    def span_sum(self, window: int = 0, chunk: int = 0, keep_first: int = 0) -> int:
         """Keys that the step's tokens attend to, summed over the tokens: a token at position p sees p + 1
-        keys, or the last ``window`` of them, or the p % chunk + 1 of its own block of ``chunk`` positions."""
-        key = ("span_sum", window, chunk)
+        keys, or the last ``window`` of them (and the first ``keep_first``), or the p % chunk + 1 of its own block of
+        ``chunk`` positions."""
+        key = ("span_sum", window, chunk, keep_first)
         n = self.memo.get(key)
         if n is None:
             n = 0
             for q, after in zip(self.q_lens, self.kv_lens):
                 first = after - q + 1                      # keys seen by the sequence's first new token
                 if window > 0:
-                    n += sum(min(first + i, window) for i in range(q))
+                    n += sum(min(first + i, window + keep_first) for i in range(q))
                 elif chunk > 0:
                     n += sum((first - 1 + i) % chunk + 1 for i in range(q))
                 else:

@@ -482,6 +482,31 @@ def qk_norm_rope_append(qkv, q_gamma, k_gamma, eps, cos_sin, tok_seq, tok_pos, b
           _i(values_are_keys), _stream())
 
 
+def qk_whole_norm_append(qkv, q_gamma, k_gamma, eps, cos_sin, tok_seq, tok_pos, block_table, k_pages, v_pages, q_out,
+                         n_heads: int, n_kv: int, head_dim: int, v_head_dim: int) -> None:
+    """As ``qk_norm_rope_append`` for mixers whose query and key norm runs over ALL of a token's query (key) lanes at once
+    (weights [n_heads * head_dim] and [n_kv * head_dim], or None: no norm), and whose rotation turns neighbouring lanes:
+    ``cos_sin`` [n, pairs, 2] turns a head's first ``pairs`` pairs (2i, 2i + 1).  A head lies in ``q_out`` and in the
+    pages in rows as long as theirs, with zeros behind its own lanes.  qkv float32 [n, >= (n_heads + n_kv) * head_dim +
+    n_kv * v_head_dim]."""
+    n = q_out.shape[0]
+    half = 0 if cos_sin is None else cos_sin.shape[1]
+    qp = q_out.shape[1] // n_heads
+    assert qkv.dtype == torch.float32 and qkv.shape[0] == n and qkv.is_contiguous() and q_out.shape[1] == qp * n_heads
+    assert qkv.shape[1] >= (n_heads + n_kv) * head_dim + n_kv * v_head_dim
+    assert q_gamma is None or q_gamma.numel() == n_heads * head_dim
+    assert k_gamma is None or k_gamma.numel() == n_kv * head_dim
+    assert q_gamma is None or k_gamma is None or q_gamma.dtype == k_gamma.dtype
+    assert cos_sin is None or (cos_sin.dtype == torch.float32 and cos_sin.shape == (n, half, 2))
+    assert n_kv == 0 or (k_pages.shape[1] == v_pages.shape[1] == n_kv and k_pages.shape[-1] == qp and k_pages.dtype == v_pages.dtype)
+    g = q_gamma if q_gamma is not None else k_gamma
+    _call("generic", "nncpu_qk_whole_norm_append", _ptr(qkv), _i(qkv.shape[1]), _ptr(q_gamma), _ptr(k_gamma), _i(_code(g)),
+          _f(eps), _ptr(cos_sin), _i(half), _ptr(tok_seq), _ptr(tok_pos), _ptr(block_table),
+          _i(block_table.shape[1] if block_table is not None else 0), _ptr(k_pages), _ptr(v_pages), _i(_code(k_pages)),
+          _ptr(q_out), _i(_code(q_out)), _i(n), _i(n_heads), _i(n_kv), _i(head_dim), _i(v_head_dim), _i(qp),
+          _i(v_pages.shape[-1] if n_kv else v_head_dim), _stream())
+
+
 def key_span(window: int = 0, chunk: int = 0) -> int:
     """The one number by which every attention kernel knows which earlier keys a query sees (their ``window``
     argument): ``window`` > 0, the last ``window`` keys up to the query, as it is; ``chunk`` > 0, the keys of the
@@ -492,29 +517,43 @@ def key_span(window: int = 0, chunk: int = 0) -> int:
 
 
 def attention(q, k_pages, v_pages, block_table, tok_seq, tok_pos, out, n_heads: int, n_kv: int, head_dim: int,
-              scale: float, window: int = 0, v_head_dim: int = 0, slope_base: float = 0.0, sinks=None) -> None:
+              scale: float, window: int = 0, v_head_dim: int = 0, slope_base: float = 0.0, sinks=None, keep: int = 0,
+              v_lanes: int = 0) -> None:
     """Causal attention of each token over its sequence's pages.  ``window``: see ``key_span`` (here and in the
-    other attention kernels).  ``v_head_dim``: lanes of a value head (and of
-    the output) when they differ from ``head_dim``.  ``slope_base`` b != 0: head h takes
+    other attention kernels).  ``keep``: with a window, the sequence's first ``keep`` keys stay visible (here and in the
+    other attention kernels).  ``v_head_dim``: lanes of a value row when they differ from ``head_dim``; ``v_lanes``: how
+    many of them the output has (0: all).  ``slope_base`` b != 0: head h takes
     2^(-b (h + 1) / n_heads) * (query position - key position) off its scaled scores.  ``sinks`` (float32
     [n_heads]): exp(sinks[h]) joins the denominator of head h's softmax (here and in the other attention kernels)."""
     n = q.shape[0]
     v_head_dim = v_head_dim or head_dim
-    assert q.shape == (n, n_heads * head_dim) and out.shape == (n, n_heads * v_head_dim)
+    v_lanes = v_lanes or v_head_dim
+    assert q.shape == (n, n_heads * head_dim) and out.shape == (n, n_heads * v_lanes)
+    assert keep == 0 or window > 0
     assert k_pages.dtype == v_pages.dtype and block_table.dtype == torch.int32
     assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == n_heads)
     _call("generic", "nncpu_attention", _ptr(q), _i(_code(q)), _ptr(k_pages), _ptr(v_pages), _i(_code(k_pages)),
           _ptr(block_table), _i(block_table.shape[1]), _ptr(tok_seq), _ptr(tok_pos), _ptr(out), _i(_code(out)),
-          _i(n), _i(n_heads), _i(n_kv), _i(head_dim), _i(v_head_dim), _f(scale), _i(window), _f(slope_base), _ptr(sinks),
-          _stream())
+          _i(n), _i(n_heads), _i(n_kv), _i(head_dim), _i(v_head_dim), _i(v_lanes), _f(scale), _i(window), _i(keep),
+          _f(slope_base), _ptr(sinks), _stream())
 
 
 def attention_mma_supported(n_heads: int, n_kv: int, head_dim: int, *tensors) -> bool:
     """The tensor-core attention kernels take bfloat16 q, cache and output with
-    head size 64 or 128 (where more than 16 query heads share a key/value head, several blocks of the decode
+    key rows of 64 or 128 lanes and value rows of 64 lanes or the keys' size, see ``attention_rows`` (where more than 16 query heads share a key/value head, several blocks of the decode
     kernel take a part of them each)."""
     return (head_dim in (64, 128) and n_kv > 0 and n_heads % n_kv == 0
             and all(t.dtype == torch.bfloat16 for t in tensors))
+
+
+def attention_rows(head_dim: int, v_head_dim: int):
+    """Lanes of the page rows of keys and of values in which the tensor-core attention kernels take heads of these sizes
+    (zeros behind a head's own lanes), or None where they take none."""
+    if head_dim > 128 or v_head_dim > 128:
+        return None
+    if v_head_dim > 64:
+        return 128, 128
+    return (64 if head_dim <= 64 else 128), 64
 
 
 # How decode attention cuts a sequence's keys into splits: the kernel's launch bounds let two of its blocks run on
@@ -540,63 +579,77 @@ def attention_decode_scratch_floats(n_tok: int, n_heads: int, n_kv: int, head_di
 
 def attention_decode_mma(q, k_pages, v_pages, block_table, tok_seq, tok_pos, out, scratch, n_heads: int, n_kv: int,
                          head_dim: int, scale: float, window: int, n_splits: int, slope_base: float = 0.0,
-                         sinks=None) -> None:
+                         sinks=None, keep: int = 0, v_lanes: int = 0) -> None:
     """One token per sequence; each token's keys are cut into ``n_splits``
-    splits that run in parallel.  With ``scratch`` (float32,
+    splits that run in parallel.  ``head_dim`` is the size of q's heads and of the pages' key rows, ``v_lanes`` that of
+    the output's heads (0: ``head_dim``; at most the value rows').  With ``scratch`` (float32,
     ``attention_decode_scratch_floats`` elements) a second kernel merges them;
     with ``scratch`` None and at most 8 splits they form a thread-block
     cluster and merge through distributed shared memory.  ``sinks`` as in ``attention``: the term joins where the
     splits merge, once."""
     n = q.shape[0]
-    assert q.shape == (n, n_heads * head_dim) and out.shape == q.shape
+    v_lanes = v_lanes or head_dim
+    assert q.shape == (n, n_heads * head_dim) and out.shape == (n, n_heads * v_lanes)
     assert scratch is None or scratch.dtype == torch.float32
     assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == n_heads)
     _call("attention_mma", "nncpu_attention_decode_mma", _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table),
           _i(block_table.shape[1]), _ptr(tok_seq), _ptr(tok_pos), _ptr(out), _ptr(scratch),
           ctypes.c_long(0 if scratch is None else scratch.numel()), _i(n), _i(n_heads), _i(n_kv), _i(head_dim),
-          _f(scale), _i(window), _i(n_splits), _f(slope_base), _ptr(sinks), _stream())
+          _i(v_pages.shape[-1]), _i(v_lanes), _f(scale), _i(window), _i(keep), _i(n_splits), _f(slope_base), _ptr(sinks), _stream())
 
 
 def attention_decode_mma_from_qkv(qkv, q_gamma, k_gamma, eps, cos_sin, k_pages, v_pages, append: bool, block_table,
                                   tok_seq, tok_pos, out, scratch, n_heads: int, n_kv: int, head_dim: int, scale: float,
                                   window: int, n_splits: int, slope_base: float = 0.0, q_temp=None, sinks=None,
-                                  values_are_keys: bool = False, gated: bool = False) -> None:
+                                  values_are_keys: bool = False, gated: bool = False, keep: int = 0, v_head_dim: int = 0,
+                                  whole_norm: bool = False, rot_pairs: bool = False) -> None:
     """Decode attention that starts from the float32 projections ``qkv`` [n, per_tok * head_dim] (q heads, then with
     ``append`` the k and v heads): every block makes its queries itself (per-head norm, rotation by ``cos_sin``
     [n, head_dim / 2, 2]), and with ``append`` the token's key and value are made, written to the cache and used.
     One launch in place of ``qk_norm_rope_append`` and ``attention_decode_mma``, with the same arithmetic;
     ``slope_base``, ``q_temp`` and ``sinks`` as there.  ``values_are_keys``: the rows hold no v heads, a token's value
     is its key as projected.  ``gated``: n_heads more heads of logits end the rows, and the output is multiplied lane by
-    lane by their sigmoid (in place of ``sigmoid_gate``)."""
+    lane by their sigmoid (in place of ``sigmoid_gate``).  ``head_dim`` and ``v_head_dim`` (0: the same) are the heads' own
+    sizes; the pages' rows may be longer (``attention_rows``), with zeros behind them.  ``whole_norm``: the norm runs over
+    all of a token's query (key) lanes at once, as in ``qk_whole_norm_append``.  ``rot_pairs``: ``cos_sin`` [n, pairs, 2]
+    turns a head's first neighbouring pairs of lanes."""
     n = out.shape[0]
-    per_tok = n_heads + (((1 if values_are_keys else 2) * n_kv) if append else 0) + (n_heads if gated else 0)
+    v_head_dim = v_head_dim or head_dim
+    row = n_heads * head_dim + ((n_kv * head_dim + (0 if values_are_keys else n_kv * v_head_dim)) if append else 0)
+    row += n_heads * v_head_dim if gated else 0
+    rot_half = 0 if cos_sin is None else cos_sin.shape[1]
     assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == n_heads)
-    assert qkv.dtype == torch.float32 and qkv.shape == (n, per_tok * head_dim) and qkv.is_contiguous()
-    assert out.shape == (n, n_heads * head_dim) and out.dtype == torch.bfloat16
+    assert qkv.dtype == torch.float32 and qkv.shape == (n, row) and qkv.is_contiguous()
+    assert out.shape == (n, n_heads * v_head_dim) and out.dtype == torch.bfloat16
     assert k_pages.dtype == v_pages.dtype == torch.bfloat16 and k_pages.is_contiguous() and v_pages.is_contiguous()
-    assert cos_sin is None or (cos_sin.dtype == torch.float32 and cos_sin.shape == (n, head_dim // 2, 2))
+    assert cos_sin is None or (cos_sin.dtype == torch.float32 and cos_sin.shape == (n, rot_half if rot_pairs else head_dim // 2, 2))
     assert q_gamma is None or k_gamma is None or q_gamma.dtype == k_gamma.dtype
+    assert q_gamma is None or q_gamma.numel() == (n_heads * head_dim if whole_norm else head_dim)
+    assert k_gamma is None or k_gamma.numel() == (n_kv * head_dim if whole_norm else head_dim)
     assert scratch is None or scratch.dtype == torch.float32
     g = q_gamma if q_gamma is not None else k_gamma
     _call("attention_mma", "nncpu_attention_decode_mma_from_qkv", _ptr(qkv), _ptr(q_gamma), _ptr(k_gamma), _i(_code(g)),
           _f(eps), _ptr(cos_sin), _ptr(k_pages), _ptr(v_pages), _i(append), _ptr(block_table), _i(block_table.shape[1]),
           _ptr(tok_seq), _ptr(tok_pos), _ptr(out), _ptr(scratch), ctypes.c_long(0 if scratch is None else scratch.numel()),
-          _i(n), _i(n_heads), _i(n_kv), _i(head_dim), _f(scale), _i(window), _i(n_splits), _f(slope_base),
+          _i(n), _i(n_heads), _i(n_kv), _i(k_pages.shape[-1]), _i(v_pages.shape[-1]), _i(head_dim), _i(v_head_dim),
+          _i(whole_norm), _i(rot_half), _i(rot_pairs), _f(scale), _i(window), _i(keep), _i(n_splits), _f(slope_base),
           _f(q_temp[0] if q_temp else 0.0), _i(q_temp[1] if q_temp else 1), _ptr(sinks), _i(values_are_keys), _i(gated),
           _stream())
 
 
 def attention_prefill_mma(q, k_pages, v_pages, block_table, cu_seqlens, tok_pos, out, n_seqs: int, n_heads: int,
                           n_kv: int, head_dim: int, scale: float, window: int, slope_base: float = 0.0,
-                          sinks=None) -> None:
-    """Any number of new tokens per sequence, at consecutive positions.  ``slope_base`` and ``sinks`` as in
-    ``attention``."""
+                          sinks=None, keep: int = 0, v_lanes: int = 0) -> None:
+    """Any number of new tokens per sequence, at consecutive positions.  ``slope_base``, ``sinks`` and ``keep`` as in
+    ``attention``, ``v_lanes`` as in ``attention_decode_mma``."""
     n = q.shape[0]
-    assert q.shape == (n, n_heads * head_dim) and out.shape == q.shape and cu_seqlens.numel() >= n_seqs + 1
+    v_lanes = v_lanes or head_dim
+    assert q.shape == (n, n_heads * head_dim) and out.shape == (n, n_heads * v_lanes) and cu_seqlens.numel() >= n_seqs + 1
     assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == n_heads)
     _call("attention_mma", "nncpu_attention_prefill_mma", _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table),
           _i(block_table.shape[1]), _ptr(cu_seqlens), _ptr(tok_pos), _ptr(out), _i(n), _i(n_seqs), _i(n_heads),
-          _i(n_kv), _i(head_dim), _f(scale), _i(window), _f(slope_base), _ptr(sinks), _stream())
+          _i(n_kv), _i(head_dim), _i(v_pages.shape[-1]), _i(v_lanes), _f(scale), _i(window), _i(keep), _f(slope_base),
+          _ptr(sinks), _stream())
 
 
 def attention_prefill_tc_supported(n_heads: int, n_kv: int, head_dim: int, *tensors) -> bool:
@@ -608,20 +661,21 @@ def attention_prefill_tc_supported(n_heads: int, n_kv: int, head_dim: int, *tens
 
 def attention_prefill_tc(q, k_pages, v_pages, block_table, cu_seqlens, tok_pos, out, status, n_seqs: int,
                          n_heads: int, n_kv: int, head_dim: int, scale: float, window: int, slope_base: float = 0.0,
-                         sinks=None) -> None:
+                         sinks=None, keep: int = 0, v_lanes: int = 0) -> None:
     """Prefill attention on the tcgen05 tensor cores: any number of new tokens per sequence, at consecutive
     positions; ``status`` is an int32 word on the device that receives a code if a bounded wait runs out.
-    ``slope_base`` and ``sinks`` as in ``attention``."""
+    ``slope_base``, ``sinks`` and ``keep`` as in ``attention``, ``v_lanes`` as in ``attention_decode_mma``."""
     assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == n_heads)
     n = q.shape[0]
-    assert q.shape == (n, n_heads * head_dim) and out.shape == q.shape and cu_seqlens.numel() >= n_seqs + 1
+    v_lanes = v_lanes or head_dim
+    assert q.shape == (n, n_heads * head_dim) and out.shape == (n, n_heads * v_lanes) and cu_seqlens.numel() >= n_seqs + 1
     assert q.is_contiguous() and out.is_contiguous() and k_pages.is_contiguous() and v_pages.is_contiguous()
-    assert k_pages.shape[1:] == (n_kv, 64, head_dim) and v_pages.shape == k_pages.shape
+    assert k_pages.shape[1:] == (n_kv, 64, head_dim) and v_pages.shape[:-1] == k_pages.shape[:-1]
     assert status.dtype == torch.int32
     _call("attention_tc", "nncpu_attention_prefill_tc", _ptr(q), _ptr(k_pages), _ptr(v_pages), _i(k_pages.shape[0]),
           _ptr(block_table), _i(block_table.shape[1]), _ptr(cu_seqlens), _ptr(tok_pos), _ptr(out), _i(n), _i(n_seqs),
-          _i(n_heads), _i(n_kv), _i(head_dim), _f(scale), _i(window), _f(slope_base), _ptr(sinks),
-          _ptr(status), _stream())
+          _i(n_heads), _i(n_kv), _i(head_dim), _i(v_pages.shape[-1]), _i(v_lanes), _f(scale), _i(window), _i(keep),
+          _f(slope_base), _ptr(sinks), _ptr(status), _stream())
 
 
 GATED_ACTS = {"silu": 0, "gelu_tanh": 1, "swish_clamp": 2}
@@ -758,24 +812,30 @@ def _route_mode(scoring):
     """``scoring`` None: the softmax over the chosen logits alone.  ("all", n_groups, keep, scale): scores are the
     softmax over all experts; the experts form ``n_groups`` equal groups of neighbours whose score is their best
     expert's, and only experts of the ``keep`` best groups can be chosen (``n_groups`` <= 1: no groups); the weights
-    are the chosen scores divided by their sum (+ 1e-20), times ``scale``."""
+    are the chosen scores divided by their sum (+ 1e-20), times ``scale``.  ("sigmoid",): scores are the sigmoids of the
+    logits, and the weights are the chosen scores as they are."""
     if scoring is None:
         return _i(0), _i(1), _i(1), _f(1.0)
+    if scoring[0] == "sigmoid":
+        return _i(2), _i(1), _i(1), _f(1.0)
     kind, n_groups, keep, scale = scoring
     if kind != "all":
         raise InvalidArgument(f"a router cannot score by {kind!r}")
     return _i(1), _i(max(1, n_groups)), _i(max(1, keep)), _f(scale)
 
 
-def moe_route(logits, top: int, ids, weights, scoring=None) -> None:
+def moe_route(logits, top: int, ids, weights, scoring=None, gate=None) -> None:
     """Per row of float32 logits [n, E]: ids [n, top] (int32) of the largest logits in descending order (the lower
     index wins a tie) and weights [n, top] (float32), the softmax over those logits alone, or what ``scoring`` says
-    (see ``_route_mode``)."""
-    n, E = logits.shape
+    (see ``_route_mode``).  ``gate`` (float32 [n]): the column after the experts' is the logit of a gate per token, whose
+    sigmoid is left there."""
+    n, cols = logits.shape
+    E = cols - (0 if gate is None else 1)
+    assert gate is None or (gate.dtype == torch.float32 and gate.numel() == n)
     assert logits.dtype == torch.float32 and ids.dtype == torch.int32 and weights.dtype == torch.float32
     assert ids.shape == weights.shape == (n, top)
     _call("generic", "nncpu_moe_route", _ptr(logits), _i(n), _i(E), _i(top), _ptr(ids), _ptr(weights),
-          *_route_mode(scoring), _stream())
+          *_route_mode(scoring), _i(cols), _ptr(gate), _stream())
 
 
 def moe_router_fits(n_experts: int, width: int) -> bool:
@@ -783,23 +843,37 @@ def moe_router_fits(n_experts: int, width: int) -> bool:
     return 0 < n_experts <= 1024 and (width + 2 * n_experts) * 4 <= 48 * 1024
 
 
-def moe_router(x, w, bias, top: int, ids, weights, scoring=None) -> None:
-    """The router in one launch: logits = x . w^T + bias in 32-bit, then ``moe_route``'s choice and weights."""
+def moe_router(x, w, bias, top: int, ids, weights, scoring=None, gate=None) -> None:
+    """The router in one launch: logits = x . w^T + bias in 32-bit, then ``moe_route``'s choice and weights (with ``gate``
+    the last row of w is the gate's)."""
     n, width = x.shape
-    E = w.shape[0]
-    assert w.shape == (E, width) and (bias is None or bias.numel() == E) and ids.shape == weights.shape == (n, top)
+    E = w.shape[0] - (0 if gate is None else 1)
+    assert gate is None or (gate.dtype == torch.float32 and gate.numel() == n and bias is None)
+    assert w.shape[1] == width and (bias is None or bias.numel() == E) and ids.shape == weights.shape == (n, top)
     assert ids.dtype == torch.int32 and weights.dtype == torch.float32
     _call("generic", "nncpu_moe_router", _ptr(x), _i(_code(x)), _ptr(w), _i(_code(w)), _ptr(bias), _i(_code(bias)), _i(n),
-          _i(E), _i(top), _i(width), _ptr(ids), _ptr(weights), *_route_mode(scoring), _stream())
+          _i(E), _i(top), _i(width), _ptr(ids), _ptr(weights), *_route_mode(scoring), _ptr(gate), _stream())
 
 
-def moe_experts(x, w_gate, w_up, w_down, ids, weights, act, out, kind: str, limit: float = 0.0) -> None:
+def moe_experts(x, w_gate, w_up, w_down, ids, weights, act, out, kind: str, limit: float = 0.0,
+                weight_on_input: bool = False, shared=None) -> None:
     """out[t] += sum_c weights[t, c] * W_down[e] act(W_gate[e] x_t, W_up[e] x_t) with e = ids[t, c].  Weights are
     [E, ff, width] (gate, up) and [E, width, ff] (down); with ``w_up`` None, ``w_gate`` is [E, 2 ff, width] with an
     expert's gate and up rows interleaved in blocks of 8 (the layout of the grouped product).  ``act`` [n * top, ff] is
     scratch in the run's type; out is the float32 stream.  Every token reads its experts' rows itself: the kernel for
-    few tokens and for every size and type."""
+    few tokens and for every size and type.  ``weight_on_input``: out[t] += sum_c W_down[e] act(W_gate[e] (w x_t), W_up[e]
+    (w x_t)) instead, w = weights[t, c].  ``shared`` = (w_gate, w_up or None, w_down, act [n, sff], gate [n]): a shared
+    feed-forward of the same form in the same launches, its output times the token's gate; its matrices [sff, width] (or
+    [2 sff, width] interleaved) and [width, sff]."""
     n, width = x.shape
+    sg = su = sd = sact = sgate = None
+    sff = 0
+    if shared is not None:
+        sg, su, sd, sact, sgate = shared
+        sff = sd.shape[1]
+        assert sd.shape == (width, sff) and sd.dtype == sg.dtype == w_down.dtype and sact.shape == (n, sff) and sact.dtype == act.dtype
+        assert sg.shape == ((2 * sff if su is None else sff), width) and (su is None or su.shape == (sff, width))
+        assert sgate.dtype == torch.float32 and sgate.numel() == n
     E, ff = w_down.shape[0], w_down.shape[2]
     top = ids.shape[1]
     assert w_down.shape == (E, width, ff) and w_gate.dtype == w_down.dtype
@@ -808,7 +882,8 @@ def moe_experts(x, w_gate, w_up, w_down, ids, weights, act, out, kind: str, limi
     assert act.shape == (n * top, ff) and out.shape == (n, width) and out.dtype == torch.float32
     _call("generic", "nncpu_moe_experts", _ptr(x), _i(_code(x)), _ptr(w_gate), _ptr(w_up), _ptr(w_down), _i(_code(w_gate)),
           _ptr(ids), _ptr(weights), _ptr(act), _i(_code(act)), _ptr(out), _i(n), _i(top), _i(width), _i(ff), _i(E),
-          _i(GATED_ACTS[kind]), _f(limit), _stream())
+          _i(GATED_ACTS[kind]), _f(limit), _i(weight_on_input), _ptr(sg), _ptr(su), _ptr(sd), _i(sff), _ptr(sact), _ptr(sgate),
+          _stream())
 
 
 def moe_plan_tiles(n_slots: int, n_experts: int) -> int:
@@ -830,19 +905,38 @@ def moe_plan(ids, n_experts: int, row_of_slot, slot_of_row, plan) -> None:
           at(1 + mt), at(1 + 2 * mt), _i(mt), _stream())
 
 
-def moe_gather(x, slot_of_row, top: int, xs) -> None:
-    """xs[row] = x[slot_of_row[row] // top] as bfloat16: the tokens' rows in the order of the grouped product."""
+def moe_gather(x, slot_of_row, top: int, xs, weights=None) -> None:
+    """xs[row] = x[slot_of_row[row] // top] as bfloat16: the tokens' rows in the order of the grouped product; with
+    ``weights`` [n, top] each times its slot's weight."""
     S, width = xs.shape
+    assert weights is None or (weights.dtype == torch.float32 and weights.numel() == S)
     assert xs.dtype == torch.bfloat16 and x.shape[1] == width and slot_of_row.numel() == S
-    _call("generic", "nncpu_moe_gather", _ptr(x), _i(_code(x)), _ptr(slot_of_row), _i(top), _ptr(xs), _i(S), _i(width), _stream())
+    _call("generic", "nncpu_moe_gather", _ptr(x), _i(_code(x)), _ptr(slot_of_row), _i(top), _ptr(weights), _ptr(xs), _i(S), _i(width),
+          _stream())
 
 
-def moe_combine(y, row_of_slot, weights, out) -> None:
-    """out[t] += sum_c weights[t, c] * y[row_of_slot[t * top + c]], choices in their order; out float32."""
-    n, top = weights.shape
-    assert out.dtype == torch.float32 and out.shape == (n, y.shape[1]) and row_of_slot.numel() == n * top
+def moe_combine_closes(width: int) -> bool:
+    """Whether ``moe_combine`` takes a shared branch or leaves the norm that follows, for rows of ``width`` lanes."""
+    return width > 0 and width % 4 == 0 and width <= 8192
+
+
+def moe_combine(y, row_of_slot, weights, out, top: int = 0, branch=None, gate=None, then_norm=None) -> None:
+    """out[t] += sum_c weights[t, c] * y[row_of_slot[t * top + c]], choices in their order; out float32.  ``weights``
+    None: ones (``top`` is then given).  ``branch`` (float32, out's shape): + gate[t] * branch[t] (``gate`` None: + branch[t]).
+    ``then_norm`` = (gamma, offset, eps, norm_out): the RMS norm of the new rows is left there in the same pass."""
+    n, width = out.shape
+    top = weights.shape[1] if weights is not None else top
+    assert out.dtype == torch.float32 and y.shape[1] == width and row_of_slot.numel() == n * top and out.is_contiguous()
+    assert branch is None or (branch.dtype == torch.float32 and branch.shape == out.shape and branch.is_contiguous())
+    assert gate is None or (gate.dtype == torch.float32 and gate.numel() == n)
+    gamma = norm_out = None
+    offset = eps = 0.0
+    if then_norm is not None:
+        gamma, offset, eps, norm_out = then_norm
+        assert gamma.numel() == width and norm_out.shape == out.shape and norm_out.is_contiguous()
     _call("generic", "nncpu_moe_combine", _ptr(y), _i(_code(y)), _ptr(row_of_slot), _ptr(weights), _ptr(out), _i(n), _i(top),
-          _i(out.shape[1]), _stream())
+          _i(width), _ptr(branch), _ptr(gate), _ptr(gamma), _i(_code(gamma)), _f(offset), _f(eps), _ptr(norm_out),
+          _i(_code(norm_out)), _stream())
 
 
 def linear_tc_grouped(xs, w, out, plan, n_experts: int, workspace: GemmWorkspace, epilogue: str = "plain",
@@ -1017,6 +1111,81 @@ def delta_scan(xc, gb, state, seq_slots, cu_seqlens, o, n_seqs: int, n_heads: in
     assert seq_slots.dtype == torch.int32 and cu_seqlens.dtype == torch.int32 and cu_seqlens.numel() >= n_seqs + 1
     _call("recurrent", "nncpu_delta_scan", _ptr(xc), _ptr(gb), _ptr(chan_g), _ptr(state), _l(state.shape[1]), _ptr(seq_slots), _ptr(cu_seqlens), _ptr(o),
           _i(n_seqs), _i(n_heads), _i(n_kv), _i(d), _i(e), _stream())
+
+
+def ssm_state_floats(n_heads: int, value_dim: int, n_groups: int, state: int, taps: int) -> int:
+    """Floats of a sequence's state row: S of every head, then the ring of the convolutions' inputs."""
+    s = (n_heads * state * value_dim + 3) // 4 * 4 + taps * (n_heads * value_dim + 2 * n_groups * state)
+    return (s + 3) // 4 * 4
+
+
+def ssm_row(n_heads: int, value_dim: int, n_groups: int, state: int) -> int:
+    """Lanes of a convolved row: the heads' x, the groups' B, the groups' C, each in a multiple of 8 lanes."""
+    return n_heads * ((value_dim + 7) // 8 * 8) + 2 * n_groups * ((state + 7) // 8 * 8)
+
+
+def _ssm_check(proj, state, sizes):
+    H, P, G, N, taps = sizes
+    assert proj.dtype == torch.float32 and proj.is_contiguous() and proj.shape[1] >= 2 * H * P + 2 * G * N + H
+    assert state.dtype == torch.float32 and state.dim() == 2 and state.is_contiguous()
+    assert state.shape[1] >= ssm_state_floats(H, P, G, N, taps)
+
+
+def ssm_conv(proj, conv_w, conv_b, state, tok_seq, tok_pos, seq_slots, cu_seqlens, dt_bias, a_log, xc, gd, sizes) -> None:
+    """What the state-space recurrence reads, from the projections.  ``sizes`` = (heads H, value lanes P, groups G, state
+    rows N, taps).  ``proj`` float32 [n, >= 2 H P + 2 G N + H] holds z, x, B, C, dt per token; ``xc`` [n, ssm_row]
+    receives silu(conv(.) + bias) of x, B and C, ``gd`` float32 [n, 2 H] the decays' logarithms -exp(A_log) dt and then
+    dt = softplus(. + dt_bias).  ``state`` float32 [slots, >= ssm_state_floats]: the inputs before this step's (read only)."""
+    H, P, G, N, taps = sizes
+    n = xc.shape[0]
+    _ssm_check(proj, state, sizes)
+    C = H * P + 2 * G * N
+    assert conv_w.shape == (C, taps) and conv_w.is_contiguous() and conv_b.numel() == C
+    assert dt_bias.numel() == a_log.numel() == H and dt_bias.dtype == a_log.dtype
+    assert xc.shape == (n, ssm_row(H, P, G, N)) and gd.shape == (n, 2 * H) and gd.dtype == torch.float32
+    assert tok_seq.dtype == tok_pos.dtype == seq_slots.dtype == cu_seqlens.dtype == torch.int32
+    _call("state_space", "nncpu_ssm_conv", _ptr(proj), _i(proj.shape[1]), _ptr(conv_w), _i(_code(conv_w)), _ptr(conv_b),
+          _i(_code(conv_b)), _ptr(state), _l(state.shape[1]), _ptr(tok_seq), _ptr(tok_pos), _ptr(seq_slots), _ptr(cu_seqlens),
+          _ptr(dt_bias), _ptr(a_log), _i(_code(a_log)), _ptr(xc), _i(_code(xc)), _ptr(gd), _i(n), _i(H), _i(P), _i(G), _i(N),
+          _i(taps), _stream())
+
+
+def ssm_scan(proj, xc, gd, state, seq_slots, cu_seqlens, tok_pos, d_skip, y, n_seqs: int, sizes) -> None:
+    """The state-space recurrence over the step's tokens, sequence by sequence in order, in 32-bit on the CUDA cores:
+    S <- exp(la) S + dt B x^T, y = S^T C + D x.  ``state`` is read and left updated for the slots in ``seq_slots``, the ring
+    of the convolutions' inputs included (negative: a padding sequence, zeros out); ``y`` float32 [n, H P]."""
+    H, P, G, N, taps = sizes
+    n = y.shape[0]
+    _ssm_check(proj, state, sizes)
+    assert xc.shape == (n, ssm_row(H, P, G, N)) and xc.is_contiguous() and gd.shape == (n, 2 * H) and d_skip.numel() == H
+    assert y.shape == (n, H * P) and y.dtype == torch.float32
+    _call("state_space", "nncpu_ssm_scan", _ptr(proj), _i(proj.shape[1]), _ptr(xc), _i(_code(xc)), _ptr(gd), _ptr(state),
+          _l(state.shape[1]), _ptr(seq_slots), _ptr(cu_seqlens), _ptr(tok_pos), _ptr(d_skip), _i(_code(d_skip)), _ptr(y),
+          _i(n_seqs), _i(H), _i(P), _i(G), _i(N), _i(taps), _stream())
+
+
+def ssm_step(proj, conv_w, conv_b, state, tok_pos, seq_slots, dt_bias, a_log, d_skip, y, sizes) -> None:
+    """A decode step, one token per sequence, from the projections to y in one launch: convolutions, step size, recurrence
+    and read-out (as ``ssm_conv`` and ``ssm_scan`` with sequences of one token)."""
+    H, P, G, N, taps = sizes
+    n = y.shape[0]
+    _ssm_check(proj, state, sizes)
+    C = H * P + 2 * G * N
+    assert conv_w.shape == (C, taps) and conv_w.is_contiguous() and conv_b.numel() == C
+    assert dt_bias.numel() == a_log.numel() == d_skip.numel() == H and dt_bias.dtype == a_log.dtype == d_skip.dtype
+    assert y.shape == (n, H * P) and y.dtype == torch.float32 and seq_slots.numel() >= n and tok_pos.numel() >= n
+    _call("state_space", "nncpu_ssm_step", _ptr(proj), _i(proj.shape[1]), _ptr(conv_w), _i(_code(conv_w)), _ptr(conv_b),
+          _i(_code(conv_b)), _ptr(state), _l(state.shape[1]), _ptr(tok_pos), _ptr(seq_slots), _ptr(dt_bias), _ptr(a_log),
+          _ptr(d_skip), _i(_code(a_log)), _ptr(y), _i(n), _i(H), _i(P), _i(G), _i(N), _i(taps), _stream())
+
+
+def ssm_gated_norm(y, proj, weight, eps: float, out, n_groups: int) -> None:
+    """out = rms-norm in ``n_groups`` equal parts of (y * silu(z)), times ``weight``; z the first lanes of ``proj``'s rows."""
+    n, inner = y.shape
+    assert y.dtype == proj.dtype == torch.float32 and proj.shape[0] == n and proj.shape[1] >= inner and weight.numel() == inner
+    assert out.shape == y.shape and out.is_contiguous() and y.is_contiguous() and proj.is_contiguous()
+    _call("state_space", "nncpu_ssm_gated_norm", _ptr(y), _ptr(proj), _i(proj.shape[1]), _ptr(weight), _i(_code(weight)),
+          _f(eps), _ptr(out), _i(_code(out)), _i(n), _i(inner), _i(n_groups), _stream())
 
 
 def gather_rows(x, rows, out) -> None:

@@ -19,6 +19,13 @@ Further options: ``values_are_keys`` (no value projection: a position's value is
 rotation), ``sink`` (a learned logit per head whose exponential joins the softmax's denominator), ``out_gate`` (the
 concatenated heads times sigmoid(W_g h), lane by lane, before the output projection; W_g's rows ride in the q/k/v
 product) and ``out_bias``.
+
+``keep_first`` n (with a window): the sequence's first n keys stay visible to every query, at their true positions.
+``qk_norm_whole``: the norm of q and of k runs over all the heads' lanes at once, before the split.  A position part of kind
+"rope_pairs" turns neighbouring lanes (2i, 2i + 1).  A mixer with either of the last two has a kernel of its own before
+the attention (``ops.qk_whole_norm_append``), which lays a head of any size up to 128 lanes, and a value head of another
+size, into the 64 or 128 lanes that the tensor-core attention kernels read (zeros behind); a decode step has the same
+inside the attention kernel.
 """
 from __future__ import annotations
 
@@ -42,6 +49,14 @@ class Attention(Mixer):
         self.shared_kv = reads_other_cache
         if s.n_heads % s.n_kv_heads:
             raise UnsupportedModel(f"{s.name}: {s.n_heads} heads over {s.n_kv_heads} key/value heads")
+        if s.keep_first and not s.window:
+            raise UnsupportedModel(f"{s.name}: {s.keep_first} kept keys without a window")
+        self.pairs = s.position is not None and s.position.kind == "rope_pairs"
+        self.apart = s.qk_norm_whole or self.pairs       # norm, rotation and append by the kernel that knows these two
+        if self.apart and (s.values_are_keys or s.q_temp_coef != 0.0 or (s.qk_norm is not None and not s.qk_norm_whole)
+                           or (s.position is not None and not self.pairs)):
+            raise UnsupportedModel(f"{s.name}: a norm over whole rows or a rotation of neighbouring lanes does not go with a "
+                                   "norm per head, a half-split rotation, a query temperature or values that are the keys")
         if s.qk_norm is not None and s.qk_norm.kind != "rmsnorm":
             raise UnsupportedModel(f"{s.name}: per-head norm of kind {s.qk_norm.kind!r} is not supported")
         if s.tensor_names not in ("proj", "short"):
@@ -63,8 +78,9 @@ class Attention(Mixer):
         # its own and knows no rows of gate logits); a decode step has them inside the attention kernel that starts
         # from the projections.  A sink is a matter of the attention kernels alone, and all of them take it; the one
         # design that has sinks has the other two as well, so a sink keeps to their path.
-        self.plain_core = self.v_dim != s.head_dim
-        self.unfused = (self.plain_core or s.slope_base != 0.0 or s.q_temp_coef != 0.0 or s.values_are_keys or s.sink
+        self.plain_core = self.v_dim != s.head_dim and not self.apart
+        self.k_row, self.v_row = s.head_dim, self.v_dim         # lanes of a head in the pages (bind may lengthen them)
+        self.unfused = (self.plain_core or self.apart or s.slope_base != 0.0 or s.q_temp_coef != 0.0 or s.values_are_keys or s.sink
                         or s.out_gate)
         self.q_temp = (s.q_temp_coef, s.q_temp_every) if s.q_temp_coef != 0.0 else None
         self.position = None if s.position is None else base.build("position", s.position)
@@ -72,8 +88,9 @@ class Attention(Mixer):
 
     def kv_request(self):
         s = self.spec
-        return None if self.shared_kv else KVRequest(s.n_kv_heads, s.head_dim, s.window,
-                                                     0 if self.v_dim == s.head_dim else self.v_dim, chunk=s.chunk)
+        return None if self.shared_kv else KVRequest(s.n_kv_heads, self.k_row, s.window,
+                                                     0 if self.v_row == self.k_row else self.v_row, chunk=s.chunk,
+                                                     keep_first=s.keep_first)
 
     def _proj_names(self):
         if self.shared_kv:
@@ -104,9 +121,10 @@ class Attention(Mixer):
         if s.out_bias or s.out_bias_optional:
             p.append(ParamSpec(self._tensor("o_proj", bias=True), (s.hidden_size,), required=s.out_bias))
         if s.qk_norm is not None:
-            p.append(ParamSpec(self._norm_tensor("q"), (s.head_dim,), init=("one_plus_normal", 0.1)))
+            q_lanes, k_lanes = (self.q_size, self.kv_size) if s.qk_norm_whole else (s.head_dim, s.head_dim)
+            p.append(ParamSpec(self._norm_tensor("q"), (q_lanes,), init=("one_plus_normal", 0.1)))
             if not self.shared_kv:
-                p.append(ParamSpec(self._norm_tensor("k"), (s.head_dim,), init=("one_plus_normal", 0.1)))
+                p.append(ParamSpec(self._norm_tensor("k"), (k_lanes,), init=("one_plus_normal", 0.1)))
         if s.sink:
             p.append(ParamSpec(f"{s.name}.sink", (s.n_heads,), init=("normal", 1.0)))
         if s.out_gate:
@@ -115,6 +133,9 @@ class Attention(Mixer):
 
     def bind(self, tensors, rt):
         s, self.rt = self.spec, rt
+        if self.apart and rt.dtype == torch.bfloat16:
+            # rows of the sizes that the tensor-core attention kernels read; where they take none, the heads' own
+            self.k_row, self.v_row = ops.attention_rows(s.head_dim, self.v_dim) or (s.head_dim, self.v_dim)
         names = self._proj_names()
         ws = [tensors.pop(self._tensor(n)) for n in names]
         if s.out_gate:
@@ -178,14 +199,20 @@ class Attention(Mixer):
                                                       ctx.tok_pos, attn, scratch, s.n_heads, s.n_kv_heads, s.head_dim,
                                                       s.scale, self.span, n_splits, s.slope_base, self.q_temp,
                                                       sinks=self.sinks, values_are_keys=s.values_are_keys,
-                                                      gated=s.out_gate)
+                                                      gated=s.out_gate, keep=s.keep_first, v_head_dim=self.v_dim,
+                                                      whole_norm=s.qk_norm_whole, rot_pairs=self.pairs)
             else:
-                q = rt.empty(n, self.q_size)
+                q = rt.empty(n, s.n_heads * self.k_row)
+                n_kv = 0 if self.shared_kv else s.n_kv_heads
                 with rt.phase("attn_rope"):
-                    ops.qk_norm_rope_append(qkv, self.q_gamma, self.k_gamma, eps, cos_sin, ctx.tok_seq, ctx.tok_pos,
-                                            cache.block_table, cache.k_pages, cache.v_pages, q, s.n_heads,
-                                            0 if self.shared_kv else s.n_kv_heads, s.head_dim, self.v_dim, self.q_temp,
-                                            values_are_keys=s.values_are_keys)
+                    if self.apart:
+                        ops.qk_whole_norm_append(qkv, self.q_gamma, self.k_gamma, eps, cos_sin, ctx.tok_seq, ctx.tok_pos,
+                                                 cache.block_table, cache.k_pages, cache.v_pages, q, s.n_heads, n_kv,
+                                                 s.head_dim, self.v_dim)
+                    else:
+                        ops.qk_norm_rope_append(qkv, self.q_gamma, self.k_gamma, eps, cos_sin, ctx.tok_seq, ctx.tok_pos,
+                                                cache.block_table, cache.k_pages, cache.v_pages, q, s.n_heads, n_kv,
+                                                s.head_dim, self.v_dim, self.q_temp, values_are_keys=s.values_are_keys)
                 with self._core_phase(ctx, cache):
                     self._attend(ctx, q, cache, attn)
                 if s.out_gate:      # (the decode kernel that starts from the projections applies the gate itself)
@@ -202,7 +229,7 @@ class Attention(Mixer):
         if not perf.enabled():
             return perf._NULL
         s = self.spec
-        keys = ctx.span_sum(s.window, s.chunk)
+        keys = ctx.span_sum(s.window, s.chunk, s.keep_first)
         return self.rt.phase("attn_core", nbytes=1.0 * keys * s.n_kv_heads * (s.head_dim + self.v_dim) * cache.k_pages.element_size(),
                              flops=2.0 * keys * (self.q_size + self.out_size))
 
@@ -210,21 +237,27 @@ class Attention(Mixer):
         """Whether this step's attention can start from the float32 projections: a decode step on the tensor-core
         kernel, every lane of a head rotated (or none), norm weights of one type."""
         s = self.spec
-        return (not self.plain_core and ctx.is_decode and self.rt.dtype == torch.bfloat16 and cache.k_pages.dtype == torch.bfloat16
-                and ops.attention_mma_supported(s.n_heads, s.n_kv_heads, s.head_dim)
+        return (self._tensor_core_rows() and ctx.is_decode and self.rt.dtype == torch.bfloat16
+                and cache.k_pages.dtype == torch.bfloat16
                 and s.n_heads // s.n_kv_heads <= 16
-                and (self.position is None or self.position.half * 2 == s.head_dim)
+                and (self.position is None or self.pairs or self.position.half * 2 == s.head_dim)
                 and (self.q_gamma is None or self.k_gamma is None or self.q_gamma.dtype == self.k_gamma.dtype))
+
+    def _tensor_core_rows(self) -> bool:
+        """Whether the heads lie in rows that the tensor-core attention kernels read."""
+        s = self.spec
+        return (not self.plain_core and ops.attention_mma_supported(s.n_heads, s.n_kv_heads, self.k_row)
+                and self.v_row in (64, self.k_row))
 
     def _decode_splits(self, ctx):
         """Splits of every token's keys in a decode step, and the scratch their merge needs (None: they merge
         inside a thread-block cluster)."""
         s = self.spec
-        limit = s.window or s.chunk
+        limit = s.window + s.keep_first if s.window else s.chunk
         longest = min(ctx.max_kv_len, limit) if limit > 0 else ctx.max_kv_len
         n_splits = ops.attention_decode_splits(ctx.n_tokens, s.n_kv_heads, longest, self.rt.sm_count)
         floats = 0 if n_splits <= ops.DECODE_CLUSTER_MAX_SPLITS else ops.attention_decode_scratch_floats(
-            ctx.n_tokens, s.n_heads, s.n_kv_heads, s.head_dim, n_splits)
+            ctx.n_tokens, s.n_heads, s.n_kv_heads, self.v_row, n_splits)
         return n_splits, (self.rt.empty(floats, dtype=torch.float32) if floats else None)
 
     def _fused_qkv(self, x, cache) -> bool:
@@ -240,24 +273,24 @@ class Attention(Mixer):
         """bfloat16 with a head size the tensor-core kernels take: split-key
         decode, tcgen05 prefill for prompts, mma.sync prefill for a few tokens
         per sequence; everything else: the 32-bit kernel."""
-        s = self.spec
-        if (self.plain_core
-                or not ops.attention_mma_supported(s.n_heads, s.n_kv_heads, s.head_dim, q, cache.k_pages, attn)):
+        s, extra = self.spec, {"keep": self.spec.keep_first, "v_lanes": self.v_dim}
+        if not (self._tensor_core_rows() and ops.attention_mma_supported(s.n_heads, s.n_kv_heads, self.k_row, q, cache.k_pages, attn)):
             ops.attention(q, cache.k_pages, cache.v_pages, cache.block_table, ctx.tok_seq, ctx.tok_pos, attn,
-                          s.n_heads, s.n_kv_heads, s.head_dim, s.scale, self.span, self.v_dim, s.slope_base, self.sinks)
+                          s.n_heads, s.n_kv_heads, self.k_row, s.scale, self.span, self.v_row, s.slope_base, self.sinks,
+                          **extra)
         elif ctx.is_decode:
             n_splits, scratch = self._decode_splits(ctx)
             ops.attention_decode_mma(q, cache.k_pages, cache.v_pages, cache.block_table, ctx.tok_seq, ctx.tok_pos,
-                                     attn, scratch, s.n_heads, s.n_kv_heads, s.head_dim, s.scale, self.span, n_splits,
-                                     s.slope_base, self.sinks)
+                                     attn, scratch, s.n_heads, s.n_kv_heads, self.k_row, s.scale, self.span, n_splits,
+                                     s.slope_base, self.sinks, **extra)
         elif ctx.n_tokens >= 32 * ctx.n_seqs and ops.attention_prefill_tc_supported(
-                s.n_heads, s.n_kv_heads, s.head_dim, q, cache.k_pages, attn):
+                s.n_heads, s.n_kv_heads, self.k_row, q, cache.k_pages, attn):
             # prompts: 128-row tiles on the tcgen05 tensor cores
             ops.attention_prefill_tc(q, cache.k_pages, cache.v_pages, cache.block_table, ctx.cu_seqlens, ctx.tok_pos,
-                                     attn, self.rt.workspace.status, ctx.n_seqs, s.n_heads, s.n_kv_heads, s.head_dim,
-                                     s.scale, self.span, s.slope_base, self.sinks)
+                                     attn, self.rt.workspace.status, ctx.n_seqs, s.n_heads, s.n_kv_heads, self.k_row,
+                                     s.scale, self.span, s.slope_base, self.sinks, **extra)
         else:
             # a few new tokens per sequence: 64-row tiles
             ops.attention_prefill_mma(q, cache.k_pages, cache.v_pages, cache.block_table, ctx.cu_seqlens, ctx.tok_pos,
-                                      attn, ctx.n_seqs, s.n_heads, s.n_kv_heads, s.head_dim, s.scale, self.span,
-                                      s.slope_base, self.sinks)
+                                      attn, ctx.n_seqs, s.n_heads, s.n_kv_heads, self.k_row, s.scale, self.span,
+                                      s.slope_base, self.sinks, **extra)

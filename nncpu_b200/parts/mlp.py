@@ -14,7 +14,7 @@ import torch
 from ..errors import UnsupportedModel
 from ..kernels import ops
 from ..weights.params import ParamSpec
-from .base import DeferredNorm, FeedForward, register_feed_forward
+from .base import DeferredNorm, FeedForward, norm_output_buffer, register_feed_forward
 
 
 GATED_ACTIVATIONS = ("silu", "gelu_tanh", "swish_clamp")
@@ -100,6 +100,11 @@ class RoutedExperts(FeedForward):
 
     ``scores`` "all" (see ``RoutedExpertsSpec``): the softmax runs over all experts, the choice may be limited to the
     best groups of experts, and the chosen scores are divided by their sum and multiplied by ``weight_scale``.
+    ``scores`` "sigmoid": the largest logits are chosen and weighted by their sigmoids as they are.  ``weight_on`` "input":
+    a weight multiplies its expert's input.  ``shared_gate``: the shared feed-forward's output is multiplied by the
+    sigmoid of one more product with the input; its row rides with the router's.  In the grouped form the shared part is a
+    branch that the sum over a token's experts takes in, and that kernel, which holds the stream's new rows, leaves the norm
+    that reads the stream next; in the form for few tokens the shared part runs in the experts' own two launches.
     ``out_scale`` (and the step's ``ctx.out_scale``) multiply what the part adds to the stream: they enter the
     tokens' weights, so the sum over a token's experts is scaled at no cost."""
     scales_output = True
@@ -109,16 +114,22 @@ class RoutedExperts(FeedForward):
             raise UnsupportedModel(f"{spec.name}: activation {spec.activation!r} is not supported")
         if not 0 < spec.top <= spec.n_experts:
             raise UnsupportedModel(f"{spec.name}: the top {spec.top} of {spec.n_experts} experts")
-        if spec.scores not in ("chosen", "all"):
-            raise UnsupportedModel(f"{spec.name}: router scores of kind {spec.scores!r}")
-        if spec.scores == "chosen" and (spec.n_groups > 1 or spec.weight_scale != 1.0 or spec.out_scale != 1.0):
+        if spec.scores not in ("chosen", "all", "sigmoid") or spec.weight_on not in ("output", "input"):
+            raise UnsupportedModel(f"{spec.name}: router scores of kind {spec.scores!r} on the {spec.weight_on!r}")
+        if spec.scores != "all" and (spec.n_groups > 1 or spec.weight_scale != 1.0 or spec.out_scale != 1.0):
             raise UnsupportedModel(f"{spec.name}: groups and scales go with scores over all experts")
         if spec.n_groups > 1 and (spec.n_experts % spec.n_groups or not 1 <= spec.keep_groups <= spec.n_groups
                                   or spec.keep_groups * (spec.n_experts // spec.n_groups) < spec.top):
             raise UnsupportedModel(f"{spec.name}: the {spec.keep_groups} best of {spec.n_groups} groups of "
                                    f"{spec.n_experts} experts cannot give the top {spec.top}")
+        if spec.shared_gate and (spec.shared is None or spec.router_bias):
+            raise UnsupportedModel(f"{spec.name}: a gate goes with a shared feed-forward and a router without a bias")
         self.spec = spec
         self.shared = None if spec.shared is None else GatedMlp(spec.shared)
+        # a shared feed-forward with a gate is part of this part's own launches; one without runs by itself
+        self.own_shared = spec.shared_gate
+        if self.own_shared and spec.shared.activation != spec.activation:
+            raise UnsupportedModel(f"{spec.name}: a gated shared feed-forward has the experts' activation")
 
     def params(self):
         s, p = self.spec, []
@@ -129,6 +140,8 @@ class RoutedExperts(FeedForward):
         p.append(ParamSpec(f"{s.name}.router", (s.n_experts, s.hidden_size), init=("normal", 0.5)))
         if s.router_bias:
             p.append(ParamSpec(f"{s.name}.router.b", (s.n_experts,), init=("normal", 0.5)))
+        if s.shared_gate:
+            p.append(ParamSpec(f"{s.shared.name}.sg", (1, s.hidden_size), init=("normal", 0.5)))
         return p + (self.shared.params() if self.shared is not None else [])
 
     def bind(self, tensors, rt):
@@ -150,6 +163,8 @@ class RoutedExperts(FeedForward):
             self.w_gate, self.w_up = gate, up
         del gate, up
         self.w_router, self.b_router = tensors[f"{s.name}.router"], tensors.get(f"{s.name}.router.b")
+        if s.shared_gate:
+            self.w_router = torch.cat([self.w_router, tensors.pop(f"{s.shared.name}.sg")], dim=0).contiguous()
         if self.shared is not None:
             self.shared.bind(tensors, rt)
 
@@ -171,27 +186,33 @@ class RoutedExperts(FeedForward):
         weights = rt.empty(n, s.top, dtype=torch.float32)
         out_scale = float(getattr(ctx, "out_scale", 1.0)) * s.out_scale
         scoring = None
+        gate = rt.empty(n, dtype=torch.float32) if s.shared_gate else None
         if s.scores == "all":
             scoring = ("all", s.n_groups, s.keep_groups, s.weight_scale * out_scale)
+        elif s.scores == "sigmoid" and out_scale == 1.0:
+            scoring = ("sigmoid",)
         elif out_scale != 1.0:
             raise UnsupportedModel(f"{s.name}: a scaled output goes with scores over all experts")
         with rt.phase("moe_route", self.w_router, n):
             many = n >= ROUTER_PRODUCT_FROM_TOKENS and rt.tensor_cores_take(x.dtype, self.w_router, s.hidden_size)
             if not many and ops.moe_router_fits(s.n_experts, s.hidden_size):
-                ops.moe_router(x, self.w_router, self.b_router, s.top, ids, weights, scoring)
+                ops.moe_router(x, self.w_router, self.b_router, s.top, ids, weights, scoring, gate)
             else:
                 # many tokens: the logits as a product of their own (bfloat16 operands are multiplied exactly and
                 # added in 32-bit on the tensor cores; a float32 run, and sizes those refuse, use the CUDA cores)
-                logits = rt.empty(n, s.n_experts, dtype=torch.float32)
+                logits = rt.empty(n, self.w_router.shape[0], dtype=torch.float32)
                 if many:
                     rt.linear(x, self.w_router, self.b_router, logits)
                 else:
                     ops.linear_simt(x, self.w_router, self.b_router, logits)
-                ops.moe_route(logits, s.top, ids, weights, scoring)
+                ops.moe_route(logits, s.top, ids, weights, scoring, gate)
         S, f, h = n * s.top, s.intermediate_size, s.hidden_size
         esize = self.w_gate.element_size()
         experts_read = min(S, s.n_experts)
-        if self.grouped and S >= GROUPED_FROM_SLOTS:
+        on_input = s.weight_on == "input"
+        then = getattr(ctx, "next_norm", None)
+        own = self.own_shared
+        if self.grouped and S >= GROUPED_FROM_SLOTS and not (own and not ops.moe_combine_closes(h)):
             # many tokens: sorted by expert, one grouped product each for gate/up (activation in its epilogue) and
             # down on the tensor cores, then the choices of a token added up in their order
             act = (s.activation, float(s.limit), 0.0) if s.activation != "silu" else None
@@ -200,20 +221,43 @@ class RoutedExperts(FeedForward):
                 plan = rt.empty(1 + 3 * ops.moe_plan_tiles(S, s.n_experts), dtype=torch.int32)
                 ops.moe_plan(ids, s.n_experts, rows, slots, plan)
                 xs = rt.empty(S, h, dtype=torch.bfloat16)
-                ops.moe_gather(x, slots, s.top, xs)
+                ops.moe_gather(x, slots, s.top, xs, weights if on_input else None)
             mid = rt.empty(S, f, dtype=torch.bfloat16)
             with rt.phase("moe_gate_up", nbytes=experts_read * 2.0 * f * h * esize, flops=4.0 * S * f * h):
                 ops.linear_tc_grouped(xs, self.w_gate, mid, plan, s.n_experts, rt.workspace, "swiglu", act)
             y = rt.empty(S, h, dtype=torch.float32)
             with rt.phase("moe_down", nbytes=experts_read * 1.0 * f * h * esize + 4.0 * S * h, flops=2.0 * S * f * h):
                 ops.linear_tc_grouped(mid, self.w_down, y, plan, s.n_experts, rt.workspace)
-            with rt.phase("moe_combine", nbytes=4.0 * S * h + 8.0 * n * h):
-                ops.moe_combine(y, rows, weights, residual)
+            branch = closing = None
+            if own:
+                # the shared part in a branch of its own; the sum over a token's experts takes it in, times the gate
+                branch = rt.empty(n, h, dtype=torch.float32)
+                ctx.branch_is_fresh, ctx.next_norm = True, None
+                try:
+                    self.shared.forward(ctx, x, branch)
+                finally:
+                    ctx.branch_is_fresh, ctx.next_norm = False, then
+            if (self.shared is None or own) and then is not None and then.residual is residual \
+                    and hasattr(then.norm, "closing_rms") and ops.moe_combine_closes(h):
+                then.output = norm_output_buffer(ctx, rt, residual.shape)
+                closing = then.norm.closing_rms(then.output)
+            with rt.phase("moe_combine", nbytes=4.0 * S * h + (12.0 if own else 8.0) * n * h + (2.0 * n * h if closing else 0.0)):
+                ops.moe_combine(y, rows, None if on_input else weights, residual, s.top, branch, gate, closing)
+        elif own:
+            # few tokens: the shared feed-forward's rows in the experts' two launches
+            sh = self.shared
+            mid, sh_mid = rt.empty(S, f), rt.empty(n, sh.spec.intermediate_size)
+            sg, su = (sh.w_gate_up, None) if sh.fused else sh.w_gate_up.chunk(2, dim=0)
+            with rt.phase("moe_experts", nbytes=experts_read * 3.0 * f * h * esize + sh.weight_bytes(),
+                          flops=6.0 * S * f * h + 6.0 * n * h * sh.spec.intermediate_size):
+                ops.moe_experts(x, self.w_gate, self.w_up, self.w_down, ids, weights, mid, residual, s.activation, s.limit,
+                                on_input, (sg, su, sh.w_down, sh_mid, gate))
         else:
             mid = rt.empty(S, f)
             with rt.phase("moe_experts", nbytes=experts_read * 3.0 * f * h * esize, flops=6.0 * S * f * h):
-                ops.moe_experts(x, self.w_gate, self.w_up, self.w_down, ids, weights, mid, residual, s.activation, s.limit)
-        if self.shared is not None:
+                ops.moe_experts(x, self.w_gate, self.w_up, self.w_down, ids, weights, mid, residual, s.activation, s.limit,
+                                on_input)
+        if self.shared is not None and not own:
             if out_scale != 1.0:
                 raise UnsupportedModel(f"{s.name}: a shared expert under a scaled output")
             self.shared.forward(ctx, x, residual)

@@ -24,6 +24,8 @@ class RMSNorm(Norm):
     def bind(self, tensors, rt):
         self.rt = rt
         self.gamma = tensors[self.tensor]
+        # what a product that carries this norm multiplies with: the weight with its offset, in 32-bit
+        self.carried_gamma = self.gamma if self.offset == 0.0 else self.gamma.to(torch.float32) + self.offset
 
     def forward(self, ctx, residual, rows=None):
         n = residual.shape[0] if rows is None else rows.numel()
@@ -40,11 +42,15 @@ class RMSNorm(Norm):
     def request(self, ctx, residual):
         """In a bfloat16 run the products around this norm can carry it: the few-token products at up to 16
         tokens, the tensor-core products of whole prompts (a launch, and at many tokens a pass over the residual
-        stream, less)."""
-        if (self.offset != 0.0 or self.rt.dtype != torch.bfloat16 or self.size % 16 or residual.dtype != torch.float32
-                or not self.rt.fuses_norms(ctx.n_tokens, self.size)):
+        stream, less).  At any number of tokens a kernel that closes a sublayer and holds the stream's new rows can leave
+        the finished output (``closing_rms``)."""
+        if self.rt.dtype != torch.bfloat16 or self.size % 16 or residual.dtype != torch.float32:
             return None
-        return NormRequest(self, residual, self.gamma, self.eps, self.size)
+        return NormRequest(self, residual, self.carried_gamma, self.eps, self.size)
+
+    def closing_rms(self, out):
+        """What ``ops.moe_combine`` takes as ``then_norm`` to leave this norm's output in ``out``."""
+        return (self.gamma, self.offset, self.eps, out)
 
 
 @register_norm("layernorm")

@@ -8,7 +8,7 @@ the cosines and sines of a step's positions are computed once per step in
 
 "rope_pairs" has the same table; its mixers turn the neighbouring lanes (2i, 2i + 1) by entry i instead.  Both take
 frequencies rescaled between two wavelengths (``PositionSpec.scaling_*``): the rescaled frequencies replace the plain
-ones when the weights are bound, and cos and sin are multiplied by one more number when the table is made.
+ones when the weights are bound, and (kind "ramp") cos and sin are multiplied by one more number when the table is made.
 """
 from __future__ import annotations
 
@@ -32,6 +32,8 @@ class RopeNeox(PositionEncoding):
     def __init__(self, spec):
         if spec.rotary_dim % 2 or spec.rotary_dim <= 0:
             raise BadFormat(f"rotary size {spec.rotary_dim} must be even and positive")
+        if spec.scaling_kind not in ("ramp", "bands"):
+            raise BadFormat(f"frequencies rescaled by {spec.scaling_kind!r}")
         self.spec = spec
         self.half = spec.rotary_dim // 2
         self.inv_freq = None
@@ -42,7 +44,15 @@ class RopeNeox(PositionEncoding):
         i = torch.arange(self.half, dtype=torch.float64)
         inv = torch.pow(torch.tensor(float(s.theta), dtype=torch.float64), -2.0 * i / s.rotary_dim)
         self.stretch = 1.0
-        if s.scaling_factor > 0.0:
+        if s.scaling_factor > 0.0 and s.scaling_kind == "bands":
+            # slow pairs (long wavelengths) turn `factor` times slower, fast ones as they are, a blend between
+            wave = 2.0 * math.pi / inv
+            width = s.scaling_fast - s.scaling_slow
+            mix = torch.clamp((s.scaling_original / wave - s.scaling_slow) / (width if width != 0.0 else 1.0), 0.0, 1.0)
+            slowed = inv / s.scaling_factor
+            inv = torch.where(wave < s.scaling_original / s.scaling_fast, inv,
+                              torch.where(wave > s.scaling_original / s.scaling_slow, slowed, (1.0 - mix) * slowed + mix * inv))
+        elif s.scaling_factor > 0.0:
             # pairs whose wavelength lies between the two limits are blended towards a frequency `factor` times lower
             def pair_of(turns: float) -> float:
                 return s.rotary_dim * math.log(s.scaling_original / (2.0 * math.pi * turns)) / (2.0 * math.log(s.theta))
