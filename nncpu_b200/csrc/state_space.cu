@@ -268,6 +268,350 @@ scan_kernel(const float* __restrict__ proj, const Sizes z, const void* __restric
 }
 
 // ---------------------------------------------------------------------------
+// Prompts of a bfloat16 run: the recurrence over chunks of 64 tokens, as products on the tensor cores (mma.sync).  With
+// cum_i the sum of la over the chunk's tokens up to i, S the state before the chunk and a = exp(cum_last):
+//     y_i   = sum over j <= i of (C_i . B_j) exp(cum_i - cum_j) dt_j x_j   +   exp(cum_i) S^T C_i   +   D x_i
+//     S_new = a S + sum over j of B_j (exp(cum_last - cum_j) dt_j x_j)^T
+// x, B and C are bfloat16 as the convolutions left them.  What is 32-bit by design stays so: the state lives in 32-bit
+// registers, decays and step sizes are 32-bit, and wherever one of them becomes an operand of a product (the masked
+// weights, the scaled x, the state that is read out) it goes in as the sum of two bfloat16 numbers, value and remainder,
+// so that a factor keeps 16 bits of mantissa and the products add up in 32-bit.
+//
+// A block of four warps owns 32 columns of one head's state for one sequence and walks its chunks in order: warp w has the
+// chunk's tokens 16 w .. 16 w + 15 as rows of y and a quarter of the state's rows in registers.  B, C and x of the next
+// chunk are copied to shared memory (cp.async, two buffers) under this chunk's arithmetic; the state goes through shared
+// memory once a chunk, so that every warp can read all of it.  What a token gets does not depend on other sequences;
+// where a sequence is cut moves the chunks' borders, which changes rounding only.
+// ---------------------------------------------------------------------------
+constexpr int kChunk = 64, kChunkCols = 32;
+
+__device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+// 16 bytes, or zeros where there is nothing to copy
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool in) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(in ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+__device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile(
+        "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+        : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+        : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// Two numbers as bfloat16 pairs: the values, and what rounding them left.
+__device__ __forceinline__ void split_pair(float a, float b, uint32_t& hi, uint32_t& lo) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+    const float2 f = __bfloat1622float2(h);
+    const __nv_bfloat162 l = __floats2bfloat162_rn(a - f.x, b - f.y);
+    hi = *reinterpret_cast<const uint32_t*>(&h);
+    lo = *reinterpret_cast<const uint32_t*>(&l);
+}
+
+// Byte offsets of 16-byte pieces in tiles whose rows hold NP (a multiple of 64) or 32 bfloat16, exchanged by the row number
+// so that 8 rows' equal pieces lie in 8 bank groups.
+template <int NP>
+__device__ __forceinline__ uint32_t wide_off(int row, int piece) {
+    return (uint32_t)(row * (NP * 2) + (((piece & ~7) | ((piece ^ row) & 7)) << 4));
+}
+__device__ __forceinline__ uint32_t narrow_off(int row, int piece) { return (uint32_t)(row * 64 + ((piece ^ ((row >> 1) & 3)) << 4)); }
+
+template <int NP>
+constexpr int chunk_smem() { return 4 * kChunk * NP * 2 + 4 * kChunk * 64 + 2 * NP * 64; }
+
+template <int NP>
+__global__ void __launch_bounds__(128)
+chunk_kernel(const float* __restrict__ proj, const Sizes z, const __nv_bfloat16* __restrict__ xc, const float* __restrict__ gd,
+             float* state, const int* __restrict__ seq_slots, const int* __restrict__ cu_seqlens, const int* __restrict__ tok_pos,
+             const void* __restrict__ d_skip, int p_dt, float* __restrict__ y) {
+    constexpr int kWide = kChunk * NP * 2, kNarrow = kChunk * 64;      // bytes of a tile of B or C, of x
+    constexpr int MT = NP / 64;                                        // 16-row tiles of the state a warp holds
+    extern __shared__ __align__(128) uint8_t chunk_smem_[];
+    __shared__ float2 cum_dt[kChunk];
+    const uint32_t base = smem_addr(chunk_smem_);
+    const uint32_t b_tile = base, c_tile = base + 2 * kWide, x_tile = base + 4 * kWide;      // two buffers each
+    const uint32_t xh_tile = x_tile + 2 * kNarrow, xl_tile = xh_tile + kNarrow;              // the scaled x, value and remainder
+    const uint32_t sh_tile = xl_tile + kNarrow, sl_tile = sh_tile + NP * 64;                 // the state, value and remainder
+    const int seq = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * kChunkCols;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, c = lane & 3, r = lane >> 2;
+    const int t0 = cu_seqlens[seq], t1 = cu_seqlens[seq + 1], slot = seq_slots[seq];
+    if (t0 >= t1) return;
+    const int inner = z.inner();
+    float* y_head = y + (size_t)h * z.P + col0;
+    if (slot < 0) {
+        for (int i = tid; i < (t1 - t0) * kChunkCols; i += 128)
+            if (col0 + i % kChunkCols < z.P) y_head[(size_t)(t0 + i / kChunkCols) * inner + i % kChunkCols] = 0.0f;
+        return;
+    }
+    const int row = z.row(), g = h / (z.H / z.G);
+    const size_t x_at = (size_t)h * z.P8 + col0, b_at = (size_t)z.H * z.P8 + (size_t)g * z.N8, c_at = b_at + (size_t)z.G * z.N8;
+    float* s_head = state + (size_t)slot * z.slot_stride + (size_t)h * z.N * z.P + col0;
+    const float skip = ld_f(d_skip, h, p_dt);
+    const int cols = min(kChunkCols, z.P - col0);
+
+    auto stage = [&](int g0, int buf) {
+        const int nt = t1 - g0;                                        // (may be more than a chunk, or none)
+        for (int i = tid; i < kChunk * (NP / 8); i += 128) {
+            const int tt = i / (NP / 8), piece = i % (NP / 8);
+            const bool in = tt < nt && piece * 8 < z.N8;
+            const __nv_bfloat16* src = xc + (in ? (size_t)(g0 + tt) * row + piece * 8 : 0);
+            cp_async16(b_tile + buf * kWide + wide_off<NP>(tt, piece), in ? src + b_at : xc, in);
+            cp_async16(c_tile + buf * kWide + wide_off<NP>(tt, piece), in ? src + c_at : xc, in);
+        }
+        for (int i = tid; i < kChunk * 4; i += 128) {
+            const int tt = i >> 2, piece = i & 3;
+            const bool in = tt < nt && col0 + piece * 8 < z.P8;
+            cp_async16(x_tile + buf * kNarrow + narrow_off(tt, piece), in ? xc + (size_t)(g0 + tt) * row + x_at + piece * 8 : xc, in);
+        }
+    };
+    stage(t0, 0);
+    cp_async_commit();
+    stage(t0 + kChunk, 1);
+    cp_async_commit();
+
+    // this warp's rows of the state: m0 + 16 mt + r (and + 8), columns 8 nt + 2 c (and + 1)
+    const int m0 = warp * (NP / 4);
+    float S[MT][4][4];
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+        for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int i = m0 + 16 * mt + r + 8 * (e >> 1), col = 8 * nt + 2 * c + (e & 1);
+                S[mt][nt][e] = (i < z.N && col < cols) ? s_head[(size_t)i * z.P + col] : 0.0f;
+            }
+    auto publish = [&]() {
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+            for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+                for (int half = 0; half < 2; ++half) {
+                    uint32_t hi, lo;
+                    split_pair(S[mt][nt][2 * half], S[mt][nt][2 * half + 1], hi, lo);
+                    const uint32_t at = narrow_off(m0 + 16 * mt + r + 8 * half, nt) + 4 * c;
+                    asm volatile("st.shared.b32 [%0], %1;" ::"r"(sh_tile + at), "r"(hi) : "memory");
+                    asm volatile("st.shared.b32 [%0], %1;" ::"r"(sl_tile + at), "r"(lo) : "memory");
+                }
+    };
+    publish();
+
+    // la and dt of the tokens 2 lane and 2 lane + 1 of a chunk, fetched one chunk ahead
+    float la0, la1, dt0, dt1;
+    auto fetch = [&](int g0) {
+        const float* p = gd + (size_t)(g0 + 2 * lane) * 2 * z.H + h;
+        const bool in0 = g0 + 2 * lane < t1, in1 = g0 + 2 * lane + 1 < t1;
+        la0 = in0 ? p[0] : 0.0f;
+        dt0 = in0 ? p[z.H] : 0.0f;
+        la1 = in1 ? p[2 * z.H] : 0.0f;
+        dt1 = in1 ? p[3 * z.H] : 0.0f;
+    };
+    fetch(t0);
+    int buf = 0;
+    for (int g0 = t0; g0 < t1; g0 += kChunk, buf ^= 1) {
+        // sums of la up to every token (tokens beyond the sequence's end add nothing)
+        float cum1 = la0 + la1;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float got = __shfl_up_sync(0xffffffffu, cum1, o);
+            if (lane >= o) cum1 += got;
+        }
+        float before = __shfl_up_sync(0xffffffffu, cum1, 1);
+        if (lane == 0) before = 0.0f;
+        const float cum0 = before + la0;
+        const float cum_last = __shfl_sync(0xffffffffu, cum1, 31);
+        const float dt_0 = dt0, dt_1 = dt1;
+        if (g0 + kChunk < t1) fetch(g0 + kChunk);
+        cp_async_wait<1>();                      // this chunk's tiles have landed (the next one's may still fly)
+        __syncthreads();                         // everybody's have; the state of the chunk before is published
+        if (warp == 0) {
+            cum_dt[2 * lane] = make_float2(cum0, dt_0);
+            cum_dt[2 * lane + 1] = make_float2(cum1, dt_1);
+        }
+        {   // x scaled by what is left of a token at the chunk's end: a thread has half of one token's columns
+            const int src = 8 * warp + (lane >> 2);
+            const bool odd = (lane >> 1) & 1;
+            const float cu = __shfl_sync(0xffffffffu, cum0, src), cv = __shfl_sync(0xffffffffu, cum1, src);
+            const float du = __shfl_sync(0xffffffffu, dt_0, src), dv = __shfl_sync(0xffffffffu, dt_1, src);
+            const float scale = expf(cum_last - (odd ? cv : cu)) * (odd ? dv : du);
+            const int tt = tid >> 1;
+#pragma unroll
+            for (int k = 0; k < 2; ++k) {
+                const uint32_t at = narrow_off(tt, 2 * (tid & 1) + k);
+                uint32_t v[4], hi[4], lo[4];
+                asm volatile("ld.shared.v4.b32 {%0, %1, %2, %3}, [%4];"
+                             : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]) : "r"(x_tile + buf * kNarrow + at));
+#pragma unroll
+                for (int q = 0; q < 4; ++q) {
+                    const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v[q]));
+                    split_pair(f.x * scale, f.y * scale, hi[q], lo[q]);
+                }
+                asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(xh_tile + at), "r"(hi[0]), "r"(hi[1]), "r"(hi[2]), "r"(hi[3]) : "memory");
+                asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(xl_tile + at), "r"(lo[0]), "r"(lo[1]), "r"(lo[2]), "r"(lo[3]) : "memory");
+            }
+        }
+        __syncthreads();
+        // C . B^T (token pairs of this warp's rows, only up to the diagonal) and C . S
+        float s[8][4], acc[4][4];
+#pragma unroll
+        for (int t = 0; t < 8; ++t) s[t][0] = s[t][1] = s[t][2] = s[t][3] = 0.0f;
+#pragma unroll
+        for (int t = 0; t < 4; ++t) acc[t][0] = acc[t][1] = acc[t][2] = acc[t][3] = 0.0f;
+        const uint32_t bt = b_tile + buf * kWide, ct = c_tile + buf * kWide, xt = x_tile + buf * kNarrow;
+#pragma unroll 2
+        for (int ks = 0; ks < NP / 16; ++ks) {
+            if (ks * 16 >= z.N) break;
+            uint32_t a[4], b[4];
+            ldmatrix_x4(a, ct + wide_off<NP>(16 * warp + ((lane >> 3) & 1) * 8 + (lane & 7), ks * 2 + (lane >> 4)));
+#pragma unroll
+            for (int tp = 0; tp < 4; ++tp) {
+                if (tp <= warp) {
+                    ldmatrix_x4(b, bt + wide_off<NP>(tp * 16 + (lane >> 4) * 8 + (lane & 7), ks * 2 + ((lane >> 3) & 1)));
+                    mma_bf16(s[2 * tp], a, b[0], b[1]);
+                    mma_bf16(s[2 * tp + 1], a, b[2], b[3]);
+                }
+            }
+            const int k_row = ks * 16 + ((lane >> 3) & 1) * 8 + (lane & 7);
+#pragma unroll
+            for (int dp = 0; dp < 2; ++dp) {
+                const uint32_t at = narrow_off(k_row, dp * 2 + (lane >> 4));
+                ldmatrix_x4_trans(b, sh_tile + at);
+                mma_bf16(acc[2 * dp], a, b[0], b[1]);
+                mma_bf16(acc[2 * dp + 1], a, b[2], b[3]);
+                ldmatrix_x4_trans(b, sl_tile + at);
+                mma_bf16(acc[2 * dp], a, b[0], b[1]);
+                mma_bf16(acc[2 * dp + 1], a, b[2], b[3]);
+            }
+        }
+        const int i_lo = 16 * warp + r, i_hi = i_lo + 8;
+        const float cum_lo = cum_dt[i_lo].x, cum_hi = cum_dt[i_hi].x;
+        const float e_lo = expf(cum_lo), e_hi = expf(cum_hi);
+#pragma unroll
+        for (int t = 0; t < 4; ++t) {
+            acc[t][0] *= e_lo; acc[t][1] *= e_lo; acc[t][2] *= e_hi; acc[t][3] *= e_hi;
+        }
+        // the weights of the chunk's own tokens, and their sum of x
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk) {
+            if (kk <= warp) {
+                uint32_t hi[4], lo[4];
+#pragma unroll
+                for (int half = 0; half < 2; ++half) {
+                    const int t = 2 * kk + half, j = t * 8 + 2 * c;
+                    const float4 cd = *reinterpret_cast<const float4*>(&cum_dt[j]);      // (cum, dt) of the tokens j and j + 1
+                    const float w0 = j <= i_lo ? s[t][0] * (expf(cum_lo - cd.x) * cd.y) : 0.0f;
+                    const float w1 = j + 1 <= i_lo ? s[t][1] * (expf(cum_lo - cd.z) * cd.w) : 0.0f;
+                    const float w2 = j <= i_hi ? s[t][2] * (expf(cum_hi - cd.x) * cd.y) : 0.0f;
+                    const float w3 = j + 1 <= i_hi ? s[t][3] * (expf(cum_hi - cd.z) * cd.w) : 0.0f;
+                    split_pair(w0, w1, hi[2 * half], lo[2 * half]);
+                    split_pair(w2, w3, hi[2 * half + 1], lo[2 * half + 1]);
+                }
+#pragma unroll
+                for (int dp = 0; dp < 2; ++dp) {
+                    uint32_t b[4];
+                    ldmatrix_x4_trans(b, xt + narrow_off(kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), dp * 2 + (lane >> 4)));
+                    mma_bf16(acc[2 * dp], hi, b[0], b[1]);
+                    mma_bf16(acc[2 * dp + 1], hi, b[2], b[3]);
+                    mma_bf16(acc[2 * dp], lo, b[0], b[1]);
+                    mma_bf16(acc[2 * dp + 1], lo, b[2], b[3]);
+                }
+            }
+        }
+        // y, with the token's own x
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+            const int i = half ? i_hi : i_lo;
+            if (g0 + i >= t1) continue;
+            float* dst = y_head + (size_t)(g0 + i) * inner;
+#pragma unroll
+            for (int t = 0; t < 4; ++t) {
+                const int col = 8 * t + 2 * c;
+                uint32_t v;
+                asm volatile("ld.shared.b32 %0, [%1];" : "=r"(v) : "r"(xt + narrow_off(i, t) + 4 * c));
+                const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v));
+                const float o0 = fmaf(skip, f.x, acc[t][2 * half]), o1 = fmaf(skip, f.y, acc[t][2 * half + 1]);
+                if (col + 1 < cols && (z.P & 1) == 0) *reinterpret_cast<float2*>(dst + col) = make_float2(o0, o1);
+                else {
+                    if (col < cols) dst[col] = o0;
+                    if (col + 1 < cols) dst[col + 1] = o1;
+                }
+            }
+        }
+        // the state after the chunk
+        const float a_all = expf(cum_last);
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+            for (int t = 0; t < 4; ++t)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) S[mt][t][e] *= a_all;
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk) {
+            uint32_t bh[2][4], bl[2][4];
+#pragma unroll
+            for (int dp = 0; dp < 2; ++dp) {
+                const uint32_t at = narrow_off(kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), dp * 2 + (lane >> 4));
+                ldmatrix_x4_trans(bh[dp], xh_tile + at);
+                ldmatrix_x4_trans(bl[dp], xl_tile + at);
+            }
+#pragma unroll
+            for (int mt = 0; mt < MT; ++mt) {
+                uint32_t a[4];
+                ldmatrix_x4_trans(a, bt + wide_off<NP>(kk * 16 + (lane >> 4) * 8 + (lane & 7), (m0 + 16 * mt) / 8 + ((lane >> 3) & 1)));
+#pragma unroll
+                for (int dp = 0; dp < 2; ++dp) {
+                    mma_bf16(S[mt][2 * dp], a, bh[dp][0], bh[dp][1]);
+                    mma_bf16(S[mt][2 * dp + 1], a, bh[dp][2], bh[dp][3]);
+                    mma_bf16(S[mt][2 * dp], a, bl[dp][0], bl[dp][1]);
+                    mma_bf16(S[mt][2 * dp + 1], a, bl[dp][2], bl[dp][3]);
+                }
+            }
+        }
+        __syncthreads();                         // the old state and this chunk's tiles are done with
+        publish();
+        if (g0 + 2 * kChunk < t1) stage(g0 + 2 * kChunk, buf);
+        cp_async_commit();
+    }
+    cp_async_wait<0>();
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+        for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int i = m0 + 16 * mt + r + 8 * (e >> 1), col = 8 * nt + 2 * c + (e & 1);
+                if (i < z.N && col < cols) s_head[(size_t)i * z.P + col] = S[mt][nt][e];
+            }
+    float* ring = state + (size_t)slot * z.slot_stride + z.conv_at;
+    const int pos0 = tok_pos[t0];
+    own_channels(z, h, col0, kChunkCols, blockIdx.z == 0, [&](int ch) { advance_ring(proj, z, ring, t0, t1, pos0, ch); });
+}
+
+template <int NP>
+int launch_chunk(const float* proj, const Sizes& z, const void* xc, const float* gd, float* state, const int* seq_slots,
+                 const int* cu_seqlens, const int* tok_pos, const void* d_skip, int p_dt, float* y, int n_seqs, cudaStream_t st) {
+    static bool configured[64] = {};
+    if (first_use_on_this_device(configured)) {
+        const cudaError_t e = cudaFuncSetAttribute(chunk_kernel<NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, chunk_smem<NP>());
+        NN_CHECK(e == cudaSuccess, "state space (chunks): cannot reserve shared memory: %s", cudaGetErrorString(e));
+    }
+    const dim3 grid(n_seqs, z.H, (z.P + kChunkCols - 1) / kChunkCols);
+    chunk_kernel<NP><<<grid, 128, chunk_smem<NP>(), st>>>(proj, z, (const __nv_bfloat16*)xc, gd, state, seq_slots, cu_seqlens, tok_pos,
+                                                          d_skip, p_dt, y);
+    NN_LAUNCH_OK("state space (chunks)");
+    return 0;
+}
+
+// ---------------------------------------------------------------------------
 // A decode step: one token per sequence, everything from the projections to y in one launch.  A block owns kStepCols
 // columns of one (token, head); its threads are groups of VEC neighbouring columns times row groups, so the state is read
 // and written at full width with all of a thread's rows in flight.  The convolutions of the head's x and of its group's B
@@ -476,6 +820,21 @@ extern "C" int nncpu_ssm_scan(const float* proj, int ld, const void* xc, int xc_
 #undef NN_SCAN
     NN_LAUNCH_OK("state space (scan)");
     return 0;
+}
+
+extern "C" int nncpu_ssm_chunk_scan(const float* proj, int ld, const void* xc, const float* gd, float* state, long slot_stride,
+                                    const int* seq_slots, const int* cu_seqlens, const int* tok_pos, const void* d_skip,
+                                    int p_dt, float* y, int n_seqs, int H, int P, int G, int N, int taps, void* stream) {
+    // xc is bfloat16
+    Sizes z;
+    if (int e = make_sizes(&z, H, P, G, N, taps, ld, slot_stride)) return e;
+    NN_CHECK(N <= 256, "state space (chunks): states of %d rows (at most 256)", N);
+    NN_CHECK((uintptr_t)xc % 16 == 0 && (uintptr_t)y % 8 == 0, "state space (chunks): rows must be 16-byte aligned");
+    if (n_seqs <= 0) return 0;
+    cudaStream_t st = (cudaStream_t)stream;
+    if (N <= 64) return launch_chunk<64>(proj, z, xc, gd, state, seq_slots, cu_seqlens, tok_pos, d_skip, p_dt, y, n_seqs, st);
+    if (N <= 128) return launch_chunk<128>(proj, z, xc, gd, state, seq_slots, cu_seqlens, tok_pos, d_skip, p_dt, y, n_seqs, st);
+    return launch_chunk<256>(proj, z, xc, gd, state, seq_slots, cu_seqlens, tok_pos, d_skip, p_dt, y, n_seqs, st);
 }
 
 extern "C" int nncpu_ssm_step(const float* proj, int ld, const void* conv_w, int w_dt, const void* conv_b, int b_dt, float* state,

@@ -1164,6 +1164,24 @@ def ssm_scan(proj, xc, gd, state, seq_slots, cu_seqlens, tok_pos, d_skip, y, n_s
           _i(n_seqs), _i(H), _i(P), _i(G), _i(N), _i(taps), _stream())
 
 
+SSM_CHUNK_MAX_STATE = 256
+
+
+def ssm_chunk_scan(proj, xc, gd, state, seq_slots, cu_seqlens, tok_pos, d_skip, y, n_seqs: int, sizes) -> None:
+    """``ssm_scan`` for prompts of a bfloat16 run, in chunks of 64 tokens as products on the tensor cores: ``xc`` bfloat16,
+    states of up to ``SSM_CHUNK_MAX_STATE`` rows.  The state, decays and step sizes are 32-bit; where they become operands
+    they are split into two bfloat16 numbers."""
+    H, P, G, N, taps = sizes
+    n = y.shape[0]
+    _ssm_check(proj, state, sizes)
+    assert xc.dtype == torch.bfloat16 and xc.shape == (n, ssm_row(H, P, G, N)) and xc.is_contiguous()
+    assert gd.shape == (n, 2 * H) and gd.dtype == torch.float32 and d_skip.numel() == H
+    assert y.shape == (n, H * P) and y.dtype == torch.float32
+    _call("state_space", "nncpu_ssm_chunk_scan", _ptr(proj), _i(proj.shape[1]), _ptr(xc), _ptr(gd), _ptr(state),
+          _l(state.shape[1]), _ptr(seq_slots), _ptr(cu_seqlens), _ptr(tok_pos), _ptr(d_skip), _i(_code(d_skip)), _ptr(y),
+          _i(n_seqs), _i(H), _i(P), _i(G), _i(N), _i(taps), _stream())
+
+
 def ssm_step(proj, conv_w, conv_b, state, tok_pos, seq_slots, dt_bias, a_log, d_skip, y, sizes) -> None:
     """A decode step, one token per sequence, from the projections to y in one launch: convolutions, step size, recurrence
     and read-out (as ``ssm_conv`` and ``ssm_scan`` with sequences of one token)."""

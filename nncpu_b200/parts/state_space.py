@@ -30,6 +30,7 @@ from .base import Mixer, register_mixer
 
 MAX_STATE = 512        # the scan kernel spreads a column's rows over the 32 lanes of a warp, 16 rows a lane
 MAX_TAPS = 32
+CHUNKS_FROM_TOKENS = 16    # new tokens per sequence from which a prompt step of a bfloat16 run goes in chunks
 
 
 @register_mixer("state_space")
@@ -103,8 +104,12 @@ class StateSpace(Mixer):
                 ops.ssm_conv(proj, self.w_conv, self.b_conv, cache.state, ctx.tok_seq, ctx.tok_pos, ctx.seq_slots,
                              ctx.cu_seqlens, self.dt_bias, self.a_log, xc, gd, self.sizes)
             with rt.phase("ssm_scan", nbytes=state_bytes + xc.numel() * xc.element_size() + 4.0 * y.numel(), flops=flops):
-                ops.ssm_scan(proj, xc, gd, cache.state, ctx.seq_slots, ctx.cu_seqlens, ctx.tok_pos, self.d_skip, y,
-                             ctx.n_seqs, self.sizes)
+                # prompts of a bfloat16 run in chunks on the tensor cores; a few tokens per sequence, and a float32 run, in order
+                chunks = (xc.dtype == torch.bfloat16 and s.state <= ops.SSM_CHUNK_MAX_STATE
+                          and n >= CHUNKS_FROM_TOKENS * ctx.n_seqs)
+                scan = ops.ssm_chunk_scan if chunks else ops.ssm_scan
+                scan(proj, xc, gd, cache.state, ctx.seq_slots, ctx.cu_seqlens, ctx.tok_pos, self.d_skip, y, ctx.n_seqs,
+                     self.sizes)
         gated = rt.empty(n, self.inner)
         with rt.phase("ssm_gate", nbytes=8.0 * y.numel() + gated.numel() * gated.element_size()):
             ops.ssm_gated_norm(y, proj, self.w_norm, s.eps, gated, s.norm_groups)
