@@ -17,7 +17,8 @@ with host token ids in and out.  The line also carries a prefill measurement (on
 ``long-context`` (larger Qwen3 sizes end to end), ``romepel`` / ``zevivik`` (those designs at two widths beside Qwen3
 layers of equal size: a 2 048-token prompt, decode at batch 8, and every phase's time and roofline fraction), and
 ``pikalorn`` (that design at two widths beside Zevivik and Romepel layers of equal size, measured the same way),
-``vodalorn`` (that design at two widths beside Pikalorn and Zevivik layers of equal size, measured the same way).
+``vodalorn`` (that design at two widths beside Pikalorn and Zevivik layers of equal size, measured the same way), ``gekilix`` (that design at two widths beside Zevivik and Romepel layers
+of equal size, measured the same way).
 """
 from __future__ import annotations
 
@@ -238,6 +239,7 @@ WORKLOADS = {
     "zevivik": dict(model="8b"),
     "pikalorn": dict(model="8b"),
     "vodalorn": dict(model="8b"),
+    "gekilix": dict(model="8b"),
 }
 
 # `--workload romepel`: the Romepel design (recurrent gla layers, windowed attention with a distance bias, sandwich
@@ -441,6 +443,50 @@ def vodalorn_configs(z: dict):
     return vod, pik, zev
 
 
+# `--workload gekilix`: the Gekilix design (state-space layers and windowed attention that keeps the first keys, routed
+# experts with weighted inputs and a gated shared one) at sizes that resemble a real model's layers, beside the two
+# closest existing designs at equal width and depth: Zevivik (the same experts in every layer, windowed attention
+# everywhere) and Romepel (gla layers whose states have as many numbers at the state-space layers' places).
+GEKILIX_SIZES = {
+    "2048": dict(width=2048, layers=8, heads=16, kv_heads=4, dim=128, vdim=128, window=1024, keep=64, inter=6144, experts=16, top=2,
+                 ssm_heads=64, ssm_vdim=64, ssm_state=128, ssm_groups=4, conv=4, vocab=32768),
+    "4096": dict(width=4096, layers=8, heads=32, kv_heads=8, dim=128, vdim=128, window=1024, keep=64, inter=12288, experts=16, top=2,
+                 ssm_heads=128, ssm_vdim=64, ssm_state=128, ssm_groups=8, conv=4, vocab=65536),
+}
+
+
+def gekilix_configs(z: dict):
+    """(Gekilix configuration, Zevivik's and Romepel's of equal size).  Layers in fours: state space, attention, state
+    space, state space.  Romepel's gla layers have heads of 128 x 256 for every four of 128 x 64."""
+    from nncpu_b200.config import config_from_dict
+    rot = {"base": 1000000.0, "dims": z["dim"]}
+    experts = {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"]}}
+    moe = dict(experts, expert={"ff": z["inter"] // 4}, shared={"ff": z["inter"] // 2})
+    ssm = {"type": "mamba2", "mlp": moe,
+           "mixer": {"heads": z["ssm_heads"], "vdim": z["ssm_vdim"], "state": z["ssm_state"], "groups": z["ssm_groups"],
+                     "conv": z["conv"], "norm_groups": z["ssm_groups"]}}
+    att = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["vdim"], "scale": z["dim"] ** -0.5}
+    gatt = {"type": "attention", "mlp": moe,
+            "mixer": dict(att, mask={"size": z["window"], "keep_first": z["keep"]},
+                          rot=dict(rot, scaling={"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}))}
+    gek = config_from_dict({"architecture": "Gekilix", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6},
+                            "layers": [gatt if i % 4 == 1 else ssm for i in range(z["layers"])]})
+    zmoe = dict(experts, expert={"ff": z["inter"] // 4, "limit": 7.0}, shared={"ff": z["inter"] // 2, "limit": 7.0})
+    zatt = {"type": "attention", "mlp": zmoe, "mixer": dict(att, mask={"size": z["window"]}, rot=rot)}
+    zev = config_from_dict({"architecture": "Zevivik", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6},
+                            "embedding": {"scale": 1.0}, "layers": [zatt] * z["layers"]})
+    dense = {"kind": "dense", "ff": z["inter"] * 3 // 2}
+    rgla = {"type": "gla", "mlp": dense,
+            "mixer": {"heads": z["ssm_heads"] // 4, "dim": z["ssm_state"], "vdim": 4 * z["ssm_vdim"], "tau": 8.0,
+                      "rank": z["width"] // 64}}
+    ratt = {"type": "attention", "mlp": dense,
+            "mixer": dict(att, mask={"size": z["window"]}, q_temp={"coef": 0.25, "every": 256})}
+    rom = config_from_dict({"architecture": "Romepel", "vocab": z["vocab"], "width": z["width"], "max_positions": CONTEXT,
+                            "norm": {"eps": 1e-6}, "logit_softcap": 30.0,
+                            "layers": [ratt if i % 4 == 1 else rgla for i in range(z["layers"])]})
+    return gek, zev, rom
+
+
 def phase_table(totals: dict, calls: int, pk: dict) -> dict:
     """Per phase of the profiler: milliseconds per step and, where the phase states its bytes and operations, the
     fraction of the roofline (the slower of bytes / copy bandwidth and operations / tensor throughput, over the time)."""
@@ -555,6 +601,18 @@ def run_vodalorn() -> dict:
         out["sizes"][name] = {"config": z, "vodalorn": run_design_point(vod, z["vocab"], pk),
                               "pikalorn_same_size": run_design_point(pik, z["vocab"], pk),
                               "zevivik_same_size": run_design_point(zev, z["vocab"], pk)}
+    return out
+
+
+def run_gekilix() -> dict:
+    pk = peaks()
+    out = {"workload": "gekilix", "dtype": "bf16", "peaks": pk["source"], "prompt": PROMPT,
+           "data": "synthetic: random weights, uniform random token ids", "sizes": {}}
+    for name, z in GEKILIX_SIZES.items():
+        gek, zev, rom = gekilix_configs(z)
+        out["sizes"][name] = {"config": z, "gekilix": run_design_point(gek, z["vocab"], pk),
+                              "zevivik_same_size": run_design_point(zev, z["vocab"], pk),
+                              "romepel_same_size": run_design_point(rom, z["vocab"], pk)}
     return out
 
 
@@ -723,7 +781,7 @@ def main() -> int:
         return 0
     if args.workload:
         special = {"long-context": run_long_context, "romepel": run_romepel, "zevivik": run_zevivik,
-                   "pikalorn": run_pikalorn, "vodalorn": run_vodalorn}
+                   "pikalorn": run_pikalorn, "vodalorn": run_vodalorn, "gekilix": run_gekilix}
         print(json.dumps(special[args.workload]() if args.workload in special else run_workload(args.workload)))
         return 0
     model = Model.random(cfg, seed=0, dtype="bfloat16", device="cuda:0")

@@ -622,6 +622,71 @@ qk_whole_norm_append_kernel(const float* __restrict__ qkv, int ld, const void* _
     }
 }
 
+// The same for a bfloat16 run whose heads and rows are multiples of 4 lanes: items of four lanes, 16-byte loads, and the
+// two sums of squares from one pass over the row.
+__global__ void __launch_bounds__(256)
+qk_whole_norm_append_vec_kernel(const float* __restrict__ qkv, int ld, const void* __restrict__ q_gamma,
+                                const void* __restrict__ k_gamma, int g_dt, float eps, const float2* __restrict__ cs, int half,
+                                const int* __restrict__ tok_seq, const int* __restrict__ tok_pos,
+                                const int* __restrict__ block_table, int bt_stride, __nv_bfloat16* __restrict__ k_pages,
+                                __nv_bfloat16* __restrict__ v_pages, __nv_bfloat16* __restrict__ q_out, int n_heads, int n_kv,
+                                int hd, int vd, int qp, int vp) {
+    __shared__ float scratch[33];
+    const int t = blockIdx.x, tid = threadIdx.x;
+    const float4* row = reinterpret_cast<const float4*>(qkv + (size_t)t * ld);
+    const int nq = n_heads * hd, nk = n_kv * hd, seq = tok_seq[t], pos = tok_pos[t];
+    const int page = (seq >= 0 && n_kv > 0) ? block_table[(size_t)seq * bt_stride + pos / kPage] : -1;
+    float q_scale = 1.0f, k_scale = 1.0f;
+    if (q_gamma != nullptr || k_gamma != nullptr) {
+        float qs = 0.0f, ks = 0.0f;
+        for (int i = tid; i < (nq + nk) >> 2; i += 256) {
+            const float4 v = row[i];
+            const float sq = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w)));
+            if (4 * i < nq) qs += sq;
+            else ks += sq;
+        }
+        q_scale = 1.0f / sqrtf(block_sum(qs, scratch) * (1.0f / (float)nq) + eps);
+        if (nk > 0) k_scale = 1.0f / sqrtf(block_sum(ks, scratch) * (1.0f / (float)nk) + eps);
+    }
+    const int pq = qp >> 2, pv = vp >> 2;
+    const int items_q = n_heads * pq, items_k = page >= 0 ? n_kv * pq : 0, items_v = page >= 0 ? n_kv * pv : 0;
+    for (int it = tid; it < items_q + items_k + items_v; it += 256) {
+        const bool is_q = it < items_q, is_v = it >= items_q + items_k;
+        const int per = is_v ? pv : pq, j = is_q ? it : is_v ? it - items_q - items_k : it - items_q;
+        const int h = j / per, d = (j % per) * 4, size = is_v ? vd : hd;
+        const int at = (is_q ? 0 : is_v ? nq + nk : nq) + h * size + d;
+        float4 v = d < size ? row[at >> 2] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        const void* gamma = is_v ? nullptr : is_q ? q_gamma : k_gamma;
+        if (gamma != nullptr && d < size) {
+            const float s = is_q ? q_scale : k_scale;
+            const int g0 = h * hd + d;
+            v.x = (v.x * s) * ld_f(gamma, g0, g_dt);
+            v.y = (v.y * s) * ld_f(gamma, g0 + 1, g_dt);
+            v.z = (v.z * s) * ld_f(gamma, g0 + 2, g_dt);
+            v.w = (v.w * s) * ld_f(gamma, g0 + 3, g_dt);
+        }
+        if (!is_v && cs != nullptr) {
+            const int p0 = d >> 1;
+            if (p0 < half) {
+                const float2 c = cs[(size_t)t * half + p0];
+                const float a = v.x;
+                v.x = c.x * a - c.y * v.y;
+                v.y = c.y * a + c.x * v.y;
+            }
+            if (p0 + 1 < half) {
+                const float2 c = cs[(size_t)t * half + p0 + 1];
+                const float a = v.z;
+                v.z = c.x * a - c.y * v.w;
+                v.w = c.y * a + c.x * v.w;
+            }
+        }
+        __nv_bfloat162 o[2] = {__floats2bfloat162_rn(v.x, v.y), __floats2bfloat162_rn(v.z, v.w)};
+        __nv_bfloat16* dst = is_q ? q_out + ((size_t)t * n_heads + h) * qp + d
+                                  : (is_v ? v_pages : k_pages) + (((size_t)page * n_kv + h) * kPage + pos % kPage) * (is_v ? vp : qp) + d;
+        *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<uint2*>(o);
+    }
+}
+
 extern "C" int nncpu_qk_whole_norm_append(const float* qkv, int ld, const void* q_gamma, const void* k_gamma, int g_dt,
                                           float eps, const float* cs, int half, const int* tok_seq, const int* tok_pos,
                                           const int* block_table, int bt_stride, void* k_pages, void* v_pages, int kv_dt,
@@ -633,6 +698,14 @@ extern "C" int nncpu_qk_whole_norm_append(const float* qkv, int ld, const void* 
     NN_CHECK(cs == nullptr || 2 * half <= hd, "q/k norm and append: %d rotated pairs of a head of %d lanes", half, hd);
     NN_CHECK((uintptr_t)cs % 8 == 0, "q/k norm and append: the rotation table must be 8-byte aligned (cos/sin pairs)");
     if (n_tok == 0) return 0;
+    if (q_dt == DT_BF16 && (n_kv == 0 || kv_dt == DT_BF16) && ((hd | vd | qp | vp | ld) & 3) == 0 &&
+        (((uintptr_t)qkv | (uintptr_t)q_out | (uintptr_t)k_pages | (uintptr_t)v_pages) % 16) == 0) {
+        qk_whole_norm_append_vec_kernel<<<n_tok, 256, 0, (cudaStream_t)stream>>>(
+            qkv, ld, q_gamma, k_gamma, g_dt, eps, (const float2*)cs, half, tok_seq, tok_pos, block_table, bt_stride,
+            (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, (__nv_bfloat16*)q_out, n_heads, n_kv, hd, vd, qp, vp);
+        NN_LAUNCH_OK("q/k norm and append");
+        return 0;
+    }
     qk_whole_norm_append_kernel<<<n_tok, 256, 0, (cudaStream_t)stream>>>(
         qkv, ld, q_gamma, k_gamma, g_dt, eps, (const float2*)cs, half, tok_seq, tok_pos, block_table, bt_stride, k_pages,
         v_pages, kv_dt, q_out, q_dt, n_heads, n_kv, hd, vd, qp, vp);

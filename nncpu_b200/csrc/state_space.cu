@@ -130,6 +130,26 @@ conv_kernel(const float* __restrict__ proj, const Sizes z, const void* __restric
             w[j] = ld_f(conv_w, (size_t)ch * z.taps + z.taps - 1 - j, w_dt);
             past[j] = 0.0f;
         }
+        // a whole tile of one sequence (a prompt's usual case): all of the tile's inputs are asked for before the first is used
+        const int seq = tok_seq[t_first];
+        const int slot = seq < 0 ? -1 : seq_slots[seq];
+        if (t_end - t_first == kConvTokens && slot >= 0 && tok_seq[t_end - 1] == seq) {
+            const int local = t_first - cu_seqlens[seq], pos = tok_pos[t_first];
+            const float* ring = state + (size_t)slot * z.slot_stride + z.conv_at;
+            float in[kConvTokens + kKept - 1];           // in[k]: the input of the tile's token k - (taps - 1)
+#pragma unroll
+            for (int k = 0; k < kConvTokens; ++k) in[k + kKept - 1] = proj[(size_t)(t_first + k) * z.ld + z.inner() + ch];
+#pragma unroll
+            for (int j = 1; j < kKept; ++j) in[kKept - 1 - j] = conv_input(proj, z, ring, t_first, local, pos, j, ch);
+#pragma unroll
+            for (int k = 0; k < kConvTokens; ++k) {
+                float acc = bias;
+#pragma unroll
+                for (int j = kKept - 1; j >= 0; --j) acc = fmaf(w[j], in[k + kKept - 1 - j], acc);
+                st_f(xc, (size_t)(t_first + k) * row + idx, xc_dt, silu_f(acc));
+            }
+            return;
+        }
     }
     for (int t = t_first; t < t_end; ++t) {
         const int seq = tok_seq[t];
@@ -757,6 +777,47 @@ gated_norm_kernel(const float* __restrict__ y, const float* __restrict__ proj, i
         st_f(out, (size_t)t * inner + g0 + i, out_dt, ((ys[i] * silu_f(zs[i])) * scale) * ld_f(w, g0 + i, w_dt));
 }
 
+// The same for parts that are a multiple of 4 lanes (at most 4 kVec blockDim) in 16-byte rows.
+template <int kVec>
+__global__ void __launch_bounds__(256)
+gated_norm_vec_kernel(const float* __restrict__ y, const float* __restrict__ proj, int ld, const void* __restrict__ w, int w_dt,
+                      float eps, void* __restrict__ out, int out_dt, int inner, int part) {
+    __shared__ float scratch[33];
+    const int t = blockIdx.x, g0 = blockIdx.y * part, n4 = part >> 2;
+    const float4* ys = reinterpret_cast<const float4*>(y + (size_t)t * inner + g0);
+    const float4* zs = reinterpret_cast<const float4*>(proj + (size_t)t * ld + g0);
+    float4 v[kVec], g[kVec];
+    float ss = 0.0f;
+#pragma unroll
+    for (int j = 0; j < kVec; ++j) {
+        const int i = threadIdx.x + j * blockDim.x;
+        v[j] = i < n4 ? ys[i] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        g[j] = i < n4 ? zs[i] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    }
+#pragma unroll
+    for (int j = 0; j < kVec; ++j) {
+        v[j].x *= silu_f(g[j].x); v[j].y *= silu_f(g[j].y); v[j].z *= silu_f(g[j].z); v[j].w *= silu_f(g[j].w);
+        ss = fmaf(v[j].x, v[j].x, ss); ss = fmaf(v[j].y, v[j].y, ss);
+        ss = fmaf(v[j].z, v[j].z, ss); ss = fmaf(v[j].w, v[j].w, ss);
+    }
+    ss = block_sum(ss, scratch);
+    const float scale = 1.0f / sqrtf(ss * (1.0f / (float)part) + eps);
+#pragma unroll
+    for (int j = 0; j < kVec; ++j) {
+        const int i = threadIdx.x + j * blockDim.x;
+        if (i >= n4) continue;
+        const int at = g0 + 4 * i;
+        const float o[4] = {(v[j].x * scale) * ld_f(w, at, w_dt), (v[j].y * scale) * ld_f(w, at + 1, w_dt),
+                            (v[j].z * scale) * ld_f(w, at + 2, w_dt), (v[j].w * scale) * ld_f(w, at + 3, w_dt)};
+        if (out_dt == DT_BF16) {
+            __nv_bfloat162 h[2] = {__floats2bfloat162_rn(o[0], o[1]), __floats2bfloat162_rn(o[2], o[3])};
+            *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(out) + (size_t)t * inner + at) = *reinterpret_cast<uint2*>(h);
+        } else {
+            *reinterpret_cast<float4*>(reinterpret_cast<float*>(out) + (size_t)t * inner + at) = make_float4(o[0], o[1], o[2], o[3]);
+        }
+    }
+}
+
 int make_sizes(Sizes* z, int H, int P, int G, int N, int taps, int ld, long slot_stride) {
     NN_CHECK(H > 0 && P > 0 && G > 0 && H % G == 0 && N > 0, "state space: %d heads over %d groups, states of %d x %d", H, G, N, P);
     NN_CHECK(taps >= 1 && taps <= kMaxTaps, "state space: convolutions of %d taps (1 to %d)", taps, kMaxTaps);
@@ -865,6 +926,19 @@ extern "C" int nncpu_ssm_gated_norm(const float* y, const float* proj, int ld, c
     if (n_tok == 0) return 0;
     const int part = inner / n_groups;
     NN_CHECK(n_groups <= 65535, "gated norm: %d parts", n_groups);
+    if (part % 4 == 0 && ld % 4 == 0 && part <= 8192 && (((uintptr_t)y | (uintptr_t)proj | (uintptr_t)out) % 16) == 0) {
+        const int vec_threads = part >= 1024 ? 256 : (part / 4 + 31) / 32 * 32;
+#define NN_GATE(V)                                                                                                         \
+    gated_norm_vec_kernel<V><<<dim3(n_tok, n_groups), vec_threads, 0, (cudaStream_t)stream>>>(y, proj, ld, w, w_dt, eps, out, \
+                                                                                              out_dt, inner, part)
+        if (part <= 1024) NN_GATE(1);
+        else if (part <= 2048) NN_GATE(2);
+        else if (part <= 4096) NN_GATE(4);
+        else NN_GATE(8);
+#undef NN_GATE
+        NN_LAUNCH_OK("gated norm");
+        return 0;
+    }
     const int threads = part >= 256 ? 256 : (part + 31) / 32 * 32;
     gated_norm_kernel<<<dim3(n_tok, n_groups), threads, 0, (cudaStream_t)stream>>>(y, proj, ld, w, w_dt, eps, out, out_dt, inner, part);
     NN_LAUNCH_OK("gated norm");
