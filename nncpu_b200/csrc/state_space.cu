@@ -640,8 +640,8 @@ int launch_chunk(const float* proj, const Sizes& z, const void* xc, const float*
 // ---------------------------------------------------------------------------
 constexpr int kStepCols = 64, kStepThreads = 256;
 
-template <int VEC>
-__global__ void __launch_bounds__(kStepThreads)
+template <int VEC, int TAPS>
+__global__ void __launch_bounds__(kStepThreads, VEC == 4 ? 3 : 1)
 step_kernel(const float* __restrict__ proj, const Sizes z, const void* __restrict__ conv_w, int w_dt,
             const void* __restrict__ conv_b, int b_dt, float* state, const int* __restrict__ tok_pos,
             const int* __restrict__ seq_slots, const void* __restrict__ dt_bias, const void* __restrict__ a_log,
@@ -685,11 +685,22 @@ step_kernel(const float* __restrict__ proj, const Sizes z, const void* __restric
         const int j = i - cols;
         const int ch = i < cols ? h * z.P + col0 + i : z.inner() + (j < z.N ? 0 : z.G * z.N) + g * z.N + j % z.N;
         float acc = ld_f(conv_b, ch, b_dt);
-        for (int back = z.taps - 1; back > 0; --back)
-            if (pos >= back)
-                acc = fmaf(ld_f(conv_w, (size_t)ch * z.taps + z.taps - 1 - back, w_dt), ring[(size_t)((pos - back) % z.taps) * C + ch], acc);
         const float now = own[ch];
-        acc = fmaf(ld_f(conv_w, (size_t)ch * z.taps + z.taps - 1, w_dt), now, acc);
+        if (TAPS > 0) {          // (known taps: every input and weight is asked for before the first is used)
+            float in[TAPS > 0 ? TAPS : 1], w[TAPS > 0 ? TAPS : 1];
+#pragma unroll
+            for (int back = TAPS - 1; back >= 0; --back) {
+                in[back] = back == 0 ? now : pos >= back ? ring[(size_t)((pos - back) % TAPS) * C + ch] : 0.0f;
+                w[back] = ld_f(conv_w, (size_t)ch * TAPS + TAPS - 1 - back, w_dt);
+            }
+#pragma unroll
+            for (int back = TAPS - 1; back >= 0; --back) acc = fmaf(w[back], in[back], acc);
+        } else {
+            for (int back = z.taps - 1; back > 0; --back)
+                if (pos >= back)
+                    acc = fmaf(ld_f(conv_w, (size_t)ch * z.taps + z.taps - 1 - back, w_dt), ring[(size_t)((pos - back) % z.taps) * C + ch], acc);
+            acc = fmaf(ld_f(conv_w, (size_t)ch * z.taps + z.taps - 1, w_dt), now, acc);
+        }
         const float v = silu_f(acc);
         if (i < cols) xs[i] = v;
         else step_smem[j] = v;
@@ -909,12 +920,13 @@ extern "C" int nncpu_ssm_step(const float* proj, int ld, const void* conv_w, int
     const dim3 grid(n_tok, H, (P + kStepCols - 1) / kStepCols);
     const size_t smem = (size_t)2 * N * sizeof(float);
     const bool vec = P % 4 == 0 && slot_stride % 4 == 0 && (uintptr_t)state % 16 == 0;
-    if (vec)
-        step_kernel<4><<<grid, kStepThreads, smem, (cudaStream_t)stream>>>(proj, z, conv_w, w_dt, conv_b, b_dt, state, tok_pos,
-                                                                           seq_slots, dt_bias, a_log, d_skip, p_dt, y);
-    else
-        step_kernel<1><<<grid, kStepThreads, smem, (cudaStream_t)stream>>>(proj, z, conv_w, w_dt, conv_b, b_dt, state, tok_pos,
-                                                                           seq_slots, dt_bias, a_log, d_skip, p_dt, y);
+#define NN_STEP(VEC, TAPS)                                                                                                 \
+    step_kernel<VEC, TAPS><<<grid, kStepThreads, smem, (cudaStream_t)stream>>>(proj, z, conv_w, w_dt, conv_b, b_dt, state,  \
+                                                                               tok_pos, seq_slots, dt_bias, a_log, d_skip, p_dt, y)
+    if (vec && taps == 4) NN_STEP(4, 4);
+    else if (vec) NN_STEP(4, 0);
+    else NN_STEP(1, 0);
+#undef NN_STEP
     NN_LAUNCH_OK("state space (step)");
     return 0;
 }

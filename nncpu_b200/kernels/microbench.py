@@ -10,6 +10,7 @@ GFLOP/s for its row kernels and one attention block.
     python -m nncpu_b200.kernels.microbench rmsnorm ROWS DIM
     python -m nncpu_b200.kernels.microbench gla BATCH TOKENS [--columns 2|4]
     python -m nncpu_b200.kernels.microbench delta BATCH TOKENS [--lanes 4|8|16|32] [--columns 1|2] [--channel-decay]
+    python -m nncpu_b200.kernels.microbench ssm BATCH TOKENS [--heads 64] [--value-dim 64] [--state 128] [--groups 4] [--in-order]
 
 Timing: the kernel is captured in a CUDA graph over enough different buffers
 that no launch finds its operands in L2, replayed, and timed with CUDA events.
@@ -243,6 +244,35 @@ def delta(args) -> None:
           f"{3.0 * n * h * d * e / ms / 1e9:.2f} T multiply-adds/s, {nbytes / ms / 1e6:.0f} GB/s of inputs, outputs and state")
 
 
+def ssm(args) -> None:
+    """The state-space recurrence over `tokens` tokens of `batch` sequences: in chunks on the tensor cores, `--in-order` the
+    scan on the CUDA cores; with one token the decode step's kernel (convolutions included)."""
+    b, t, h, p, g, n_, taps = args.batch, args.tokens, args.heads, args.value_dim, args.groups, args.state, 4
+    n, c, sizes = b * t, h * p + 2 * g * n_, (h, p, g, n_, 4)
+    proj = torch.randn(n, (h * p + c + h + 7) // 8 * 8, device=DEV) * 0.3
+    state = torch.zeros(b + 1, ops.ssm_state_floats(*sizes), device=DEV)
+    slots = torch.arange(b, dtype=torch.int32, device=DEV)
+    cu = torch.arange(0, n + 1, t, dtype=torch.int32, device=DEV)
+    pos = torch.arange(t, dtype=torch.int32, device=DEV).repeat(b)
+    per_head = torch.zeros(h, device=DEV)
+    y = torch.empty(n, h * p, device=DEV)
+    if t == 1:
+        conv_w, conv_b = torch.randn(c, taps, device=DEV).bfloat16(), torch.zeros(c, device=DEV).bfloat16()
+        pos += 100
+        run = lambda: ops.ssm_step(proj, conv_w, conv_b, state, pos, slots, per_head, per_head, per_head, y, sizes)
+        nbytes = 8.0 * b * h * p * n_ + 4.0 * (n * (c + h) + y.numel())
+    else:
+        xc = (torch.randn(n, ops.ssm_row(h, p, g, n_), device=DEV) * 0.3).bfloat16()
+        gd = torch.cat([-torch.rand(n, h, device=DEV) * 0.1, torch.rand(n, h, device=DEV)], dim=1).contiguous()
+        fn = ops.ssm_scan if args.in_order else ops.ssm_chunk_scan
+        run = lambda: fn(proj, xc, gd, state, slots, cu, pos, per_head, y, b, sizes)
+        nbytes = 2.0 * xc.numel() + 4.0 * (gd.numel() + y.numel()) + 8.0 * b * h * p * n_
+    ms = _time([run], args.once)
+    print(f"state space {'step' if t == 1 else 'in order' if args.in_order else 'in chunks'} batch={b} tokens={t} heads={h} on {g} "
+          f"state={n_} x {p}: {ms * 1e3:.1f} us, {2.0 * n * h * p * n_ / ms / 1e9:.2f} T multiply-adds/s of the recurrence, "
+          f"{nbytes / ms / 1e6:.0f} GB/s of inputs, outputs and state")
+
+
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
     ap.add_argument("--once", action="store_true", help="three plain launches, no timing (for a profiler)")
@@ -293,6 +323,12 @@ def main(argv=None) -> int:
     p.add_argument("--columns", type=int, default=0, choices=[0, 1, 2], help="columns of the state a lane (0: by the layer's sizes)")
     p.add_argument("--channel-decay", action="store_true", help="a decay per head and key channel instead of one per head")
     p.set_defaults(fn=delta)
+    p = sub.add_parser("ssm")
+    p.add_argument("batch", type=int); p.add_argument("tokens", type=int)
+    p.add_argument("--heads", type=int, default=64); p.add_argument("--value-dim", type=int, default=64)
+    p.add_argument("--groups", type=int, default=4); p.add_argument("--state", type=int, default=128)
+    p.add_argument("--in-order", action="store_true", help="the scan on the CUDA cores instead of chunks on the tensor cores")
+    p.set_defaults(fn=ssm)
     args = ap.parse_args(argv)
     if args.no_overlap:
         ops.launch_overlap(False)
