@@ -12,6 +12,7 @@ from .zevivik import ZevivikConfig
 from .pikalorn import PikalornConfig
 from .vodalorn import VodalornConfig
 from .gekilix import GekilixConfig
+from .vuvalorn import VuvalornConfig
 
 __all__ = [
     "architectures", "config_class", "config_from_dict", "load_config", "register_architecture",
@@ -19,5 +20,5 @@ __all__ = [
     "ModelSpec", "NormSpec", "OutputSpec", "PositionSpec", "ScheduleEntry", "Qwen3Config", "RomepelConfig",
     "DenseMlpSpec", "GatedLinearAttentionSpec", "LatentAttentionSpec", "RoutedExpertsSpec", "StreamInjection",
     "ZevivikConfig", "GatedDeltaSpec", "PikalornConfig", "MixerPairSpec", "RetentionSpec", "TokenSideSpec",
-    "VodalornConfig", "GekilixConfig", "StateSpaceSpec",
+    "VodalornConfig", "GekilixConfig", "VuvalornConfig", "StateSpaceSpec",
 ]

@@ -29,6 +29,7 @@ class NormSpec:
     suffix: str = ".weight"
     offset: float = 0.0
     bias_suffix: str = ".b"
+    gain: float = 1.0        # multiplies the norm's output (a constant factor on whatever reads it linearly); "rmsnorm"
 
 
 @dataclass(frozen=True)
@@ -92,6 +93,11 @@ class AttentionSpec(MixerSpec):
                                      # denominator: it has no key and no value, is not scaled, and counts once
     out_gate: bool = False           # the concatenated heads are multiplied, lane by lane, by sigmoid(W_g h)
                                      # ("<name>.g", n_heads * v_head_dim rows) before the output projection
+    head_gate: bool = False          # the same with one number per head ("<name>.g", n_heads rows)
+    score_cap: float = 0.0           # c > 0: a scaled score z becomes c * tanh(z / c) before the softmax
+    conv: int = 0                    # n > 0: q and k (and so a value that is the key) pass a causal convolution over time of
+                                     # n taps per channel ("<name>.q.conv", ".k.conv" [channels, n]) right after the
+                                     # projection; the last n - 1 projections are per-sequence state
 
 
 @dataclass(frozen=True)
@@ -257,6 +263,12 @@ class RoutedExpertsSpec(FeedForwardSpec):
     out_scale: float = 1.0
     weight_on: str = "output"
     shared_gate: bool = False
+    # ``scores`` "plain": the softmax over all the router's outputs; the weights are the chosen scores as they are, times
+    # ``weight_scale``.
+    correction: bool = False    # ("plain") the largest score + correction is chosen ("<name>.correction", one per output);
+                                # the weights know nothing of it
+    identity: int = 0           # the router has this many more outputs after the experts': experts without tensors whose
+                                # output is their input
 
 
 @dataclass(frozen=True)

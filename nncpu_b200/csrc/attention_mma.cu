@@ -74,11 +74,22 @@ __device__ __forceinline__ float ld_cluster_(const float* local, uint32_t rank) 
     return v;
 }
 
+// A gate on the output: with `per_head` one logit a head (a row holds n_heads of them), else one a lane.
+struct OutGate {
+    const float* logits;    // row t at t * ld, or null: no gate
+    long ld;
+    int per_head;
+};
+__device__ __forceinline__ float out_gate(const OutGate& g, int t, int head, int vo, int d) {
+    const float z = g.logits[(size_t)t * g.ld + (g.per_head ? (size_t)head : (size_t)head * vo + min(d, vo - 1))];
+    return 1.0f / (1.0f + expf(-z));
+}
+
 // Merges the splits of every (token, head) in split order.  grid = (n_heads, n_tok), VD threads.
 template <int VD>
 __global__ void merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                              __nv_bfloat16* __restrict__ out, int n_heads, int n_kv, int n_splits,
-                             const float* __restrict__ sinks, const float* __restrict__ gate, long gate_ld, int vo) {
+                             const float* __restrict__ sinks, const OutGate gate, int vo) {
     const int h = blockIdx.x, t = blockIdx.y, d = threadIdx.x;
     const int G = n_heads / n_kv, kvh = h / G, head = h % G;
     const size_t pb = ((size_t)t * n_kv + kvh) * n_splits;
@@ -94,7 +105,7 @@ __global__ void merge_kernel(const float* __restrict__ part_o, const float* __re
     if (sinks != nullptr && l > 0.0f) l += exp2f(sinks[h] * kLog2e - m);
     float res = l > 0.0f ? o / l : 0.0f;
     if (d >= vo) return;
-    if (gate != nullptr) res *= 1.0f / (1.0f + expf(-gate[(size_t)t * gate_ld + (size_t)h * vo + d]));
+    if (gate.logits != nullptr) res *= out_gate(gate, t, h, vo, d);
     out[((size_t)t * n_heads + h) * vo + d] = __float2bfloat16_rn(res);
 }
 
@@ -134,7 +145,7 @@ prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restr
                const __nv_bfloat16* __restrict__ v_pages, const int* __restrict__ block_table, int bt_stride,
                const int* __restrict__ cu_seqlens, const int* __restrict__ tok_pos, __nv_bfloat16* __restrict__ out,
                int n_seqs, int n_heads, int n_kv, float scale2, int window, int keep, float slope_base,
-               const float* __restrict__ sinks, int vo) {
+               const float* __restrict__ sinks, int vo, const ScoreCap cap, const OutGate gate) {
     constexpr int kTileBytes = kPage * HD * 2;           // one page of K for one head
     constexpr int kStageBytes = kPage * (HD + VD) * 2;   // and of V behind it
     constexpr int kChunks = HD / 8, kVChunks = VD / 8;   // 16-byte chunks per row
@@ -253,7 +264,7 @@ prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restr
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const int row = e >> 1;
-                    float v = s[t][e] * scale2;
+                    float v = cap.out > 0.0f ? capped_score(s[t][e], cap) : s[t][e] * scale2;
                     if (!full || slope2 != 0.0f) {
                         const int key = k_base + t * 8 + 2 * c + (e & 1);
                         v -= slope2 * (float)(lim_hi[row] - key);
@@ -315,7 +326,8 @@ prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restr
         if (!(row == 0 ? has_lo : has_hi)) continue;
         // a sink: one more term of the denominator, with no key and no value (the softmax works in powers of two)
         if (sinks != nullptr && l[row] > 0.0f) l[row] += exp2f(sinks[h] * kLog2e - m[row]);
-        const float inv = l[row] > 0.0f ? 1.0f / l[row] : 0.0f;
+        float inv = l[row] > 0.0f ? 1.0f / l[row] : 0.0f;
+        if (gate.logits != nullptr) inv *= out_gate(gate, q0 + (row == 0 ? row_lo : row_hi), h, vo, 0);    // one a head
         __nv_bfloat16* dst = out + ((size_t)(q0 + (row == 0 ? row_lo : row_hi)) * n_heads + h) * vo;
 #pragma unroll
         for (int t = 0; t < VD / 8; ++t) {
@@ -369,22 +381,19 @@ struct FusedQK {
     float temp_coef;          // c != 0: the query at position p is multiplied by 1 + c ln(floor((p + 1) / temp_every) + 1)
     int temp_every;
     int values_are_keys;      // the row holds no v heads: a token's value is its key as projected (before norm and rotation)
-    int gate_at;              // >= 0: the row's floats from gate_at on are logits, one a lane of the output: the output is
-                              // multiplied by their sigmoid; < 0: no gate
+    ShortConv conv;           // w not null: q and k (C = all their lanes) pass it before norm and rotation; a token is then a
+                              // whole sequence of the step, and a value that is the key is taken after it
 };
 
 // One head's float32 values (n of them, zeros up to HD) through norm (if gamma) and rotation (if cs) to bfloat16; a
 // warp's job.  A lane holds HD / 32 neighbouring lanes of the head, so a rotation pair (i, i + HD / 2) sits in the lanes
 // l and l ^ 16, and a pair (2 i, 2 i + 1) in one lane.  given_scale > 0: the norm's scale is known (it runs over more
-// than this head).
-template <int HD>
-__device__ __forceinline__ void finish_head(const float* __restrict__ src, int n, const void* __restrict__ gamma, int gamma_at,
-                                            int g_dt, float eps, float given_scale, const float2* __restrict__ cs_row,
-                                            int half, int pairs, __nv_bfloat16* __restrict__ dst, int lane,
-                                            float times = 1.0f) {
-    constexpr int EPL = HD / 32;
-    float x[EPL];
-    if (n == HD && (reinterpret_cast<uintptr_t>(src) & 15) == 0) {
+// than this head).  With a convolution (`conv` not null, `ch` the head's first channel, `kept` the sequence's last inputs,
+// which begin at that channel) the values pass it first; `next` not null: this warp leaves the inputs advanced by the token
+// there.
+template <int EPL>
+__device__ __forceinline__ void load_head(const float* src, int n, int lane, float (&x)[EPL]) {
+    if (n == 32 * EPL && (reinterpret_cast<uintptr_t>(src) & 15) == 0) {
         if (EPL == 4) {
             const float4 v = *reinterpret_cast<const float4*>(src + lane * EPL);
             x[0] = v.x; x[1] = v.y; x[2 % EPL] = v.z; x[3 % EPL] = v.w;
@@ -395,6 +404,41 @@ __device__ __forceinline__ void finish_head(const float* __restrict__ src, int n
     } else {
 #pragma unroll
         for (int e = 0; e < EPL; ++e) x[e] = lane * EPL + e < n ? src[lane * EPL + e] : 0.0f;
+    }
+}
+
+template <int HD>
+__device__ __forceinline__ void finish_head(const float* __restrict__ src, int n, const void* __restrict__ gamma, int gamma_at,
+                                            int g_dt, float eps, float given_scale, const float2* __restrict__ cs_row,
+                                            int half, int pairs, __nv_bfloat16* __restrict__ dst, int lane,
+                                            float times = 1.0f, const ShortConv* conv = nullptr, int ch = 0,
+                                            const float* kept = nullptr, float* next = nullptr) {
+    constexpr int EPL = HD / 32;
+    float x[EPL];
+    load_head<EPL>(src, n, lane, x);
+    if (conv != nullptr) {
+        // the same order of additions as in a prompt: the oldest input first
+        float now[EPL], w[EPL], u[EPL];
+#pragma unroll
+        for (int e = 0; e < EPL; ++e) { now[e] = x[e]; x[e] = 0.0f; }
+        for (int j = 0; j + 1 < conv->taps; ++j) {
+            load_head<EPL>(conv->w + (size_t)j * conv->C + ch, n, lane, w);
+            load_head<EPL>(kept + (size_t)j * conv->C, n, lane, u);
+#pragma unroll
+            for (int e = 0; e < EPL; ++e) x[e] = fmaf(w[e], u[e], x[e]);
+            if (next != nullptr && j > 0) {
+#pragma unroll
+                for (int e = 0; e < EPL; ++e)
+                    if (lane * EPL + e < n) next[(size_t)(j - 1) * conv->C + lane * EPL + e] = u[e];
+            }
+        }
+        load_head<EPL>(conv->w + (size_t)(conv->taps - 1) * conv->C + ch, n, lane, w);
+#pragma unroll
+        for (int e = 0; e < EPL; ++e) {
+            x[e] = fmaf(w[e], now[e], x[e]);
+            if (next != nullptr && conv->taps > 1 && lane * EPL + e < n)
+                next[(size_t)(conv->taps - 2) * conv->C + lane * EPL + e] = now[e];
+        }
     }
     if (gamma) {
         float scale = given_scale;
@@ -467,7 +511,8 @@ decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restri
                    const __nv_bfloat16* __restrict__ v_pages, const int* __restrict__ block_table, int bt_stride,
                    const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, __nv_bfloat16* __restrict__ out,
                    float* __restrict__ part_o, float* __restrict__ part_ml, int n_heads, int n_kv, float scale2,
-                   int window, int keep, const FusedQK f, const float* __restrict__ sinks, int kv_rep, int vo) {
+                   int window, int keep, const FusedQK f, const float* __restrict__ sinks, int kv_rep, int vo,
+                   const ScoreCap cap, const OutGate gate) {
     constexpr int kTileBytes = kPage * HD * 2, kStageBytes = kPage * (HD + VD) * 2;
     constexpr int kChunks = HD / 8, kVChunks = VD / 8;
     constexpr int W = VD + 2;
@@ -537,15 +582,30 @@ decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restri
             if (f.k_gamma && owner) k_scale = 1.0f / sqrtf(row_squares(row + f.k_at, n_kv * f.hd, sq_s) * (1.0f / (float)(n_kv * f.hd)) + f.eps);
         }
         const float temp = f.temp_coef != 0.0f ? 1.0f + f.temp_coef * logf((float)((pos + 1) / f.temp_every) + 1.0f) : 1.0f;
-        for (int g = warp; g < G; g += 4)
-            finish_head<HD>(row + (size_t)(kvh * G + g) * f.hd, f.hd, f.q_gamma, f.whole ? (kvh * G + g) * f.hd : 0, f.g_dt,
-                            f.eps, q_scale, cs_row, f.half, f.pairs, q_s + g * HD, lane, temp);
+        // A short convolution: every block reads the inputs kept from earlier steps; the first split's blocks leave those
+        // of the queries advanced in the state's other copy, the owner those of its key.
+        const ShortConv* conv = f.conv.w != nullptr ? &f.conv : nullptr;
+        const float* kept = nullptr;
+        float* next = nullptr;
+        if (conv != nullptr) {
+            const int slot = f.conv.seq_slots[seq], copy = conv_copy_in_use(f.conv, slot, pos);
+            kept = conv_copy(f.conv, slot, copy);
+            next = conv_copy(f.conv, slot, 1 - copy);
+            if (split == 0 && kvh == 0 && threadIdx.x == 0) conv_mark(f.conv, slot, 1 - copy, pos + 1);
+        }
+        for (int g = warp; g < G; g += 4) {
+            const int ch = (kvh * G + g) * f.hd;
+            finish_head<HD>(row + ch, f.hd, f.q_gamma, f.whole ? ch : 0, f.g_dt, f.eps, q_scale, cs_row, f.half, f.pairs,
+                            q_s + g * HD, lane, temp, conv, ch, kept + ch, split == 0 && next != nullptr ? next + ch : nullptr);
+        }
         if (owner) {
+            const int ch = f.k_at + kvh * f.hd;
             if (warp == 0)
-                finish_head<HD>(row + f.k_at + (size_t)kvh * f.hd, f.hd, f.k_gamma, f.whole ? kvh * f.hd : 0, f.g_dt, f.eps,
-                                k_scale, cs_row, f.half, f.pairs, kv_s, lane);
+                finish_head<HD>(row + ch, f.hd, f.k_gamma, f.whole ? kvh * f.hd : 0, f.g_dt, f.eps, k_scale, cs_row, f.half,
+                                f.pairs, kv_s, lane, 1.0f, conv, ch, kept + ch, next != nullptr ? next + ch : nullptr);
             if (warp == 1)
-                finish_head<VD>(row + f.v_at + (size_t)kvh * f.vd, f.vd, nullptr, 0, 0, 0.0f, 0.0f, nullptr, 0, 0, kv_s + HD, lane);
+                finish_head<VD>(row + f.v_at + (size_t)kvh * f.vd, f.vd, nullptr, 0, 0, 0.0f, 0.0f, nullptr, 0, 0, kv_s + HD, lane,
+                                1.0f, f.values_are_keys ? conv : nullptr, ch, kept + ch, nullptr);
         }
         __syncthreads();
         if (owner && threadIdx.x < kChunks + kVChunks) {
@@ -631,10 +691,17 @@ decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restri
                     b_hi[j] = slope2 * (float)(pos - (k0 + r + 8));
                 }
             }
-            sv[0] = lo_ok ? sv[0] * scale2 - b_lo[0] : -INFINITY;
-            sv[1] = lo_ok ? sv[1] * scale2 - b_lo[1] : -INFINITY;
-            sv[2] = hi_ok ? sv[2] * scale2 - b_hi[0] : -INFINITY;
-            sv[3] = hi_ok ? sv[3] * scale2 - b_hi[1] : -INFINITY;
+            if (cap.out > 0.0f) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) sv[e] = capped_score(sv[e], cap);
+            } else {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) sv[e] *= scale2;
+            }
+            sv[0] = lo_ok ? sv[0] - b_lo[0] : -INFINITY;
+            sv[1] = lo_ok ? sv[1] - b_lo[1] : -INFINITY;
+            sv[2] = hi_ok ? sv[2] - b_hi[0] : -INFINITY;
+            sv[3] = hi_ok ? sv[3] - b_hi[1] : -INFINITY;
             float mx0 = fmaxf(sv[0], sv[2]), mx1 = fmaxf(sv[1], sv[3]);
 #pragma unroll
             for (int sh = 4; sh <= 16; sh <<= 1) {
@@ -719,8 +786,7 @@ decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restri
         if (n_splits == 1) {
             if (sinks != nullptr && ll > 0.0f) ll += exp2f(sinks[kvh * G + head] * kLog2e - mm);
             float res = ll > 0.0f ? oo / ll : 0.0f;
-            if (kFused && f.gate_at >= 0)
-                res *= 1.0f / (1.0f + expf(-f.qkv[(size_t)t * f.ld + f.gate_at + (size_t)(kvh * G + head) * vo + min(d, vo - 1)]));
+            if (gate.logits != nullptr) res *= out_gate(gate, t, kvh * G + head, vo, d);
             if (d < vo) out[out_row + (size_t)head * vo + d] = __float2bfloat16_rn(res);
         } else if (kCluster) {
             merged[head * W + d] = oo;
@@ -768,8 +834,7 @@ decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restri
             }
             if (sinks != nullptr && ll > 0.0f) ll += exp2f(sinks[kvh * G + head] * kLog2e - mm);
             float res = ll > 0.0f ? oo / ll : 0.0f;
-            if (kFused && f.gate_at >= 0)
-                res *= 1.0f / (1.0f + expf(-f.qkv[(size_t)t * f.ld + f.gate_at + (size_t)(kvh * G + head) * vo + min(d, vo - 1)]));
+            if (gate.logits != nullptr) res *= out_gate(gate, t, kvh * G + head, vo, d);
             if (d < vo) out[out_row + (size_t)head * vo + d] = __float2bfloat16_rn(res);
         }
         cluster_barrier_();   // no block leaves while its result may still be read
@@ -780,10 +845,10 @@ template <int HD, int VD>
 int launch_decode(const void* q, const void* k_pages, const void* v_pages, const int* block_table, int bt_stride,
                   const int* tok_seq, const int* tok_pos, void* out, float* scratch, int n_tok, int n_heads, int n_kv,
                   float scale, int window, int keep, int vo, int n_splits, cudaStream_t stream, const FusedQK* fused = nullptr,
-                  float slope_base = 0.0f, const float* sinks = nullptr) {
+                  float slope_base = 0.0f, const float* sinks = nullptr, float cap = 0.0f, const OutGate gate = OutGate{}) {
     using Kernel = void (*)(const __nv_bfloat16*, const __nv_bfloat16*, const __nv_bfloat16*, const int*, int, const int*,
                             const int*, __nv_bfloat16*, float*, float*, int, int, float, int, int, const FusedQK, const float*,
-                            int, int);
+                            int, int, const ScoreCap, const OutGate);
     // a block serves at most 16 heads of a key/value head: where more share one, kv_rep blocks take a part each
     int kv_rep = 1;
     while ((n_heads / n_kv) % kv_rep != 0 || n_heads / n_kv / kv_rep > 16) ++kv_rep;
@@ -824,14 +889,12 @@ int launch_decode(const void* q, const void* k_pages, const void* v_pages, const
     const cudaError_t e = cudaLaunchKernelEx(&cfg, kernel, (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pages,
                                              (const __nv_bfloat16*)v_pages, block_table, bt_stride, tok_seq, tok_pos,
                                              (__nv_bfloat16*)out, part_o, part_ml, n_heads, n_kv, scale * kLog2e, window, keep, f,
-                                             sinks, kv_rep, vo);
+                                             sinks, kv_rep, vo, score_cap(scale, cap), gate);
     NN_CHECK(e == cudaSuccess, "attention decode (%d splits%s): launch failed: %s", n_splits, cluster ? ", cluster" : "",
              cudaGetErrorString(e));
     if (n_splits > 1 && !cluster) {
-        const bool gated = fused && fused->gate_at >= 0;
-        merge_kernel<VD><<<dim3(n_heads, n_tok), VD, 0, stream>>>(
-            part_o, part_ml, (__nv_bfloat16*)out, n_heads, n_kv, n_splits, sinks,
-            gated ? f.qkv + f.gate_at : nullptr, gated ? (long)f.ld : 0l, vo);
+        merge_kernel<VD><<<dim3(n_heads, n_tok), VD, 0, stream>>>(part_o, part_ml, (__nv_bfloat16*)out, n_heads, n_kv, n_splits,
+                                                                  sinks, gate, vo);
         NN_LAUNCH_OK("attention merge");
     }
     return 0;
@@ -840,7 +903,8 @@ int launch_decode(const void* q, const void* k_pages, const void* v_pages, const
 template <int HD, int VD>
 int launch_prefill(const void* q, const void* k_pages, const void* v_pages, const int* block_table, int bt_stride,
                    const int* cu_seqlens, const int* tok_pos, void* out, int n_tok, int n_seqs, int n_heads, int n_kv,
-                   float scale, int window, int keep, int vo, float slope_base, const float* sinks, cudaStream_t stream) {
+                   float scale, int window, int keep, int vo, float slope_base, const float* sinks, float cap,
+                   const OutGate gate, cudaStream_t stream) {
     const int max_tiles = n_tok / 64 + n_seqs;
     constexpr int smem = 2 * kPage * (HD + VD) * 2;
     static bool configured[64] = {};
@@ -852,7 +916,7 @@ int launch_prefill(const void* q, const void* k_pages, const void* v_pages, cons
     prefill_kernel<HD, VD><<<grid, 128, smem, stream>>>((const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pages,
                                                  (const __nv_bfloat16*)v_pages, block_table, bt_stride, cu_seqlens,
                                                  tok_pos, (__nv_bfloat16*)out, n_seqs, n_heads, n_kv, scale * kLog2e,
-                                                 window, keep, slope_base, sinks, vo);
+                                                 window, keep, slope_base, sinks, vo, score_cap(scale, cap), gate);
     NN_LAUNCH_OK("attention prefill");
     return 0;
 }
@@ -881,9 +945,13 @@ extern "C" int nncpu_attention_decode_mma(const void* q, const void* k_pages, co
                                           const int* block_table, int bt_stride, const int* tok_seq,
                                           const int* tok_pos, void* out, float* scratch, long scratch_floats,
                                           int n_tok, int n_heads, int n_kv, int hd, int vp, int vo, float scale, int window,
-                                          int keep, int n_splits, float slope_base, const float* sinks, void* stream) {
+                                          int keep, int n_splits, float slope_base, const float* sinks, float cap,
+                                          const float* head_gate, int gate_ld, void* stream) {
     // pages of keys have rows of hd lanes, pages of values rows of vp; a head's output has vo lanes.  keep: with a
-    // window, the sequence's first keys that stay visible.
+    // window, the sequence's first keys that stay visible.  cap > 0: a scaled score z becomes cap tanh(z / cap).
+    // head_gate (or null): token t's n_heads logits at t * gate_ld, whose sigmoids multiply the heads' outputs.
+    NN_CHECK(cap >= 0.0f && (head_gate == nullptr || gate_ld >= n_heads), "attention decode: cap %f, gate rows of %d", cap, gate_ld);
+    const OutGate gate{head_gate, gate_ld, 1};
     NN_CHECK(nncpu_attention_mma_supported(n_heads, n_kv, hd),
              "attention (tensor cores): %d heads over %d key/value heads of size %d is not supported "
              "(head size 64 or 128, heads a multiple of key/value heads)", n_heads, n_kv, hd);
@@ -899,7 +967,8 @@ extern "C" int nncpu_attention_decode_mma(const void* q, const void* k_pages, co
     if (n_tok == 0) return 0;
 #define NN_DECODE(HD_, VD_)                                                                                                 \
     return launch_decode<HD_, VD_>(q, k_pages, v_pages, block_table, bt_stride, tok_seq, tok_pos, out, scratch, n_tok,      \
-                                   n_heads, n_kv, scale, window, keep, vo, n_splits, (cudaStream_t)stream, nullptr, slope_base, sinks)
+                                   n_heads, n_kv, scale, window, keep, vo, n_splits, (cudaStream_t)stream, nullptr, slope_base, sinks, \
+                                   cap, gate)
     if (hd == 64) NN_DECODE(64, 64);
     if (vp == 64) NN_DECODE(128, 64);
     NN_DECODE(128, 128);
@@ -922,7 +991,10 @@ extern "C" int nncpu_attention_decode_mma_from_qkv(const float* qkv, const void*
                                                    int head_dim, int v_head_dim, int whole_norm, int rot_half,
                                                    int rot_pairs, float scale, int window, int keep, int n_splits, float slope_base,
                                                    float temp_coef, int temp_every, const float* sinks,
-                                                   int values_are_keys, int gated, void* stream) {
+                                                   int values_are_keys, int gated, float cap, const float* conv_w, int taps,
+                                                   float* conv_state, long conv_stride, const int* seq_slots, void* stream) {
+    // gated: 1 a logit a lane of the output ends a token's row, 2 a logit a head, 0 none.  cap: as above.  conv_w (or null)
+    // [taps, C]: the short convolution over the C lanes of q and k, its state rows conv_stride floats apart.
     NN_CHECK(nncpu_attention_mma_supported(n_heads, n_kv, hd),
              "attention (tensor cores): %d heads over %d key/value heads of size %d is not supported "
              "(head size 64 or 128, heads a multiple of key/value heads)", n_heads, n_kv, hd);
@@ -954,12 +1026,18 @@ extern "C" int nncpu_attention_decode_mma_from_qkv(const float* qkv, const void*
     f.k_at = n_heads * head_dim;
     f.v_at = values_are_keys ? f.k_at : f.k_at + n_kv * head_dim;
     const int gate_at = n_heads * head_dim + (append ? n_kv * head_dim + (values_are_keys ? 0 : n_kv * v_head_dim) : 0);
-    f.ld = gate_at + (gated ? n_heads * v_head_dim : 0);
+    f.ld = gate_at + (gated == 1 ? n_heads * v_head_dim : gated == 2 ? n_heads : 0);
+    const OutGate gate{gated ? qkv + gate_at : nullptr, f.ld, gated == 2};
+    NN_CHECK(cap >= 0.0f && gated >= 0 && gated <= 2, "attention decode (from projections): cap %f, gate %d", cap, gated);
+    const int C = (n_heads + n_kv) * head_dim;
+    NN_CHECK(conv_w == nullptr || (append && taps >= 1 && conv_state != nullptr && seq_slots != nullptr && (conv_stride & 3) == 0 &&
+                                   conv_stride >= kConvHead + 2l * (taps - 1) * C && ((uintptr_t)conv_state % 16) == 0),
+             "attention decode (from projections): a convolution of %d taps over %d lanes, state rows of %ld", taps, C, conv_stride);
+    f.conv = ShortConv{conv_w, conv_state, seq_slots, conv_stride, taps, C};
     f.whole = whole_norm;
     f.half = rot_half;
     f.pairs = rot_pairs;
     f.values_are_keys = values_are_keys;
-    f.gate_at = gated ? gate_at : -1;
     f.q_gamma = q_gamma; f.k_gamma = k_gamma; f.g_dt = g_dt; f.eps = eps;
     f.cs = (const float2*)cos_sin;
     f.k_pages = append ? (__nv_bfloat16*)k_pages : nullptr;
@@ -970,7 +1048,8 @@ extern "C" int nncpu_attention_decode_mma_from_qkv(const float* qkv, const void*
     f.temp_every = temp_every;
 #define NN_DECODE(HD_, VD_)                                                                                                 \
     return launch_decode<HD_, VD_>(nullptr, k_pages, v_pages, block_table, bt_stride, tok_seq, tok_pos, out, scratch, n_tok, \
-                                   n_heads, n_kv, scale, window, keep, v_head_dim, n_splits, (cudaStream_t)stream, &f, 0.0f, sinks)
+                                   n_heads, n_kv, scale, window, keep, v_head_dim, n_splits, (cudaStream_t)stream, &f, 0.0f, sinks, \
+                                   cap, gate)
     if (hd == 64) NN_DECODE(64, 64);
     if (vp == 64) NN_DECODE(128, 64);
     NN_DECODE(128, 128);
@@ -983,16 +1062,19 @@ extern "C" int nncpu_attention_prefill_mma(const void* q, const void* k_pages, c
                                            const int* block_table, int bt_stride, const int* cu_seqlens,
                                            const int* tok_pos, void* out, int n_tok, int n_seqs, int n_heads,
                                            int n_kv, int hd, int vp, int vo, float scale, int window, int keep,
-                                           float slope_base, const float* sinks, void* stream) {
+                                           float slope_base, const float* sinks, float cap, const float* head_gate,
+                                           int gate_ld, void* stream) {
     NN_CHECK(nncpu_attention_mma_supported(n_heads, n_kv, hd),
              "attention (tensor cores): %d heads over %d key/value heads of size %d is not supported "
              "(head size 64 or 128, heads a multiple of key/value heads)", n_heads, n_kv, hd);
     NN_CHECK(n_tok >= 0 && n_seqs >= 0, "attention prefill: %d tokens of %d sequences", n_tok, n_seqs);
+    NN_CHECK(cap >= 0.0f && (head_gate == nullptr || gate_ld >= n_heads), "attention prefill: cap %f, gate rows of %d", cap, gate_ld);
+    const OutGate gate{head_gate, gate_ld, 1};
     NN_CHECK(value_size_ok(hd, vp, vo) && keep >= 0, "attention prefill: value rows of %d lanes, %d of them used", vp, vo);
     if (n_tok == 0 || n_seqs == 0) return 0;
 #define NN_PREFILL(HD_, VD_)                                                                                                \
     return launch_prefill<HD_, VD_>(q, k_pages, v_pages, block_table, bt_stride, cu_seqlens, tok_pos, out, n_tok, n_seqs,   \
-                                    n_heads, n_kv, scale, window, keep, vo, slope_base, sinks, (cudaStream_t)stream)
+                                    n_heads, n_kv, scale, window, keep, vo, slope_base, sinks, cap, gate, (cudaStream_t)stream)
     if (hd == 64) NN_PREFILL(64, 64);
     if (vp == 64) NN_PREFILL(128, 64);
     NN_PREFILL(128, 128);
@@ -1076,5 +1158,6 @@ extern "C" int nncpu_attention_decode_mma_static(const void* q, const void* k_pa
     float* scratch = nullptr;
     if (int e = static_scratch(&scratch)) return e;
     return nncpu_attention_decode_mma(q, k_pages, v_pages, block_table, bt_stride, tok_seq, tok_pos, out, scratch,
-                                      kStaticScratchFloats, n_tok, n_heads, n_kv, hd, hd, hd, scale, window, 0, n_splits, 0.0f, nullptr, stream);
+                                      kStaticScratchFloats, n_tok, n_heads, n_kv, hd, hd, hd, scale, window, 0, n_splits, 0.0f, nullptr,
+                                      0.0f, nullptr, 0, stream);
 }

@@ -66,6 +66,12 @@ struct AttnParams {
     int vo;         // lanes of a head in the output (at most the value rows' VD)
     float slope_base;   // b != 0: head h takes 2^(-b (h + 1) / n_heads) * (query position - key position) off its scaled scores
     const float* sinks; // float32 [n_heads] or null: exp(sinks[h]) joins the denominator of head h's softmax, with no key and no value
+    // The weight of a key is 2^(u score_mul + score_add - m): without a cap u is the unscaled score, score_mul = scale2 and
+    // score_add = 0.  With a cap c (kCap) the score is c tanh(z / c) = c - 2 c / (1 + exp(2 z / c)), so
+    // u = -1 / (1 + 2^(cap_in * unscaled score)), score_mul = 2 c log2(e) and score_add = c log2(e).
+    float cap_in, score_mul, score_add;
+    const float* head_gate;   // or null: row t (at t * gate_ld) holds a logit a head, whose sigmoid multiplies the head's output
+    long gate_ld;
     int* status;
 };
 
@@ -95,6 +101,12 @@ __device__ __forceinline__ float fast_exp2(float x) {
     return y;
 }
 
+__device__ __forceinline__ float fast_rcp(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
 __device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
     const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
     return *reinterpret_cast<const uint32_t*>(&h);
@@ -113,7 +125,7 @@ __device__ __forceinline__ void umma_bf16_ts(uint32_t tmem_d, uint32_t tmem_a, u
 }
 
 // Threads: warp 0 producer, warp 1 tensor-core issue and tensor memory, then one warpgroup per head.
-template <int HD, int VD, int kStreams>
+template <int HD, int VD, int kStreams, bool kCap>
 __global__ void __launch_bounds__(64 + 128 * kStreams, 1)
 prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                   const __grid_constant__ CUtensorMap map_v, const AttnParams p) {
@@ -375,6 +387,13 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
                     for (int c = 0; c < 64; ++c)
                         u[c] = __float_as_uint(fmaf(bias_per_key, (float)c - far, __uint_as_float(u[c])));
                 }
+                if (kCap) {
+#pragma unroll
+                    for (int c = 0; c < 64; ++c) {
+                        const float e = fast_exp2(__uint_as_float(u[c]) * p.cap_in);
+                        u[c] = __float_as_uint(fast_rcp(-1.0f - e));
+                    }
+                }
                 if (!((kb >= lim_lo || kb + 63 < p.keep) && kb + 63 <= lim_hi)) {
                     // the page crosses this row's limits
 #pragma unroll
@@ -383,7 +402,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
                 }
             };
             auto weights = [&]() {
-                const float neg_m = m_ref == -INFINITY ? 0.0f : 0.0f - m_ref;
+                const float neg_m = m_ref == -INFINITY ? 0.0f : (kCap ? p.score_add : 0.0f) - m_ref;
                 float sm[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
                 for (int hf = 0; hf < 2; ++hf) {
@@ -392,8 +411,8 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
                         load_half(hf, u);
 #pragma unroll
                         for (int c = 0; c < 64; c += 2) {
-                            const float e0 = fast_exp2(fmaf(__uint_as_float(u[c]), p.scale2, neg_m));
-                            const float e1 = fast_exp2(fmaf(__uint_as_float(u[c + 1]), p.scale2, neg_m));
+                            const float e0 = fast_exp2(fmaf(__uint_as_float(u[c]), p.score_mul, neg_m));
+                            const float e1 = fast_exp2(fmaf(__uint_as_float(u[c + 1]), p.score_mul, neg_m));
                             sm[c & 3] += e0;
                             sm[(c & 3) + 1] += e1;
                             w[hf][c >> 1] = pack_bf16(e0, e1);
@@ -415,7 +434,8 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
                         for (int c = 0; c < 64; ++c) mx[c & 3] = fmaxf(mx[c & 3], __uint_as_float(u[c]));
                     }
                 }
-                const float tmax = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * p.scale2;   // the scale is positive
+                const float tmax = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * p.score_mul
+                                   + (kCap ? p.score_add : 0.0f);                                // the factor is positive
                 float alpha = 1.0f;
                 if (tmax > m_ref) {
                     alpha = fast_exp2(m_ref - tmax);    // 0 when nothing was seen yet
@@ -449,7 +469,9 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             // the sink's term, in the unit of the row's sums: powers of two relative to the reference maximum
             if (p.sinks != nullptr && l > 0.0f) l += exp2f(p.sinks[h] * 1.4426950408889634f - m_ref);
-            const float inv = l > 0.0f ? 1.0f / l : 0.0f;
+            float inv = l > 0.0f ? 1.0f / l : 0.0f;
+            if (p.head_gate != nullptr && row < n_rows)
+                inv *= 1.0f / (1.0f + expf(-p.head_gate[(size_t)(q0 + row) * p.gate_ld + h]));
             __nv_bfloat16* dst = p.out + ((size_t)(q0 + row) * p.n_heads + h) * p.vo;
 #pragma unroll 1
             for (int c0 = 0; c0 < VD; c0 += 32) {
@@ -533,13 +555,13 @@ struct MapCache {
 
 MapCache g_maps;
 
-template <int HD, int VD, int kStreams>
-int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const AttnParams& p, int n_tok,
+template <int HD, int VD, int kStreams, bool kCap>
+int launch_one(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const AttnParams& p, int n_tok,
            cudaStream_t stream) {
     constexpr int smem = kStreams * kQRows * HD * 2 + kStages * kKeys * (HD + VD) * 2 + 256 + 1024;
     static bool configured[64] = {};
     if (first_use_on_this_device(configured)) {
-        const cudaError_t e = cudaFuncSetAttribute(prefill_tc_kernel<HD, VD, kStreams>,
+        const cudaError_t e = cudaFuncSetAttribute(prefill_tc_kernel<HD, VD, kStreams, kCap>,
                                                    cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         NN_CHECK(e == cudaSuccess, "attention (tensor cores): %d bytes of shared memory refused: %s", smem,
                  cudaGetErrorString(e));
@@ -555,9 +577,16 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, 
     cudaLaunchAttribute attr[1];
     cfg.attrs = attr;
     cfg.numAttrs = overlap_attribute(attr);
-    const cudaError_t e = cudaLaunchKernelEx(&cfg, prefill_tc_kernel<HD, VD, kStreams>, mq, mk, mv, p);
+    const cudaError_t e = cudaLaunchKernelEx(&cfg, prefill_tc_kernel<HD, VD, kStreams, kCap>, mq, mk, mv, p);
     NN_CHECK(e == cudaSuccess, "attention prefill (tensor cores): launch failed: %s", cudaGetErrorString(e));
     return 0;
+}
+
+template <int HD, int VD, int kStreams>
+int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const AttnParams& p, int n_tok,
+           cudaStream_t stream) {
+    return p.cap_in != 0.0f ? launch_one<HD, VD, kStreams, true>(mq, mk, mv, p, n_tok, stream)
+                            : launch_one<HD, VD, kStreams, false>(mq, mk, mv, p, n_tok, stream);
 }
 
 }  // namespace
@@ -569,12 +598,15 @@ extern "C" int nncpu_attention_prefill_tc_supported(int n_heads, int n_kv, int h
 // q: bfloat16 [n_tok, n_heads * head_dim], out: bfloat16 [n_tok, n_heads * vo]; K and V pages: bfloat16 [n_pages, n_kv,
 // 64, head_dim] and [n_pages, n_kv, 64, vp] holding every key the new tokens may see, their own included; keep: with a
 // window, the sequence's first keys that stay visible; cu_seqlens [n_seqs + 1] row ranges of the sequences;
-// tok_pos [n_tok] positions (consecutive within a sequence).  *status receives a code if a wait runs out.
+// tok_pos [n_tok] positions (consecutive within a sequence); cap > 0: a scaled score z becomes cap tanh(z / cap) (not
+// together with a distance bias); head_gate (or null): token t's n_heads logits at t * gate_ld, whose sigmoids multiply the
+// heads' outputs.  *status receives a code if a wait runs out.
 extern "C" int nncpu_attention_prefill_tc(const void* q, const void* k_pages, const void* v_pages, int n_pages,
                                           const int* block_table, int bt_stride, const int* cu_seqlens,
                                           const int* tok_pos, void* out, int n_tok, int n_seqs, int n_heads, int n_kv,
                                           int head_dim, int vp, int vo, float scale, int window, int keep,
-                                          float slope_base, const float* sinks, int* status, void* stream_) {
+                                          float slope_base, const float* sinks, float cap, const float* head_gate,
+                                          int gate_ld, int* status, void* stream_) {
     NN_CHECK(nncpu_attention_prefill_tc_supported(n_heads, n_kv, head_dim),
              "attention (tensor cores): head size %d with %d heads over %d key/value heads is not supported "
              "(head size 64 or 128, heads a multiple of key/value heads)", head_dim, n_heads, n_kv);
@@ -585,6 +617,8 @@ extern "C" int nncpu_attention_prefill_tc(const void* q, const void* k_pages, co
     NN_CHECK(((uintptr_t)q % 16) == 0 && ((uintptr_t)k_pages % 16) == 0 && ((uintptr_t)v_pages % 16) == 0 &&
              ((uintptr_t)out % 16) == 0, "attention (tensor cores): operands must be 16-byte aligned");
     NN_CHECK(status != nullptr, "attention (tensor cores): no status word");
+    NN_CHECK(cap >= 0.0f && (cap == 0.0f || slope_base == 0.0f) && (head_gate == nullptr || gate_ld >= n_heads),
+             "attention (tensor cores): cap %f with a distance bias of %f, gate rows of %d", cap, slope_base, gate_ld);
     if (n_tok == 0 || n_seqs == 0) return 0;
     CUtensorMap mq, mk, mv;
     if (int e = g_maps.get(&mq, q, n_tok, (long)n_heads * head_dim, 0, 0)) return e;
@@ -605,6 +639,12 @@ extern "C" int nncpu_attention_prefill_tc(const void* q, const void* k_pages, co
     p.vo = vo;
     p.slope_base = slope_base;
     p.sinks = sinks;
+    const ScoreCap sc = score_cap(scale, cap);
+    p.cap_in = sc.in;
+    p.score_mul = cap > 0.0f ? 2.0f * sc.out : p.scale2;
+    p.score_add = sc.out;
+    p.head_gate = head_gate;
+    p.gate_ld = gate_ld;
     p.status = status;
     cudaStream_t stream = (cudaStream_t)stream_;
     // two heads to a block where a key/value head has two to give; one head per block otherwise

@@ -55,6 +55,15 @@ __device__ __forceinline__ float ld_f(const void* p, size_t i, int dt) {
                         : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p)[i]);
 }
 
+// Four neighbouring elements from i on (a multiple of 4; 16-byte aligned rows).
+__device__ __forceinline__ float4 ld_f4(const void* p, size_t i, int dt) {
+    if (dt == DT_F32) return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p) + i);
+    const uint2 u = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(p) + i);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+
 __device__ __forceinline__ void st_f(void* p, size_t i, int dt, float v) {
     if (dt == DT_F32) reinterpret_cast<float*>(p)[i] = v;
     else reinterpret_cast<__nv_bfloat16*>(p)[i] = __float2bfloat16_rn(v);
@@ -190,6 +199,49 @@ struct PageWalk {
     }
     __device__ __forceinline__ int page(int i) const { return i < n_kept ? i : lo + i - n_kept; }
 };
+
+// A short causal convolution over time, channel by channel: y_t = sum_j w[j] u_(t - taps + 1 + j).  The last taps - 1 inputs
+// u of a sequence are per-sequence state.  A slot's row of the state area holds two copies of them ([taps - 1, C] floats,
+// oldest first) behind a head of kConvHead words, the first two of which say after how many tokens each copy was taken.
+// The copy in use is the one whose number is the position at which the step starts; a step writes the OTHER copy, so
+// that every block of a kernel may read the old inputs while others leave the new ones.  A sequence that starts finds
+// zeros: both copies then stand for position 0.
+constexpr int kConvHead = 4;
+struct ShortConv {
+    const float* w;     // [taps, C], the last row is the current token's; null: no convolution
+    float* state;       // [slots, stride]
+    const int* seq_slots;
+    long stride;
+    int taps, C;
+};
+__device__ __forceinline__ int conv_copy_in_use(const ShortConv& c, int slot, int start) {
+    return __float_as_int(c.state[(size_t)slot * c.stride]) == start ? 0 : 1;
+}
+__device__ __forceinline__ float* conv_copy(const ShortConv& c, int slot, int which) {
+    return c.state + (size_t)slot * c.stride + kConvHead + (size_t)which * (c.taps - 1) * c.C;
+}
+__device__ __forceinline__ void conv_mark(const ShortConv& c, int slot, int which, int length) {
+    c.state[(size_t)slot * c.stride + which] = __int_as_float(length);
+}
+
+// A score's cap: c tanh(z / c) with z = raw * scale, in the tensor-core attention kernels' unit (powers of two). With
+// in = 2 scale log2(e) / c and out = c log2(e), log2(e) c tanh(raw scale / c) = out - 2 out / (1 + 2^(raw in)): a power of
+// two and a reciprocal, whose error (some 1e-7 of the cap) does not grow with the score.  out 0: no cap.
+struct ScoreCap {
+    float in, out;
+};
+__host__ __device__ __forceinline__ ScoreCap score_cap(float scale, float cap) {
+    ScoreCap c;
+    c.in = cap > 0.0f ? 2.0f * scale * 1.4426950408889634f / cap : 0.0f;
+    c.out = cap > 0.0f ? cap * 1.4426950408889634f : 0.0f;
+    return c;
+}
+__device__ __forceinline__ float capped_score(float raw, const ScoreCap& c) {
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(raw * c.in));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+    return fmaf(-2.0f * c.out, r, c.out);
+}
 
 // Gated activations act(gate) * up of the feed-forwards, on 32-bit values.  kGateSilu: silu(g) u.  kGateGeluTanh: the
 // tanh form of GELU, g/2 (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))) u.  kGateSwishClamp: with g' = min(g, limit) and

@@ -714,6 +714,225 @@ extern "C" int nncpu_qk_whole_norm_append(const float* qkv, int ld, const void* 
 }
 
 // ---------------------------------------------------------------------------
+// The same step for mixers with a short convolution over time on every channel of q and k (common.cuh: ShortConv) and
+// values that are the keys: proj float32 [n_tok, ld] holds the heads of q and of k (hd lanes each).  Per head: the
+// convolution; a key head's result is the position's value as it is; then the RMS norm per head (weights [hd]) and the
+// rotation of the first `half` pairs (2 i, 2 i + 1).  A head lies in q_out and in the pages in rows of qp and vp lanes, zeros
+// behind its own.  A warp takes one head of kConvRun consecutive tokens and keeps the last taps - 1 inputs in registers
+// (kTaps 0: any number of taps, read again for every token).  It also leaves the sequence's last inputs as the state.
+// kVec: a head is a multiple of kEpl lanes and so is a row.
+// ---------------------------------------------------------------------------
+constexpr int kConvRun = 8;
+
+template <int kEpl, bool kVec>
+__device__ __forceinline__ void ld_lanes(const float* __restrict__ row, int lane, int n, float (&x)[kEpl]) {
+    if (kVec && kEpl == 4) {
+        const float4 v = lane * 4 < n ? reinterpret_cast<const float4*>(row)[lane] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        x[0] = v.x; x[1 % kEpl] = v.y; x[2 % kEpl] = v.z; x[3 % kEpl] = v.w;
+    } else if (kVec && kEpl == 2) {
+        const float2 v = lane * 2 < n ? reinterpret_cast<const float2*>(row)[lane] : make_float2(0.0f, 0.0f);
+        x[0] = v.x; x[1 % kEpl] = v.y;
+    } else {
+#pragma unroll
+        for (int e = 0; e < kEpl; ++e) x[e] = lane * kEpl + e < n ? row[lane * kEpl + e] : 0.0f;
+    }
+}
+
+template <int kEpl, bool kVec>
+__device__ __forceinline__ void st_lanes(float* __restrict__ row, int lane, int n, const float (&x)[kEpl]) {
+    if (kVec && kEpl == 4) {
+        if (lane * 4 < n) reinterpret_cast<float4*>(row)[lane] = make_float4(x[0], x[1 % kEpl], x[2 % kEpl], x[3 % kEpl]);
+    } else if (kVec && kEpl == 2) {
+        if (lane * 2 < n) reinterpret_cast<float2*>(row)[lane] = make_float2(x[0], x[1 % kEpl]);
+    } else {
+#pragma unroll
+        for (int e = 0; e < kEpl; ++e)
+            if (lane * kEpl + e < n) row[lane * kEpl + e] = x[e];
+    }
+}
+
+// A head's lanes to a row of `size` elements (zeros behind the head's own are in x already).
+template <int kEpl>
+__device__ __forceinline__ void st_row(void* __restrict__ dst, size_t at, int dt, int size, int lane, const float (&x)[kEpl]) {
+    if (dt == DT_BF16 && size == 32 * kEpl && kEpl <= 4) {
+        __nv_bfloat16* p = reinterpret_cast<__nv_bfloat16*>(dst) + at + lane * kEpl;
+        if (kEpl == 4) {
+            __nv_bfloat162 h[2] = {__floats2bfloat162_rn(x[0], x[1 % kEpl]), __floats2bfloat162_rn(x[2 % kEpl], x[3 % kEpl])};
+            *reinterpret_cast<uint2*>(p) = *reinterpret_cast<uint2*>(h);
+        } else {
+            *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(x[0], x[1 % kEpl]);
+        }
+        return;
+    }
+#pragma unroll
+    for (int e = 0; e < kEpl; ++e)
+        if (lane * kEpl + e < size) st_f(dst, at + lane * kEpl + e, dt, x[e]);
+}
+
+template <int kEpl, int kTaps, bool kVec>
+__global__ void __launch_bounds__(256)
+qk_conv_norm_append_kernel(const float* __restrict__ proj, int ld, const ShortConv cv, const int* __restrict__ cu_seqlens,
+                           const void* __restrict__ q_gamma, const void* __restrict__ k_gamma, int g_dt, float eps,
+                           const float2* __restrict__ cs, int half, const int* __restrict__ tok_seq,
+                           const int* __restrict__ tok_pos, const int* __restrict__ block_table, int bt_stride,
+                           void* __restrict__ k_pages, void* __restrict__ v_pages, int kv_dt, void* __restrict__ q_out,
+                           int q_dt, int n_tok, int n_heads, int n_kv, int hd, int qp, int vp) {
+    constexpr int kKeep = kTaps > 1 ? kTaps - 1 : 1;
+    const int lane = threadIdx.x & 31;
+    const long item = (long)blockIdx.x * 8 + (threadIdx.x >> 5);
+    const int n_rows = n_heads + n_kv;                  // heads of a token; warps of a block share tokens
+    const int h = (int)(item % n_rows);
+    const long t0l = item / n_rows * kConvRun;
+    if (t0l >= n_tok) return;
+    const int t0 = (int)t0l, taps = kTaps > 0 ? kTaps : cv.taps, ch0 = h * hd;
+    const bool is_q = h < n_heads;
+    const void* gamma = is_q ? q_gamma : k_gamma;
+    float w[kTaps > 0 ? kTaps : 1][kEpl], win[kKeep][kEpl], u[kTaps > 0 ? kConvRun : 1][kEpl];
+    if (kTaps > 0) {
+#pragma unroll
+        for (int i = 0; i < kConvRun; ++i)              // all the inputs are asked for before the first is used
+            if (t0 + i < n_tok) ld_lanes<kEpl, kVec>(proj + (size_t)(t0 + i) * ld + ch0, lane, hd, u[kTaps > 0 ? i : 0]);
+#pragma unroll
+        for (int j = 0; j < kTaps; ++j) ld_lanes<kEpl, kVec>(cv.w + (size_t)j * cv.C + ch0, lane, hd, w[j]);
+    }
+    float g[kEpl];
+#pragma unroll
+    for (int e = 0; e < kEpl; ++e) g[e] = gamma != nullptr && lane * kEpl + e < hd ? ld_f(gamma, lane * kEpl + e, g_dt) : 1.0f;
+    int seq = -1, first = 0, end = 0, slot = 0, copy = 0;
+#pragma unroll
+    for (int i = 0; i < kConvRun; ++i) {
+        const int t = t0 + i;
+        if (t >= n_tok) break;
+        const int s = tok_seq[t];
+        if (s < 0) { seq = -1; continue; }              // padding: nobody reads its query, and it has no place in the cache
+        const bool entered = s != seq;
+        if (entered) {
+            seq = s;
+            first = cu_seqlens[s];
+            end = cu_seqlens[s + 1];
+            slot = cv.seq_slots[s];
+            copy = conv_copy_in_use(cv, slot, tok_pos[first]);
+        }
+        const float* kept = conv_copy(cv, slot, copy);
+        float* next = conv_copy(cv, slot, 1 - copy);
+        // the input that lies `back` tokens before t
+        auto earlier = [&](int back, float (&x)[kEpl]) {
+            const int at = t - back;
+            ld_lanes<kEpl, kVec>(at >= first ? proj + (size_t)at * ld + ch0
+                                             : kept + (size_t)(taps - 1 + at - first) * cv.C + ch0, lane, hd, x);
+        };
+        float x[kEpl], now[kEpl];
+        if (kTaps > 0) {
+            if (entered) {
+#pragma unroll
+                for (int j = 0; j + 1 < kTaps; ++j) earlier(kTaps - 1 - j, win[j]);
+            }
+#pragma unroll
+            for (int e = 0; e < kEpl; ++e) {
+                now[e] = u[kTaps > 0 ? i : 0][e];
+                float a = 0.0f;
+#pragma unroll
+                for (int j = 0; j + 1 < kTaps; ++j) a = fmaf(w[j][e], win[j][e], a);
+                x[e] = fmaf(w[kTaps > 0 ? kTaps - 1 : 0][e], now[e], a);
+#pragma unroll
+                for (int j = 0; j + 2 < kTaps; ++j) win[j][e] = win[j + 1][e];
+                win[kKeep - 1][e] = now[e];
+            }
+        } else {
+            ld_lanes<kEpl, kVec>(proj + (size_t)t * ld + ch0, lane, hd, now);
+#pragma unroll
+            for (int e = 0; e < kEpl; ++e) x[e] = 0.0f;
+            for (int j = 0; j < taps; ++j) {
+                float wj[kEpl], uj[kEpl];
+                ld_lanes<kEpl, kVec>(cv.w + (size_t)j * cv.C + ch0, lane, hd, wj);
+                earlier(taps - 1 - j, uj);
+#pragma unroll
+                for (int e = 0; e < kEpl; ++e) x[e] = fmaf(wj[e], uj[e], x[e]);
+            }
+        }
+        // the state after this step: its last taps - 1 inputs, older ones moved up where the step has fewer
+        if (t >= end - (taps - 1)) st_lanes<kEpl, kVec>(next + (size_t)(t - (end - (taps - 1))) * cv.C + ch0, lane, hd, now);
+        if (t == first) {
+            for (int j = 0; j < taps - 1 - (end - first); ++j) {
+                float old[kEpl];
+                ld_lanes<kEpl, kVec>(kept + (size_t)(j + end - first) * cv.C + ch0, lane, hd, old);
+                st_lanes<kEpl, kVec>(next + (size_t)j * cv.C + ch0, lane, hd, old);
+            }
+        }
+        if (t == end - 1 && h == 0 && lane == 0 && taps > 1) conv_mark(cv, slot, 1 - copy, tok_pos[t] + 1);
+
+        const int pos = tok_pos[t];
+        const int page = is_q ? 0 : block_table[(size_t)s * bt_stride + pos / kPage];
+        const size_t row = is_q ? (size_t)t * n_heads + h : ((size_t)page * n_kv + (h - n_heads)) * kPage + pos % kPage;
+        if (!is_q && page >= 0) st_row<kEpl>(v_pages, row * vp, kv_dt, vp, lane, x);
+        if (gamma != nullptr) {
+            float ss = 0.0f;
+#pragma unroll
+            for (int e = 0; e < kEpl; ++e) ss = fmaf(x[e], x[e], ss);
+            const float scale = 1.0f / sqrtf(warp_sum(ss) * (1.0f / (float)hd) + eps);
+#pragma unroll
+            for (int e = 0; e < kEpl; ++e) x[e] = (x[e] * scale) * g[e];
+        }
+        if (cs != nullptr) {
+#pragma unroll
+            for (int e = 0; e < kEpl; e += 2) {
+                const int p = (lane * kEpl + e) >> 1;
+                if (p < half) {
+                    const float2 c = cs[(size_t)t * half + p];
+                    const float a = x[e], b = x[e + 1];
+                    x[e] = c.x * a - c.y * b;
+                    x[e + 1] = c.y * a + c.x * b;
+                }
+            }
+        }
+        if (is_q) st_row<kEpl>(q_out, row * qp, q_dt, qp, lane, x);
+        else if (page >= 0) st_row<kEpl>(k_pages, row * qp, kv_dt, qp, lane, x);
+    }
+}
+
+// Floats of a slot's state row for a convolution of `taps` taps over C channels.
+extern "C" long nncpu_conv_state_floats(int taps, int C) { return kConvHead + ((2l * (taps - 1) * C + 3) & ~3l); }
+
+extern "C" int nncpu_qk_conv_norm_append(const float* proj, int ld, const float* conv_w, int taps, float* state, long stride,
+                                         const int* seq_slots, const int* cu_seqlens, const void* q_gamma,
+                                         const void* k_gamma, int g_dt, float eps, const float* cs, int half,
+                                         const int* tok_seq, const int* tok_pos, const int* block_table, int bt_stride,
+                                         void* k_pages, void* v_pages, int kv_dt, void* q_out, int q_dt, int n_tok,
+                                         int n_heads, int n_kv, int hd, int qp, int vp, void* stream) {
+    NN_CHECK(n_tok >= 0 && n_heads > 0 && n_kv > 0 && hd > 0 && hd <= 1024 && qp >= hd && vp >= hd && qp <= 1024 && vp <= qp,
+             "q/k convolution and append: %d and %d heads of %d lanes in rows of %d and %d", n_heads, n_kv, hd, qp, vp);
+    const int C = (n_heads + n_kv) * hd;
+    NN_CHECK(taps >= 1 && ld >= C && stride >= nncpu_conv_state_floats(taps, C) && (stride & 3) == 0,
+             "q/k convolution: %d taps over %d channels, rows of %d, state rows of %ld", taps, C, ld, stride);
+    NN_CHECK(cs == nullptr || 2 * half <= hd, "q/k convolution and append: %d rotated pairs of a head of %d lanes", half, hd);
+    NN_CHECK((uintptr_t)cs % 8 == 0 && (uintptr_t)state % 16 == 0, "q/k convolution: the rotation table and the state must be aligned");
+    if (n_tok == 0) return 0;
+    const ShortConv cv{conv_w, state, seq_slots, stride, taps, C};
+    const long items = (long)((n_tok + kConvRun - 1) / kConvRun) * (n_heads + n_kv);
+    const unsigned blocks = (unsigned)((items + 7) / 8);
+#define NN_QK(E, T, V)                                                                                                     \
+    qk_conv_norm_append_kernel<E, T, V><<<blocks, 256, 0, (cudaStream_t)stream>>>(                                         \
+        proj, ld, cv, cu_seqlens, q_gamma, k_gamma, g_dt, eps, (const float2*)cs, half, tok_seq, tok_pos, block_table,     \
+        bt_stride, k_pages, v_pages, kv_dt, q_out, q_dt, n_tok, n_heads, n_kv, hd, qp, vp)
+    const int epl = qp <= 64 ? 2 : qp <= 128 ? 4 : 32;
+    const bool vec = epl <= 4 && hd % epl == 0 && ld % epl == 0 && ((uintptr_t)proj % 16) == 0 && ((uintptr_t)conv_w % 16) == 0;
+    if (epl == 32) NN_QK(32, 0, false);
+    else if (!vec && epl == 4) NN_QK(4, 0, false);
+    else if (!vec) NN_QK(2, 0, false);
+    else if (epl == 4 && taps == 2) NN_QK(4, 2, true);
+    else if (epl == 4 && taps == 3) NN_QK(4, 3, true);
+    else if (epl == 4 && taps == 4) NN_QK(4, 4, true);
+    else if (epl == 4) NN_QK(4, 0, true);
+    else if (taps == 2) NN_QK(2, 2, true);
+    else if (taps == 3) NN_QK(2, 3, true);
+    else if (taps == 4) NN_QK(2, 4, true);
+    else NN_QK(2, 0, true);
+#undef NN_QK
+    NN_LAUNCH_OK("q/k convolution and append");
+    return 0;
+}
+
+// ---------------------------------------------------------------------------
 // Attention of every (token, head) over the cache of the token's sequence:
 // keys first..pos with first = first_visible_key(pos, window): a sliding window (window > 0), blocks of
 // -window positions (window < 0) or every earlier key (0); with a window the sequence's first `keep` keys too.
@@ -723,7 +942,8 @@ extern "C" int nncpu_qk_whole_norm_append(const float* qkv, int ld, const void* 
 // Values have vd lanes a head in their pages and vo (at most vd) in the output.  With slope_base != 0 head h
 // takes slope_h * (pos - key) off its scaled scores, slope_h = 2^(-slope_base (h + 1) / n_heads).
 // With sinks (float32 [n_heads]) the softmax's denominator of head h also holds exp(sinks[h]): a term without
-// key or value, not scaled, counted once.
+// key or value, not scaled, counted once.  With cap != 0 a scaled score z becomes cap tanh(z / cap).  With head_gate
+// (float32, row t at t * gate_ld) head h's output is multiplied by sigmoid(head_gate[t, h]).
 // ---------------------------------------------------------------------------
 constexpr int kAttnThreads = 128;
 
@@ -732,7 +952,8 @@ attention_kernel(const void* __restrict__ q, int q_dt, const void* __restrict__ 
                  const void* __restrict__ v_pages, int kv_dt, const int* __restrict__ block_table, int bt_stride,
                  const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, void* __restrict__ out,
                  int out_dt, int n_heads, int n_kv, int hd, int vd, int vo, float scale, int window, int keep,
-                 float slope_base, const float* __restrict__ sinks) {
+                 float slope_base, const float* __restrict__ sinks, float cap, const float* __restrict__ head_gate,
+                 int gate_ld) {
     extern __shared__ float smem[];
     float* qs = smem;                       // hd
     float* p = smem + hd;                   // kAttnThreads
@@ -771,7 +992,9 @@ attention_kernel(const void* __restrict__ q, int q_dt, const void* __restrict__ 
             off = ((long long)page * n_kv + kvh) * kPage + key % kPage;      // the key's row in its pages
             float dot = 0.0f;
             for (int d = 0; d < hd; ++d) dot = fmaf(qs[d], ld_f(k_pages, (size_t)off * hd + d, kv_dt), dot);
-            s = dot * scale - slope * (float)(pos - key);
+            s = dot * scale;
+            if (cap != 0.0f) s = cap * tanhf(s / cap);
+            s -= slope * (float)(pos - key);
         }
         const float m_new = fmaxf(m, block_max(s, scratch));
         const float w = has_key ? expf(s - m_new) : 0.0f;
@@ -794,7 +1017,8 @@ attention_kernel(const void* __restrict__ q, int q_dt, const void* __restrict__ 
         __syncthreads();
     }
     if (sinks != nullptr) l += expf(sinks[h] - m);      // the maximum is that of the keys: a query sees itself at least
-    const float inv = l > 0.0f ? 1.0f / l : 0.0f;
+    float inv = l > 0.0f ? 1.0f / l : 0.0f;
+    if (head_gate != nullptr) inv *= 1.0f / (1.0f + expf(0.0f - head_gate[(size_t)t * gate_ld + h]));
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
         const int d = tid + kAttnThreads * j;
@@ -805,9 +1029,11 @@ attention_kernel(const void* __restrict__ q, int q_dt, const void* __restrict__ 
 extern "C" int nncpu_attention(const void* q, int q_dt, const void* k_pages, const void* v_pages, int kv_dt,
                                const int* block_table, int bt_stride, const int* tok_seq, const int* tok_pos,
                                void* out, int out_dt, int n_tok, int n_heads, int n_kv, int hd, int vd, int vo, float scale,
-                               int window, int keep, float slope_base, const float* sinks, void* stream) {
+                               int window, int keep, float slope_base, const float* sinks, float cap,
+                               const float* head_gate, int gate_ld, void* stream) {
     NN_CHECK(n_tok >= 0 && n_heads > 0 && n_kv > 0 && n_heads % n_kv == 0,
              "attention: %d heads over %d key/value heads", n_heads, n_kv);
+    NN_CHECK(cap >= 0.0f && (head_gate == nullptr || gate_ld >= n_heads), "attention: cap %f, gate rows of %d", cap, gate_ld);
     NN_CHECK(hd > 0 && hd <= 1024, "attention: head size %d must be positive and at most 1024", hd);
     NN_CHECK(vd > 0 && vd <= 1024, "attention: value size %d must be positive and at most 1024", vd);
     NN_CHECK(vo > 0 && vo <= vd && keep >= 0, "attention: %d lanes of values of %d, %d kept keys", vo, vd, keep);
@@ -817,7 +1043,8 @@ extern "C" int nncpu_attention(const void* q, int q_dt, const void* k_pages, con
     attention_kernel<<<grid, kAttnThreads, smem, (cudaStream_t)stream>>>(q, q_dt, k_pages, v_pages, kv_dt,
                                                                          block_table, bt_stride, tok_seq, tok_pos,
                                                                          out, out_dt, n_heads, n_kv, hd, vd, vo, scale,
-                                                                         window, keep, slope_base, sinks);
+                                                                         window, keep, slope_base, sinks, cap, head_gate,
+                                                                         gate_ld);
     NN_LAUNCH_OK("attention");
     return 0;
 }
@@ -2188,12 +2415,66 @@ __device__ __forceinline__ void route_top_sigmoid(float* z, int n_experts, int t
     }
 }
 
-constexpr int kScoresChosen = 0, kScoresAll = 1, kScoresSigmoid = 2;
+// Scores over all experts, s = softmax(z), chosen by s + corr (float32 or bfloat16, one per expert; null: by s alone) and
+// weighted by s itself, times `scale`: not renormalised.  One warp; z is overwritten; sbuf holds n_experts floats.
+__device__ __forceinline__ void route_top_plain(float* z, float* sbuf, int n_experts, int top, float scale,
+                                                const void* __restrict__ corr, int corr_dt, int* __restrict__ ids,
+                                                float* __restrict__ weights, int lane) {
+    float zmax = -INFINITY;
+    for (int e = lane; e < n_experts; e += 32) zmax = fmaxf(zmax, z[e]);
+    zmax = warp_max(zmax);
+    float den = 0.0f;
+    for (int e = lane; e < n_experts; e += 32) den += expf(z[e] - zmax);
+    den = warp_sum(den);
+    for (int e = lane; e < n_experts; e += 32) {
+        const float s = expf(z[e] - zmax) / den;
+        sbuf[e] = s;
+        if (corr != nullptr) z[e] = s + ld_f(corr, e, corr_dt);      // (without one the logits have the scores' order)
+    }
+    __syncwarp();
+    for (int c = 0; c < top; ++c) {
+        float best = -INFINITY;
+        int at = n_experts;
+        for (int e = lane; e < n_experts; e += 32) {
+            const float v = z[e];
+            if (v > best || (v == best && e < at)) { best = v; at = e; }
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+            const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+            if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
+        }
+        if (at >= n_experts) at = 0;
+        if (lane == 0) {
+            ids[c] = at;
+            weights[c] = sbuf[at] * scale;
+            z[at] = __int_as_float(0x7FC00000);
+        }
+        __syncwarp();
+    }
+}
 
-__device__ __forceinline__ void route_one(float* z, float* gbuf, int n_experts, int top, int scores, int n_groups, int keep,
-                                          float scale, int* __restrict__ ids, float* __restrict__ weights, int lane) {
-    if (scores == kScoresAll) route_top_all(z, gbuf, n_experts, top, n_groups, keep, scale, ids, weights, lane);
-    else if (scores == kScoresSigmoid) route_top_sigmoid(z, n_experts, top, ids, weights, lane);
+// A choice among experts: which scores, groups (kScoresAll), a factor on the weights, a correction of the choice
+// (kScoresPlain).
+struct RouteRule {
+    int scores, n_groups, keep;
+    float scale;
+    const void* corr;
+    int corr_dt;
+    // floats of a warp's second buffer: the groups' scores, or every expert's
+    __host__ __device__ int extra(int n_experts) const;
+};
+constexpr int kScoresChosen = 0, kScoresAll = 1, kScoresSigmoid = 2, kScoresPlain = 3;
+__host__ __device__ __forceinline__ int RouteRule::extra(int n_experts) const {
+    return scores == kScoresPlain ? n_experts : n_groups;
+}
+
+__device__ __forceinline__ void route_one(float* z, float* gbuf, int n_experts, int top, const RouteRule& r,
+                                          int* __restrict__ ids, float* __restrict__ weights, int lane) {
+    if (r.scores == kScoresAll) route_top_all(z, gbuf, n_experts, top, r.n_groups, r.keep, r.scale, ids, weights, lane);
+    else if (r.scores == kScoresSigmoid) route_top_sigmoid(z, n_experts, top, ids, weights, lane);
+    else if (r.scores == kScoresPlain) route_top_plain(z, gbuf, n_experts, top, r.scale, r.corr, r.corr_dt, ids, weights, lane);
     else route_top(z, n_experts, top, ids, weights, lane);
 }
 
@@ -2201,18 +2482,16 @@ __device__ __forceinline__ void route_one(float* z, float* gbuf, int n_experts, 
 // feed-forward.
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const float* __restrict__ logits, int n_tok, int n_experts, int top, int* __restrict__ ids,
-                 float* __restrict__ weights, int all_scores, int n_groups, int keep, float scale, int ld,
-                 float* __restrict__ gate) {
+                 float* __restrict__ weights, const RouteRule rule, int ld, float* __restrict__ gate) {
     extern __shared__ float smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x * (blockDim.x >> 5) + warp;
     if (t >= n_tok) return;
-    float* z = smem + (size_t)warp * (n_experts + n_groups);
+    float* z = smem + (size_t)warp * (n_experts + rule.extra(n_experts));
     for (int e = lane; e < n_experts; e += 32) z[e] = logits[(size_t)t * ld + e];
     if (gate != nullptr && lane == 0) gate[t] = 1.0f / (1.0f + expf(0.0f - logits[(size_t)t * ld + n_experts]));
     __syncwarp();
-    route_one(z, z + n_experts, n_experts, top, all_scores, n_groups, keep, scale, ids + (size_t)t * top,
-              weights + (size_t)t * top, lane);
+    route_one(z, z + n_experts, n_experts, top, rule, ids + (size_t)t * top, weights + (size_t)t * top, lane);
 }
 
 // Whether a choice among groups can be made: equal groups, and the kept ones hold enough experts.
@@ -2222,19 +2501,23 @@ static bool route_groups_ok(int n_experts, int top, int n_groups, int keep) {
 }
 
 extern "C" int nncpu_moe_route(const float* logits, int n_tok, int n_experts, int top, int* ids, float* weights,
-                               int all_scores, int n_groups, int keep, float scale, int ld, float* gate, void* stream) {
-    // all_scores: 0 the softmax over the chosen logits, 1 over all (with groups and a scale), 2 sigmoids; ld: floats a row
-    // of logits (with `gate`, the gate's logit follows the experts')
+                               int all_scores, int n_groups, int keep, float scale, const void* corr, int corr_dt, int ld,
+                               float* gate, void* stream) {
+    // all_scores: 0 the softmax over the chosen logits, 1 over all (with groups and a scale), 2 sigmoids, 3 over all, chosen
+    // with the correction `corr` [n_experts] (or null) and not renormalised (with a scale); ld: floats a row of logits
+    // (with `gate`, the gate's logit follows the experts')
     NN_CHECK(n_tok >= 0 && n_experts > 0 && n_experts <= kRouteMaxExperts && top > 0 && top <= n_experts,
              "router: %d tokens, the top %d of %d experts (at most %d)", n_tok, top, n_experts, kRouteMaxExperts);
     NN_CHECK(all_scores == kScoresAll ? route_groups_ok(n_experts, top, n_groups, keep) : n_groups <= 1,
              "router: the %d best of %d groups of %d experts for the top %d", keep, n_groups, n_experts, top);
     NN_CHECK(ld >= n_experts + (gate != nullptr ? 1 : 0), "router: rows of %d logits for %d experts", ld, n_experts);
+    NN_CHECK(all_scores >= 0 && all_scores <= kScoresPlain && (corr == nullptr || all_scores == kScoresPlain),
+             "router: scores of kind %d", all_scores);
     if (n_tok == 0) return 0;
-    if (n_groups < 1) n_groups = 1;
-    const size_t smem = (size_t)4 * (n_experts + n_groups) * sizeof(float);
-    moe_route_kernel<<<(n_tok + 3) / 4, 128, smem, (cudaStream_t)stream>>>(logits, n_tok, n_experts, top, ids, weights,
-                                                                          all_scores, n_groups, keep, scale, ld, gate);
+    const RouteRule rule{all_scores, n_groups < 1 ? 1 : n_groups, keep, scale, corr, corr_dt};
+    const size_t smem = (size_t)4 * (n_experts + rule.extra(n_experts)) * sizeof(float);
+    moe_route_kernel<<<(n_tok + 3) / 4, 128, smem, (cudaStream_t)stream>>>(logits, n_tok, n_experts, top, ids, weights, rule,
+                                                                          ld, gate);
     NN_LAUNCH_OK("router");
     return 0;
 }
@@ -2275,8 +2558,7 @@ __device__ __forceinline__ float warp_dot(const void* __restrict__ w, size_t row
 __global__ void __launch_bounds__(256)
 moe_router_kernel(const void* __restrict__ x, int x_dt, const void* __restrict__ w, int w_dt, const void* __restrict__ bias,
                   int b_dt, int n_tok, int per_block, int n_experts, int top, int width, int* __restrict__ ids,
-                  float* __restrict__ weights, int all_scores, int n_groups, int keep, float scale,
-                  float* __restrict__ gate) {
+                  float* __restrict__ weights, const RouteRule rule, float* __restrict__ gate) {
     extern __shared__ float smem[];          // a token's input, then its logits
     float* z = smem + width;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
@@ -2291,8 +2573,7 @@ moe_router_kernel(const void* __restrict__ x, int x_dt, const void* __restrict__
         }
         __syncthreads();
         if (warp == 0)
-            route_one(z, z + n_experts, n_experts, top, all_scores, n_groups, keep, scale, ids + (size_t)t * top,
-                      weights + (size_t)t * top, lane);
+            route_one(z, z + n_experts, n_experts, top, rule, ids + (size_t)t * top, weights + (size_t)t * top, lane);
         __syncthreads();
     }
 }
@@ -2303,19 +2584,22 @@ extern "C" int nncpu_moe_router_fits(int n_experts, int width) {
 
 extern "C" int nncpu_moe_router(const void* x, int x_dt, const void* w, int w_dt, const void* bias, int b_dt, int n_tok,
                                 int n_experts, int top, int width, int* ids, float* weights, int all_scores, int n_groups,
-                                int keep, float scale, float* gate, void* stream) {
+                                int keep, float scale, const void* corr, int corr_dt, float* gate, void* stream) {
     // gate (optional, float [n_tok]): w has one row more, whose product's sigmoid is left there
     NN_CHECK(n_tok >= 0 && width > 0 && top > 0 && top <= n_experts && nncpu_moe_router_fits(n_experts, width),
              "router: %d tokens of %d, the top %d of %d experts", n_tok, width, top, n_experts);
     NN_CHECK(all_scores == kScoresAll ? route_groups_ok(n_experts, top, n_groups, keep) : n_groups <= 1,
              "router: the %d best of %d groups of %d experts for the top %d", keep, n_groups, n_experts, top);
+    NN_CHECK(all_scores >= 0 && all_scores <= kScoresPlain && (corr == nullptr || all_scores == kScoresPlain),
+             "router: scores of kind %d", all_scores);
     if (n_tok == 0) return 0;
-    if (n_groups < 1) n_groups = 1;
+    const RouteRule rule{all_scores, n_groups < 1 ? 1 : n_groups, keep, scale, corr, corr_dt};
     // One token a block: with several a block the router's rows did not stay in L1 and the grid got too small
     // (2 048 tokens of 4 096 lanes, 16 experts: 88 us a launch with one token a block, 124 us with eight).
     const int per_block = 1;
-    moe_router_kernel<<<(n_tok + per_block - 1) / per_block, 256, (size_t)(width + n_experts + n_groups) * 4, (cudaStream_t)stream>>>(
-        x, x_dt, w, w_dt, bias, b_dt, n_tok, per_block, n_experts, top, width, ids, weights, all_scores, n_groups, keep, scale, gate);
+    moe_router_kernel<<<(n_tok + per_block - 1) / per_block, 256, (size_t)(width + n_experts + rule.extra(n_experts)) * 4,
+                        (cudaStream_t)stream>>>(x, x_dt, w, w_dt, bias, b_dt, n_tok, per_block, n_experts, top, width, ids,
+                                                weights, rule, gate);
     NN_LAUNCH_OK("router");
     return 0;
 }
@@ -2356,8 +2640,10 @@ __global__ void __launch_bounds__(kMoeWarps * 32)
 moe_down_kernel(const void* __restrict__ act, int act_dt, const void* __restrict__ wd, int w_dt,
                 const int* __restrict__ ids, const float* __restrict__ weights, float* __restrict__ out, int top,
                 int width, int ff, int n_experts, const void* __restrict__ sh_act, const void* __restrict__ sh_wd, int sh_ff,
-                const float* __restrict__ sh_gate) {
+                const float* __restrict__ sh_gate, const void* __restrict__ x, int x_dt, int fresh) {
     // weights null: ones.  sh_act (optional) [n_tok, sh_ff]: the shared feed-forward's part, times the token's gate.
+    // x (optional) [n_tok, width]: a choice beyond the experts hands the input on, times its weight.  fresh: out is written,
+    // not added to.
     extern __shared__ float smem[];          // the token's top * ff activations as floats, then the shared ones
     const int t = blockIdx.x;
     float* sh_smem = smem + (size_t)top * ff;
@@ -2370,12 +2656,13 @@ moe_down_kernel(const void* __restrict__ act, int act_dt, const void* __restrict
         float sum = 0.0f;
         for (int c = 0; c < top; ++c) {
             const int e = ids[(size_t)t * top + c];
-            if (e < 0 || e >= n_experts) continue;
-            const float d = warp_dot(wd, ((size_t)e * width + i) * ff, w_dt, smem + (size_t)c * ff, ff, lane);
+            if (e < 0 || (e >= n_experts && x == nullptr)) continue;
+            const float d = e >= n_experts ? ld_f(x, (size_t)t * width + i, x_dt)
+                                           : warp_dot(wd, ((size_t)e * width + i) * ff, w_dt, smem + (size_t)c * ff, ff, lane);
             sum = weights != nullptr ? fmaf(weights[(size_t)t * top + c], d, sum) : sum + d;
         }
         if (sh_act != nullptr) sum = fmaf(sh_gate[t], warp_dot(sh_wd, (size_t)i * sh_ff, w_dt, sh_smem, sh_ff, lane), sum);
-        if (lane == 0) out[(size_t)t * width + i] += sum;
+        if (lane == 0) out[(size_t)t * width + i] = fresh ? sum : out[(size_t)t * width + i] + sum;
     }
 }
 
@@ -2383,13 +2670,15 @@ extern "C" int nncpu_moe_experts(const void* x, int x_dt, const void* wg, const 
                                  const int* ids, const float* weights, void* act, int act_dt, float* out, int n_tok,
                                  int top, int width, int ff, int n_experts, int kind, float limit, int weight_on_input,
                                  const void* sh_g, const void* sh_u, const void* sh_wd, int sh_ff, void* sh_act,
-                                 const float* sh_gate, void* stream) {
+                                 const float* sh_gate, int identity, int fresh, void* stream) {
+    // identity: ids from n_experts on hand the input on (times the weight).  fresh: out is written, not added to.
     // weight_on_input: the weights multiply the experts' inputs instead of their outputs.  sh_wd (optional): a shared
     // feed-forward in the same launches (its gate/up rows interleaved like the experts' when sh_u is null), its output
     // times sh_gate [n_tok]; sh_act [n_tok, sh_ff] is scratch.
     NN_CHECK(n_tok >= 0 && top > 0 && width > 0 && ff > 0 && n_experts > 0, "experts: %d tokens, top %d, %d x %d, %d experts",
              n_tok, top, width, ff, n_experts);
     NN_CHECK(kind >= kGateSilu && kind <= kGateSwishClamp, "experts: activation kind %d", kind);
+    NN_CHECK(!identity || !weight_on_input, "experts: an identity expert's weight multiplies its output");
     NN_CHECK(wu != nullptr || ff % 8 == 0, "experts: interleaved gate and up rows need a multiple of 8 of them (%d)", ff);
     constexpr size_t kMost = 200 * 1024;
     const bool with_shared = sh_wd != nullptr;
@@ -2417,7 +2706,7 @@ extern "C" int nncpu_moe_experts(const void* x, int x_dt, const void* wg, const 
     NN_LAUNCH_OK("experts (gate and up)");
     moe_down_kernel<<<dim3(n_tok, split_down), kMoeWarps * 32, ((size_t)top * ff + sh_ff) * 4, (cudaStream_t)stream>>>(
         act, act_dt, wd, w_dt, ids, weight_on_input ? nullptr : weights, out, top, width, ff, n_experts, sh_act, sh_wd, sh_ff,
-        sh_gate);
+        sh_gate, identity ? x : nullptr, x_dt, fresh);
     NN_LAUNCH_OK("experts (down)");
     return 0;
 }
@@ -2427,12 +2716,16 @@ extern "C" int nncpu_moe_experts(const void* x, int x_dt, const void* wg, const 
 // as one grouped product on the tensor cores (gemm_sm100.cu), and the choices of a token are added up afterwards.
 //   plan: counts the slots of every expert, gives every slot a row (its expert's rows follow one another; the order
 //     inside an expert is whatever the atomics give, which changes no result: a row's product does not depend on its
-//     place), and lists the 128-row tiles of the grouped product.  One block.
+//     place), and lists the 128-row tiles of the grouped product.  A slot whose id lies beyond the experts (an identity
+//     expert) gets row kIdentityRow and takes no part in the products; the rows that are left over hold slot -1.  One block.
 //   gather: xs[row] = x[slot_of_row[row] / top] (times the slot's weight, where that multiplies the experts' input).
 //   combine: out[t] += sum_c weight[t, c] * y[row_of_slot[t * top + c]], choices in their order; with a shared
 //     feed-forward's branch also + gate[t] * branch[t]; and it can leave the RMS norm that reads the stream next, since it
-//     holds the stream's new row.
+//     holds the stream's new row.  An identity slot adds weight * x[t].  In a layer that norms its sublayers' outputs it
+//     closes the whole sublayer: the sum stays in registers, is normed and added to the stream, and the next norm is left.
 // ---------------------------------------------------------------------------
+constexpr int kIdentityRow = -2;
+
 __global__ void __launch_bounds__(1024)
 moe_plan_kernel(const int* __restrict__ ids, int n_slots, int n_experts, int* __restrict__ row_of_slot,
                 int* __restrict__ slot_of_row, int* __restrict__ n_tiles, int* __restrict__ tile_group,
@@ -2462,11 +2755,13 @@ moe_plan_kernel(const int* __restrict__ ids, int n_slots, int n_experts, int* __
             acc += count[e];
         }
         *n_tiles = tiles < max_tiles ? tiles : max_tiles;
+        plan_smem[3 * n_experts] = acc;
     }
     __syncthreads();
+    for (int r = plan_smem[3 * n_experts] + threadIdx.x; r < n_slots; r += blockDim.x) slot_of_row[r] = -1;
     for (int s = threadIdx.x; s < n_slots; s += blockDim.x) {
         const int e = ids[s];
-        if (e < 0 || e >= n_experts) { row_of_slot[s] = -1; continue; }
+        if (e < 0 || e >= n_experts) { row_of_slot[s] = e < 0 ? -1 : kIdentityRow; continue; }
         const int row = offset[e] + atomicAdd(&cursor[e], 1);
         row_of_slot[s] = row;
         slot_of_row[row] = s;
@@ -2478,7 +2773,7 @@ extern "C" int nncpu_moe_plan(const int* ids, int n_slots, int n_experts, int* r
                               void* stream) {
     NN_CHECK(n_slots > 0 && n_experts > 0 && n_experts <= kRouteMaxExperts && max_tiles >= (n_slots + 127) / 128 + n_experts,
              "experts (plan): %d slots, %d experts, room for %d tiles", n_slots, n_experts, max_tiles);
-    moe_plan_kernel<<<1, 1024, (size_t)3 * n_experts * sizeof(int), (cudaStream_t)stream>>>(
+    moe_plan_kernel<<<1, 1024, ((size_t)3 * n_experts + 1) * sizeof(int), (cudaStream_t)stream>>>(
         ids, n_slots, n_experts, row_of_slot, slot_of_row, n_tiles, tile_group, tile_row0, tile_row_end, max_tiles);
     NN_LAUNCH_OK("experts (plan)");
     return 0;
@@ -2488,6 +2783,7 @@ __global__ void __launch_bounds__(256)
 moe_gather_kernel(const void* __restrict__ x, int x_dt, const int* __restrict__ slot_of_row, int top,
                   const float* __restrict__ weights, __nv_bfloat16* __restrict__ xs, int width) {
     const int row = blockIdx.x;
+    if (slot_of_row[row] < 0) return;       // no slot came here: no product reads the row for a result
     const int t = slot_of_row[row] / top;
     if (weights != nullptr) {
         const float w = weights[slot_of_row[row]];
@@ -2530,7 +2826,8 @@ extern "C" int nncpu_moe_gather(const void* x, int x_dt, const int* slot_of_row,
 
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const void* __restrict__ y, int y_dt, const int* __restrict__ row_of_slot,
-                   const float* __restrict__ weights, float* __restrict__ out, int top, int width) {
+                   const float* __restrict__ weights, float* __restrict__ out, int top, int width,
+                   const void* __restrict__ x, int x_dt, int fresh) {
     const int t = blockIdx.x;
     if (y_dt == DT_F32 && (width & 3) == 0) {
         // 16 bytes a thread; the choices' rows are asked for one after the other and added in their order
@@ -2539,16 +2836,19 @@ moe_combine_kernel(const void* __restrict__ y, int y_dt, const int* __restrict__
             float4 sum = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
             for (int c = 0; c < top; ++c) {
                 const int row = row_of_slot[(size_t)t * top + c];
-                if (row < 0) continue;
+                if (row < 0 && (row != kIdentityRow || x == nullptr)) continue;
                 const float w = weights[(size_t)t * top + c];
-                const float4 v = reinterpret_cast<const float4*>(yf + (size_t)row * width)[i];
+                const float4 v = row < 0 ? ld_f4(x, (size_t)t * width + 4 * i, x_dt)
+                                         : reinterpret_cast<const float4*>(yf + (size_t)row * width)[i];
                 sum.x = fmaf(w, v.x, sum.x); sum.y = fmaf(w, v.y, sum.y);
                 sum.z = fmaf(w, v.z, sum.z); sum.w = fmaf(w, v.w, sum.w);
             }
             float4* o = reinterpret_cast<float4*>(out + (size_t)t * width) + i;
-            float4 was = *o;
-            was.x += sum.x; was.y += sum.y; was.z += sum.z; was.w += sum.w;
-            *o = was;
+            if (!fresh) {
+                const float4 was = *o;
+                sum.x += was.x; sum.y += was.y; sum.z += was.z; sum.w += was.w;
+            }
+            *o = sum;
         }
         return;
     }
@@ -2557,8 +2857,10 @@ moe_combine_kernel(const void* __restrict__ y, int y_dt, const int* __restrict__
         for (int c = 0; c < top; ++c) {
             const int row = row_of_slot[(size_t)t * top + c];
             if (row >= 0) sum = fmaf(weights[(size_t)t * top + c], ld_f(y, (size_t)row * width + i, y_dt), sum);
+            else if (row == kIdentityRow && x != nullptr)
+                sum = fmaf(weights[(size_t)t * top + c], ld_f(x, (size_t)t * width + i, x_dt), sum);
         }
-        out[(size_t)t * width + i] += sum;
+        out[(size_t)t * width + i] = fresh ? sum : out[(size_t)t * width + i] + sum;
     }
 }
 
@@ -2625,13 +2927,18 @@ extern "C" int nncpu_moe_combine_closes(int width) { return width > 0 && width %
 
 extern "C" int nncpu_moe_combine(const void* y, int y_dt, const int* row_of_slot, const float* weights, float* out,
                                  int n_tok, int top, int width, const float* branch, const float* gate, const void* gamma,
-                                 int g_dt, float gamma_offset, float eps, void* norm_out, int norm_dt, void* stream) {
+                                 int g_dt, float gamma_offset, float eps, void* norm_out, int norm_dt, const void* x, int x_dt,
+                                 int fresh, void* stream) {
+    // x (optional) [n_tok, width]: what identity slots add, times their weight; fresh: out is written, not added to
     NN_CHECK(n_tok > 0 && top > 0 && width > 0, "experts (combine): %d tokens of %d", n_tok, width);
+    NN_CHECK((uintptr_t)x % 16 == 0, "experts (combine): rows must be 16-byte aligned");
     if (branch == nullptr && norm_out == nullptr && weights != nullptr) {
-        moe_combine_kernel<<<n_tok, 256, 0, (cudaStream_t)stream>>>(y, y_dt, row_of_slot, weights, out, top, width);
+        moe_combine_kernel<<<n_tok, 256, 0, (cudaStream_t)stream>>>(y, y_dt, row_of_slot, weights, out, top, width, x, x_dt,
+                                                                    fresh);
         NN_LAUNCH_OK("experts (combine)");
         return 0;
     }
+    NN_CHECK(x == nullptr && !fresh, "experts (combine): identity slots and a fresh branch go with weights and without a norm");
     NN_CHECK(y_dt == DT_F32 && nncpu_moe_combine_closes(width), "experts (combine): rows of %d lanes cannot be closed", width);
     NN_CHECK(((uintptr_t)y | (uintptr_t)out | (uintptr_t)branch | (uintptr_t)norm_out) % 16 == 0,
              "experts (combine): rows must be 16-byte aligned");
@@ -2643,6 +2950,92 @@ extern "C" int nncpu_moe_combine(const void* y, int y_dt, const int* row_of_slot
     else if (width <= 256 * 4 * 4) NN_CLOSE(4);
     else NN_CLOSE(8);
 #undef NN_CLOSE
+    NN_LAUNCH_OK("experts (combine)");
+    return 0;
+}
+
+// The closing of a sublayer whose output is normed: b = sum_c weight[t, c] * y[row] (or x[t] for an identity slot) stays in
+// registers, r <- r + norm(b) * (g1 + off1), and (y2 given) y2 = norm(r) * (g2 + off2), the norm that opens what follows.
+// Rows as in moe_combine_close_kernel.
+template <int kVec>
+__global__ void __launch_bounds__(256)
+moe_combine_pair_kernel(const float* __restrict__ y, const int* __restrict__ row_of_slot, const float* __restrict__ weights,
+                        int top, int width, const void* __restrict__ x, int x_dt, float* __restrict__ r,
+                        const void* __restrict__ g1, float off1, float eps1, const void* __restrict__ g2, float off2,
+                        float eps2, int g_dt, void* __restrict__ y2, int y2_dt) {
+    __shared__ float scratch[33];
+    const int t = blockIdx.x, n4 = width >> 2;
+    float4 v[kVec];
+    float ss = 0.0f;
+#pragma unroll
+    for (int j = 0; j < kVec; ++j) v[j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    for (int c = 0; c < top; ++c) {
+        const int row = row_of_slot[(size_t)t * top + c];
+        if (row < 0 && (row != kIdentityRow || x == nullptr)) continue;
+        const float w = weights[(size_t)t * top + c];
+#pragma unroll
+        for (int j = 0; j < kVec; ++j) {
+            const int i = threadIdx.x + j * 256;
+            if (i >= n4) continue;
+            const float4 q = row < 0 ? ld_f4(x, (size_t)t * width + 4 * i, x_dt)
+                                     : reinterpret_cast<const float4*>(y + (size_t)row * width)[i];
+            v[j].x = fmaf(w, q.x, v[j].x); v[j].y = fmaf(w, q.y, v[j].y);
+            v[j].z = fmaf(w, q.z, v[j].z); v[j].w = fmaf(w, q.w, v[j].w);
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < kVec; ++j) {
+        ss = fmaf(v[j].x, v[j].x, ss); ss = fmaf(v[j].y, v[j].y, ss);
+        ss = fmaf(v[j].z, v[j].z, ss); ss = fmaf(v[j].w, v[j].w, ss);
+    }
+    const float s1 = 1.0f / sqrtf(block_sum(ss, scratch) * (1.0f / (float)width) + eps1);
+    float4* r4 = reinterpret_cast<float4*>(r + (size_t)t * width);
+    ss = 0.0f;
+#pragma unroll
+    for (int j = 0; j < kVec; ++j) {
+        const int i = threadIdx.x + j * 256;
+        if (i >= n4) continue;
+        const float4 was = r4[i], g = ld_f4(g1, (size_t)4 * i, g_dt);
+        v[j] = make_float4(fmaf(v[j].x * s1, g.x + off1, was.x), fmaf(v[j].y * s1, g.y + off1, was.y),
+                           fmaf(v[j].z * s1, g.z + off1, was.z), fmaf(v[j].w * s1, g.w + off1, was.w));
+        r4[i] = v[j];
+        ss = fmaf(v[j].x, v[j].x, ss); ss = fmaf(v[j].y, v[j].y, ss);
+        ss = fmaf(v[j].z, v[j].z, ss); ss = fmaf(v[j].w, v[j].w, ss);
+    }
+    if (y2 == nullptr) return;
+    const float s2 = 1.0f / sqrtf(block_sum(ss, scratch) * (1.0f / (float)width) + eps2);
+#pragma unroll
+    for (int j = 0; j < kVec; ++j) {
+        const int i = threadIdx.x + j * 256;
+        if (i >= n4) continue;
+        const float4 g = ld_f4(g2, (size_t)4 * i, g_dt);
+        const float o[4] = {(v[j].x * s2) * (g.x + off2), (v[j].y * s2) * (g.y + off2), (v[j].z * s2) * (g.z + off2),
+                            (v[j].w * s2) * (g.w + off2)};
+        const size_t at = (size_t)t * width + 4 * i;
+        if (y2_dt == DT_BF16) {
+            __nv_bfloat162 h[2] = {__floats2bfloat162_rn(o[0], o[1]), __floats2bfloat162_rn(o[2], o[3])};
+            *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(y2) + at) = *reinterpret_cast<uint2*>(h);
+        } else {
+            *reinterpret_cast<float4*>(reinterpret_cast<float*>(y2) + at) = make_float4(o[0], o[1], o[2], o[3]);
+        }
+    }
+}
+
+extern "C" int nncpu_moe_combine_pair(const float* y, const int* row_of_slot, const float* weights, int n_tok, int top,
+                                      int width, const void* x, int x_dt, float* r, const void* g1, float off1, float eps1,
+                                      const void* g2, float off2, float eps2, int g_dt, void* y2, int y2_dt, void* stream) {
+    NN_CHECK(n_tok > 0 && top > 0 && nncpu_moe_combine_closes(width), "experts (combine): rows of %d lanes cannot be closed", width);
+    NN_CHECK(weights != nullptr && g1 != nullptr && (y2 == nullptr || g2 != nullptr), "experts (combine): a norm without weights");
+    NN_CHECK(((uintptr_t)y | (uintptr_t)x | (uintptr_t)r | (uintptr_t)y2 | (uintptr_t)g1 | (uintptr_t)g2) % 16 == 0,
+             "experts (combine): rows must be 16-byte aligned");
+#define NN_PAIR(V)                                                                                                       \
+    moe_combine_pair_kernel<V><<<n_tok, 256, 0, (cudaStream_t)stream>>>(y, row_of_slot, weights, top, width, x, x_dt, r, \
+                                                                        g1, off1, eps1, g2, off2, eps2, g_dt, y2, y2_dt)
+    if (width <= 256 * 4) NN_PAIR(1);
+    else if (width <= 256 * 4 * 2) NN_PAIR(2);
+    else if (width <= 256 * 4 * 4) NN_PAIR(4);
+    else NN_PAIR(8);
+#undef NN_PAIR
     NN_LAUNCH_OK("experts (combine)");
     return 0;
 }

@@ -507,6 +507,50 @@ def qk_whole_norm_append(qkv, q_gamma, k_gamma, eps, cos_sin, tok_seq, tok_pos, 
           _i(v_pages.shape[-1] if n_kv else v_head_dim), _stream())
 
 
+CONV_STATE_HEAD = 4      # words of a convolution's state row before its two copies of the last inputs
+
+
+def conv_state_floats(taps: int, channels: int) -> int:
+    """Floats of a sequence's state row for a short convolution of ``taps`` taps over ``channels`` lanes: two copies of the
+    last taps - 1 inputs and after how many tokens each was taken (a step reads one copy and leaves the other)."""
+    return CONV_STATE_HEAD + (2 * (taps - 1) * channels + 3) // 4 * 4
+
+
+def _conv_check(w, state, seq_slots, channels: int) -> None:
+    taps = w.shape[0]
+    assert w.dtype == torch.float32 and w.shape == (taps, channels) and w.is_contiguous() and taps >= 1
+    assert state.dtype == torch.float32 and state.dim() == 2 and state.is_contiguous() and state.shape[1] % 4 == 0
+    assert state.shape[1] >= conv_state_floats(taps, channels) and seq_slots.dtype == torch.int32
+
+
+def qk_conv_norm_append(proj, conv_w, state, seq_slots, cu_seqlens, q_gamma, k_gamma, eps, cos_sin, tok_seq, tok_pos,
+                        block_table, k_pages, v_pages, q_out, n_heads: int, n_kv: int, head_dim: int) -> None:
+    """For mixers with a short convolution over time on every channel of q and k, and values that are the keys: ``proj``
+    float32 [n, >= (n_heads + n_kv) * head_dim] holds the heads of q, then of k.  y_t = sum_j conv_w[j] proj_(t - taps + 1 + j)
+    (``conv_w`` float32 [taps, C], the last row the current token's); a key head's y goes to its value page as it is; then
+    the RMS norm per head (weights [head_dim] or None) and the rotation of the first ``cos_sin.shape[1]`` neighbouring pairs;
+    q to ``q_out``, k to its page, in rows as long as theirs with zeros behind the head's lanes.  ``state`` float32 [slots,
+    ``conv_state_floats``] holds every sequence's last inputs; it is read and left advanced by the step's tokens."""
+    n = q_out.shape[0]
+    half = 0 if cos_sin is None else cos_sin.shape[1]
+    qp = q_out.shape[1] // n_heads
+    C = (n_heads + n_kv) * head_dim
+    assert proj.dtype == torch.float32 and proj.shape[0] == n and proj.shape[1] >= C and proj.is_contiguous()
+    _conv_check(conv_w, state, seq_slots, C)
+    assert cu_seqlens.dtype == tok_seq.dtype == tok_pos.dtype == torch.int32 and q_out.shape[1] == qp * n_heads
+    assert q_gamma is None or k_gamma is None or q_gamma.dtype == k_gamma.dtype
+    assert (q_gamma is None or q_gamma.numel() == head_dim) and (k_gamma is None or k_gamma.numel() == head_dim)
+    assert cos_sin is None or (cos_sin.dtype == torch.float32 and cos_sin.shape == (n, half, 2))
+    assert k_pages.shape[1] == v_pages.shape[1] == n_kv and k_pages.shape[-1] == qp and k_pages.dtype == v_pages.dtype
+    assert q_out.is_contiguous() and k_pages.is_contiguous() and v_pages.is_contiguous()
+    g = q_gamma if q_gamma is not None else k_gamma
+    _call("generic", "nncpu_qk_conv_norm_append", _ptr(proj), _i(proj.shape[1]), _ptr(conv_w), _i(conv_w.shape[0]), _ptr(state),
+          _l(state.shape[1]), _ptr(seq_slots), _ptr(cu_seqlens), _ptr(q_gamma), _ptr(k_gamma), _i(_code(g)), _f(eps),
+          _ptr(cos_sin), _i(half), _ptr(tok_seq), _ptr(tok_pos), _ptr(block_table), _i(block_table.shape[1]), _ptr(k_pages),
+          _ptr(v_pages), _i(_code(k_pages)), _ptr(q_out), _i(_code(q_out)), _i(n), _i(n_heads), _i(n_kv), _i(head_dim), _i(qp),
+          _i(v_pages.shape[-1]), _stream())
+
+
 def key_span(window: int = 0, chunk: int = 0) -> int:
     """The one number by which every attention kernel knows which earlier keys a query sees (their ``window``
     argument): ``window`` > 0, the last ``window`` keys up to the query, as it is; ``chunk`` > 0, the keys of the
@@ -516,15 +560,26 @@ def key_span(window: int = 0, chunk: int = 0) -> int:
     return window if window else -chunk
 
 
+def _head_gate(head_gate, n: int, n_heads: int):
+    """The attention kernels' pair (first logit, floats from a token's logits to the next one's)."""
+    if head_gate is None:
+        return None, _i(0)
+    rows, col = head_gate
+    assert rows.dtype == torch.float32 and rows.is_contiguous() and rows.shape[0] == n and 0 <= col <= rows.shape[1] - n_heads
+    return (None if (rows.is_meta and _dry) else _vp(rows.data_ptr() + 4 * col)), _i(rows.shape[1])
+
+
 def attention(q, k_pages, v_pages, block_table, tok_seq, tok_pos, out, n_heads: int, n_kv: int, head_dim: int,
               scale: float, window: int = 0, v_head_dim: int = 0, slope_base: float = 0.0, sinks=None, keep: int = 0,
-              v_lanes: int = 0) -> None:
+              v_lanes: int = 0, cap: float = 0.0, head_gate=None) -> None:
     """Causal attention of each token over its sequence's pages.  ``window``: see ``key_span`` (here and in the
     other attention kernels).  ``keep``: with a window, the sequence's first ``keep`` keys stay visible (here and in the
     other attention kernels).  ``v_head_dim``: lanes of a value row when they differ from ``head_dim``; ``v_lanes``: how
     many of them the output has (0: all).  ``slope_base`` b != 0: head h takes
     2^(-b (h + 1) / n_heads) * (query position - key position) off its scaled scores.  ``sinks`` (float32
-    [n_heads]): exp(sinks[h]) joins the denominator of head h's softmax (here and in the other attention kernels)."""
+    [n_heads]): exp(sinks[h]) joins the denominator of head h's softmax (here and in the other attention kernels).
+    ``cap`` c > 0: a scaled score z becomes c tanh(z / c), and ``head_gate = (rows, col)``: head h's output is multiplied
+    by sigmoid(rows[t, col + h]), rows float32 [n, >= col + n_heads] (both here and in the other attention kernels)."""
     n = q.shape[0]
     v_head_dim = v_head_dim or head_dim
     v_lanes = v_lanes or v_head_dim
@@ -535,7 +590,7 @@ def attention(q, k_pages, v_pages, block_table, tok_seq, tok_pos, out, n_heads: 
     _call("generic", "nncpu_attention", _ptr(q), _i(_code(q)), _ptr(k_pages), _ptr(v_pages), _i(_code(k_pages)),
           _ptr(block_table), _i(block_table.shape[1]), _ptr(tok_seq), _ptr(tok_pos), _ptr(out), _i(_code(out)),
           _i(n), _i(n_heads), _i(n_kv), _i(head_dim), _i(v_head_dim), _i(v_lanes), _f(scale), _i(window), _i(keep),
-          _f(slope_base), _ptr(sinks), _stream())
+          _f(slope_base), _ptr(sinks), _f(cap), *_head_gate(head_gate, n, n_heads), _stream())
 
 
 def attention_mma_supported(n_heads: int, n_kv: int, head_dim: int, *tensors) -> bool:
@@ -579,7 +634,7 @@ def attention_decode_scratch_floats(n_tok: int, n_heads: int, n_kv: int, head_di
 
 def attention_decode_mma(q, k_pages, v_pages, block_table, tok_seq, tok_pos, out, scratch, n_heads: int, n_kv: int,
                          head_dim: int, scale: float, window: int, n_splits: int, slope_base: float = 0.0,
-                         sinks=None, keep: int = 0, v_lanes: int = 0) -> None:
+                         sinks=None, keep: int = 0, v_lanes: int = 0, cap: float = 0.0, head_gate=None) -> None:
     """One token per sequence; each token's keys are cut into ``n_splits``
     splits that run in parallel.  ``head_dim`` is the size of q's heads and of the pages' key rows, ``v_lanes`` that of
     the output's heads (0: ``head_dim``; at most the value rows').  With ``scratch`` (float32,
@@ -595,14 +650,16 @@ def attention_decode_mma(q, k_pages, v_pages, block_table, tok_seq, tok_pos, out
     _call("attention_mma", "nncpu_attention_decode_mma", _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table),
           _i(block_table.shape[1]), _ptr(tok_seq), _ptr(tok_pos), _ptr(out), _ptr(scratch),
           ctypes.c_long(0 if scratch is None else scratch.numel()), _i(n), _i(n_heads), _i(n_kv), _i(head_dim),
-          _i(v_pages.shape[-1]), _i(v_lanes), _f(scale), _i(window), _i(keep), _i(n_splits), _f(slope_base), _ptr(sinks), _stream())
+          _i(v_pages.shape[-1]), _i(v_lanes), _f(scale), _i(window), _i(keep), _i(n_splits), _f(slope_base), _ptr(sinks),
+          _f(cap), *_head_gate(head_gate, n, n_heads), _stream())
 
 
 def attention_decode_mma_from_qkv(qkv, q_gamma, k_gamma, eps, cos_sin, k_pages, v_pages, append: bool, block_table,
                                   tok_seq, tok_pos, out, scratch, n_heads: int, n_kv: int, head_dim: int, scale: float,
                                   window: int, n_splits: int, slope_base: float = 0.0, q_temp=None, sinks=None,
                                   values_are_keys: bool = False, gated: bool = False, keep: int = 0, v_head_dim: int = 0,
-                                  whole_norm: bool = False, rot_pairs: bool = False) -> None:
+                                  whole_norm: bool = False, rot_pairs: bool = False, cap: float = 0.0,
+                                  head_gated: bool = False, conv=None) -> None:
     """Decode attention that starts from the float32 projections ``qkv`` [n, per_tok * head_dim] (q heads, then with
     ``append`` the k and v heads): every block makes its queries itself (per-head norm, rotation by ``cos_sin``
     [n, head_dim / 2, 2]), and with ``append`` the token's key and value are made, written to the cache and used.
@@ -612,11 +669,19 @@ def attention_decode_mma_from_qkv(qkv, q_gamma, k_gamma, eps, cos_sin, k_pages, 
     lane by their sigmoid (in place of ``sigmoid_gate``).  ``head_dim`` and ``v_head_dim`` (0: the same) are the heads' own
     sizes; the pages' rows may be longer (``attention_rows``), with zeros behind them.  ``whole_norm``: the norm runs over
     all of a token's query (key) lanes at once, as in ``qk_whole_norm_append``.  ``rot_pairs``: ``cos_sin`` [n, pairs, 2]
-    turns a head's first neighbouring pairs of lanes."""
+    turns a head's first neighbouring pairs of lanes.  ``cap``: as in ``attention``.  ``head_gated``: n_heads logits end the
+    rows, one a head.  ``conv = (w [taps, C], state, seq_slots)``: the short convolution of ``qk_conv_norm_append`` (every token
+    is its sequence's only one); a value that is the key is taken after it."""
     n = out.shape[0]
     v_head_dim = v_head_dim or head_dim
     row = n_heads * head_dim + ((n_kv * head_dim + (0 if values_are_keys else n_kv * v_head_dim)) if append else 0)
-    row += n_heads * v_head_dim if gated else 0
+    assert not (gated and head_gated)
+    row += n_heads * v_head_dim if gated else n_heads if head_gated else 0
+    conv_w = conv_state = slots = None
+    if conv is not None:
+        conv_w, conv_state, slots = conv
+        _conv_check(conv_w, conv_state, slots, (n_heads + n_kv) * head_dim)
+        assert values_are_keys and append and not whole_norm
     rot_half = 0 if cos_sin is None else cos_sin.shape[1]
     assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == n_heads)
     assert qkv.dtype == torch.float32 and qkv.shape == (n, row) and qkv.is_contiguous()
@@ -633,13 +698,14 @@ def attention_decode_mma_from_qkv(qkv, q_gamma, k_gamma, eps, cos_sin, k_pages, 
           _ptr(tok_seq), _ptr(tok_pos), _ptr(out), _ptr(scratch), ctypes.c_long(0 if scratch is None else scratch.numel()),
           _i(n), _i(n_heads), _i(n_kv), _i(k_pages.shape[-1]), _i(v_pages.shape[-1]), _i(head_dim), _i(v_head_dim),
           _i(whole_norm), _i(rot_half), _i(rot_pairs), _f(scale), _i(window), _i(keep), _i(n_splits), _f(slope_base),
-          _f(q_temp[0] if q_temp else 0.0), _i(q_temp[1] if q_temp else 1), _ptr(sinks), _i(values_are_keys), _i(gated),
-          _stream())
+          _f(q_temp[0] if q_temp else 0.0), _i(q_temp[1] if q_temp else 1), _ptr(sinks), _i(values_are_keys),
+          _i(2 if head_gated else 1 if gated else 0), _f(cap), _ptr(conv_w), _i(0 if conv is None else conv_w.shape[0]),
+          _ptr(conv_state), _l(0 if conv is None else conv_state.shape[1]), _ptr(slots), _stream())
 
 
 def attention_prefill_mma(q, k_pages, v_pages, block_table, cu_seqlens, tok_pos, out, n_seqs: int, n_heads: int,
                           n_kv: int, head_dim: int, scale: float, window: int, slope_base: float = 0.0,
-                          sinks=None, keep: int = 0, v_lanes: int = 0) -> None:
+                          sinks=None, keep: int = 0, v_lanes: int = 0, cap: float = 0.0, head_gate=None) -> None:
     """Any number of new tokens per sequence, at consecutive positions.  ``slope_base``, ``sinks`` and ``keep`` as in
     ``attention``, ``v_lanes`` as in ``attention_decode_mma``."""
     n = q.shape[0]
@@ -649,7 +715,7 @@ def attention_prefill_mma(q, k_pages, v_pages, block_table, cu_seqlens, tok_pos,
     _call("attention_mma", "nncpu_attention_prefill_mma", _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table),
           _i(block_table.shape[1]), _ptr(cu_seqlens), _ptr(tok_pos), _ptr(out), _i(n), _i(n_seqs), _i(n_heads),
           _i(n_kv), _i(head_dim), _i(v_pages.shape[-1]), _i(v_lanes), _f(scale), _i(window), _i(keep), _f(slope_base),
-          _ptr(sinks), _stream())
+          _ptr(sinks), _f(cap), *_head_gate(head_gate, n, n_heads), _stream())
 
 
 def attention_prefill_tc_supported(n_heads: int, n_kv: int, head_dim: int, *tensors) -> bool:
@@ -661,7 +727,7 @@ def attention_prefill_tc_supported(n_heads: int, n_kv: int, head_dim: int, *tens
 
 def attention_prefill_tc(q, k_pages, v_pages, block_table, cu_seqlens, tok_pos, out, status, n_seqs: int,
                          n_heads: int, n_kv: int, head_dim: int, scale: float, window: int, slope_base: float = 0.0,
-                         sinks=None, keep: int = 0, v_lanes: int = 0) -> None:
+                         sinks=None, keep: int = 0, v_lanes: int = 0, cap: float = 0.0, head_gate=None) -> None:
     """Prefill attention on the tcgen05 tensor cores: any number of new tokens per sequence, at consecutive
     positions; ``status`` is an int32 word on the device that receives a code if a bounded wait runs out.
     ``slope_base``, ``sinks`` and ``keep`` as in ``attention``, ``v_lanes`` as in ``attention_decode_mma``."""
@@ -675,7 +741,7 @@ def attention_prefill_tc(q, k_pages, v_pages, block_table, cu_seqlens, tok_pos, 
     _call("attention_tc", "nncpu_attention_prefill_tc", _ptr(q), _ptr(k_pages), _ptr(v_pages), _i(k_pages.shape[0]),
           _ptr(block_table), _i(block_table.shape[1]), _ptr(cu_seqlens), _ptr(tok_pos), _ptr(out), _i(n), _i(n_seqs),
           _i(n_heads), _i(n_kv), _i(head_dim), _i(v_pages.shape[-1]), _i(v_lanes), _f(scale), _i(window), _i(keep),
-          _f(slope_base), _ptr(sinks), _ptr(status), _stream())
+          _f(slope_base), _ptr(sinks), _f(cap), *_head_gate(head_gate, n, n_heads), _ptr(status), _stream())
 
 
 GATED_ACTS = {"silu": 0, "gelu_tanh": 1, "swish_clamp": 2}
@@ -813,15 +879,21 @@ def _route_mode(scoring):
     softmax over all experts; the experts form ``n_groups`` equal groups of neighbours whose score is their best
     expert's, and only experts of the ``keep`` best groups can be chosen (``n_groups`` <= 1: no groups); the weights
     are the chosen scores divided by their sum (+ 1e-20), times ``scale``.  ("sigmoid",): scores are the sigmoids of the
-    logits, and the weights are the chosen scores as they are."""
+    logits, and the weights are the chosen scores as they are.  ("plain", correction, scale): scores are the softmax over
+    all experts; those with the largest score + correction (a tensor [E], or None) are chosen, and the weights are their
+    scores as they are, times ``scale``."""
     if scoring is None:
-        return _i(0), _i(1), _i(1), _f(1.0)
+        return _i(0), _i(1), _i(1), _f(1.0), None, _i(0)
     if scoring[0] == "sigmoid":
-        return _i(2), _i(1), _i(1), _f(1.0)
+        return _i(2), _i(1), _i(1), _f(1.0), None, _i(0)
+    if scoring[0] == "plain":
+        _, corr, scale = scoring
+        assert corr is None or corr.dim() == 1
+        return _i(3), _i(1), _i(1), _f(scale), _ptr(corr), _i(_code(corr))
     kind, n_groups, keep, scale = scoring
     if kind != "all":
         raise InvalidArgument(f"a router cannot score by {kind!r}")
-    return _i(1), _i(max(1, n_groups)), _i(max(1, keep)), _f(scale)
+    return _i(1), _i(max(1, n_groups)), _i(max(1, keep)), _f(scale), None, _i(0)
 
 
 def moe_route(logits, top: int, ids, weights, scoring=None, gate=None) -> None:
@@ -856,7 +928,7 @@ def moe_router(x, w, bias, top: int, ids, weights, scoring=None, gate=None) -> N
 
 
 def moe_experts(x, w_gate, w_up, w_down, ids, weights, act, out, kind: str, limit: float = 0.0,
-                weight_on_input: bool = False, shared=None) -> None:
+                weight_on_input: bool = False, shared=None, identity: bool = False, fresh: bool = False) -> None:
     """out[t] += sum_c weights[t, c] * W_down[e] act(W_gate[e] x_t, W_up[e] x_t) with e = ids[t, c].  Weights are
     [E, ff, width] (gate, up) and [E, width, ff] (down); with ``w_up`` None, ``w_gate`` is [E, 2 ff, width] with an
     expert's gate and up rows interleaved in blocks of 8 (the layout of the grouped product).  ``act`` [n * top, ff] is
@@ -864,7 +936,8 @@ def moe_experts(x, w_gate, w_up, w_down, ids, weights, act, out, kind: str, limi
     few tokens and for every size and type.  ``weight_on_input``: out[t] += sum_c W_down[e] act(W_gate[e] (w x_t), W_up[e]
     (w x_t)) instead, w = weights[t, c].  ``shared`` = (w_gate, w_up or None, w_down, act [n, sff], gate [n]): a shared
     feed-forward of the same form in the same launches, its output times the token's gate; its matrices [sff, width] (or
-    [2 sff, width] interleaved) and [width, sff]."""
+    [2 sff, width] interleaved) and [width, sff].  ``identity``: a chosen id from E on stands for x_t itself, times its weight.
+    ``fresh``: out is written, not added to."""
     n, width = x.shape
     sg = su = sd = sact = sgate = None
     sff = 0
@@ -883,7 +956,7 @@ def moe_experts(x, w_gate, w_up, w_down, ids, weights, act, out, kind: str, limi
     _call("generic", "nncpu_moe_experts", _ptr(x), _i(_code(x)), _ptr(w_gate), _ptr(w_up), _ptr(w_down), _i(_code(w_gate)),
           _ptr(ids), _ptr(weights), _ptr(act), _i(_code(act)), _ptr(out), _i(n), _i(top), _i(width), _i(ff), _i(E),
           _i(GATED_ACTS[kind]), _f(limit), _i(weight_on_input), _ptr(sg), _ptr(su), _ptr(sd), _i(sff), _ptr(sact), _ptr(sgate),
-          _stream())
+          _i(identity), _i(fresh), _stream())
 
 
 def moe_plan_tiles(n_slots: int, n_experts: int) -> int:
@@ -894,7 +967,8 @@ def moe_plan_tiles(n_slots: int, n_experts: int) -> int:
 def moe_plan(ids, n_experts: int, row_of_slot, slot_of_row, plan) -> None:
     """Sorts the token slots (row-major ``ids`` [n, top]) by expert: ``row_of_slot`` / ``slot_of_row`` (int32 [n * top])
     map slots to rows and back, and ``plan`` (int32 [1 + 3 * moe_plan_tiles]) receives the number of 128-row tiles and
-    per tile its expert, first row and its expert's last row + 1, for ``linear_tc_grouped``."""
+    per tile its expert, first row and its expert's last row + 1, for ``linear_tc_grouped``.  A slot whose id is n_experts or
+    more (an identity expert) gets row -2; the rows beyond the experts' slots get slot -1."""
     S = ids.numel()
     mt = moe_plan_tiles(S, n_experts)
     assert ids.dtype == row_of_slot.dtype == slot_of_row.dtype == plan.dtype == torch.int32
@@ -920,10 +994,13 @@ def moe_combine_closes(width: int) -> bool:
     return width > 0 and width % 4 == 0 and width <= 8192
 
 
-def moe_combine(y, row_of_slot, weights, out, top: int = 0, branch=None, gate=None, then_norm=None) -> None:
+def moe_combine(y, row_of_slot, weights, out, top: int = 0, branch=None, gate=None, then_norm=None, identity_x=None,
+                fresh: bool = False) -> None:
     """out[t] += sum_c weights[t, c] * y[row_of_slot[t * top + c]], choices in their order; out float32.  ``weights``
     None: ones (``top`` is then given).  ``branch`` (float32, out's shape): + gate[t] * branch[t] (``gate`` None: + branch[t]).
-    ``then_norm`` = (gamma, offset, eps, norm_out): the RMS norm of the new rows is left there in the same pass."""
+    ``then_norm`` = (gamma, offset, eps, norm_out): the RMS norm of the new rows is left there in the same pass.
+    ``identity_x`` [n, width]: a slot of row -2 adds its weight times x[t].  ``fresh``: out is written, not added to (both
+    without a branch and a norm)."""
     n, width = out.shape
     top = weights.shape[1] if weights is not None else top
     assert out.dtype == torch.float32 and y.shape[1] == width and row_of_slot.numel() == n * top and out.is_contiguous()
@@ -936,7 +1013,24 @@ def moe_combine(y, row_of_slot, weights, out, top: int = 0, branch=None, gate=No
         assert gamma.numel() == width and norm_out.shape == out.shape and norm_out.is_contiguous()
     _call("generic", "nncpu_moe_combine", _ptr(y), _i(_code(y)), _ptr(row_of_slot), _ptr(weights), _ptr(out), _i(n), _i(top),
           _i(width), _ptr(branch), _ptr(gate), _ptr(gamma), _i(_code(gamma)), _f(offset), _f(eps), _ptr(norm_out),
-          _i(_code(norm_out)), _stream())
+          _i(_code(norm_out)), _ptr(identity_x), _i(_code(identity_x)), _i(fresh), _stream())
+
+
+def moe_combine_pair(y, row_of_slot, weights, residual, post_norm, then_norm=None, identity_x=None) -> None:
+    """The closing of a sublayer that norms its output: with b[t] = sum_c weights[t, c] * y[row] (or x[t] for a slot of row
+    -2), residual += rmsnorm(b) with ``post_norm`` = (gamma, offset, eps), and with ``then_norm`` = (gamma, offset, eps, out)
+    out = rmsnorm(residual), in one pass.  Rows as ``moe_combine_closes`` says; y float32."""
+    n, width = residual.shape
+    top = weights.shape[1]
+    g1, off1, eps1 = post_norm
+    g2, off2, eps2, out = then_norm if then_norm is not None else (None, 0.0, 0.0, None)
+    assert moe_combine_closes(width) and residual.dtype == y.dtype == torch.float32 and y.shape[1] == width
+    assert row_of_slot.numel() == n * top and weights.shape == (n, top) and residual.is_contiguous()
+    assert g1.numel() == width and (g2 is None or (g2.numel() == width and g2.dtype == g1.dtype and out.shape == residual.shape))
+    assert identity_x is None or identity_x.shape == (n, width)
+    _call("generic", "nncpu_moe_combine_pair", _ptr(y), _ptr(row_of_slot), _ptr(weights), _i(n), _i(top), _i(width),
+          _ptr(identity_x), _i(_code(identity_x)), _ptr(residual), _ptr(g1), _f(off1), _f(eps1), _ptr(g2), _f(off2), _f(eps2),
+          _i(_code(g1)), _ptr(out), _i(_code(out)), _stream())
 
 
 def linear_tc_grouped(xs, w, out, plan, n_experts: int, workspace: GemmWorkspace, epilogue: str = "plain",

@@ -26,18 +26,30 @@ product) and ``out_bias``.
 the attention (``ops.qk_whole_norm_append``), which lays a head of any size up to 128 lanes, and a value head of another
 size, into the 64 or 128 lanes that the tensor-core attention kernels read (zeros behind); a decode step has the same
 inside the attention kernel.
+
+``conv`` n (with values that are the keys): q and k pass a causal convolution over time of n taps per channel right after
+the projection, so the value is the convolved key; the last n - 1 projections of a sequence are its state, 32-bit, in the
+cache's state area.  Convolution, per-head norm, rotation (neighbouring lanes) and append are one kernel in a prompt step
+(``ops.qk_conv_norm_append``) and the attention kernel's own first steps in a decode step; both leave the state advanced.
+``score_cap`` c: a scaled score z becomes c tanh(z / c), 32-bit, inside every attention kernel.  ``head_gate``: one gate
+logit per head, whose rows ride in the projection's product; the attention kernels apply the sigmoid where they divide by
+the softmax's sum.
 """
 from __future__ import annotations
 
 import torch
 
 from .. import perf
-from ..cache import KVRequest
+from ..cache import KVRequest, StateRequest
 from ..errors import UnsupportedModel
 from ..kernels import ops
 from ..weights.params import ParamSpec
 from . import base
 from .base import Mixer, register_mixer
+
+
+# The tensor-core kernels' cap is a difference of two numbers of the cap's size; beyond this one its rounding would show.
+MAX_FAST_CAP = 4096.0
 
 
 @register_mixer("attention")
@@ -52,7 +64,15 @@ class Attention(Mixer):
         if s.keep_first and not s.window:
             raise UnsupportedModel(f"{s.name}: {s.keep_first} kept keys without a window")
         self.pairs = s.position is not None and s.position.kind == "rope_pairs"
-        self.apart = s.qk_norm_whole or self.pairs       # norm, rotation and append by the kernel that knows these two
+        self.convolved = s.conv > 0                      # convolution, norm, rotation and append by the kernel of these
+        # norm, rotation and append by the kernel that knows whole rows and neighbouring lanes
+        self.apart = (s.qk_norm_whole or self.pairs) and not self.convolved
+        if self.convolved and (reads_other_cache or not s.values_are_keys or s.qk_norm_whole or s.q_temp_coef != 0.0
+                               or (s.position is not None and not self.pairs)):
+            raise UnsupportedModel(f"{s.name}: convolutions of q and k go with values that are the keys, a norm per head and a "
+                                   "rotation of neighbouring lanes, and with a cache of the layer's own")
+        if s.head_gate and s.out_gate:
+            raise UnsupportedModel(f"{s.name}: a gate per head and a gate per lane")
         if self.apart and (s.values_are_keys or s.q_temp_coef != 0.0 or (s.qk_norm is not None and not s.qk_norm_whole)
                            or (s.position is not None and not self.pairs)):
             raise UnsupportedModel(f"{s.name}: a norm over whole rows or a rotation of neighbouring lanes does not go with a "
@@ -68,7 +88,7 @@ class Attention(Mixer):
         self.kv_size = 0 if reads_other_cache else s.n_kv_heads * s.head_dim
         self.v_size = 0 if (reads_other_cache or s.values_are_keys) else s.n_kv_heads * self.v_dim
         self.out_size = s.n_heads * self.v_dim
-        self.gate_size = self.out_size if s.out_gate else 0
+        self.gate_size = self.out_size if s.out_gate else s.n_heads if s.head_gate else 0
         self.gate_col = self.q_size + self.kv_size + self.v_size      # the gate's logits follow the heads in a row
         # Value heads of their own size are known to the 32-bit kernel alone.  A distance bias or a query temperature
         # keeps a prompt step off the fused q/k/v epilogue of the projection (which knows neither): the temperature is
@@ -81,7 +101,7 @@ class Attention(Mixer):
         self.plain_core = self.v_dim != s.head_dim and not self.apart
         self.k_row, self.v_row = s.head_dim, self.v_dim         # lanes of a head in the pages (bind may lengthen them)
         self.unfused = (self.plain_core or self.apart or s.slope_base != 0.0 or s.q_temp_coef != 0.0 or s.values_are_keys or s.sink
-                        or s.out_gate)
+                        or s.out_gate or s.head_gate or self.convolved)
         self.q_temp = (s.q_temp_coef, s.q_temp_every) if s.q_temp_coef != 0.0 else None
         self.position = None if s.position is None else base.build("position", s.position)
         self.span = ops.key_span(s.window, s.chunk)     # what the kernels take as their ``window``
@@ -91,6 +111,11 @@ class Attention(Mixer):
         return None if self.shared_kv else KVRequest(s.n_kv_heads, self.k_row, s.window,
                                                      0 if self.v_row == self.k_row else self.v_row, chunk=s.chunk,
                                                      keep_first=s.keep_first)
+
+    def state_request(self):
+        if not self.convolved:
+            return None
+        return StateRequest((ops.conv_state_floats(self.spec.conv, self.q_size + self.kv_size),), torch.float32)
 
     def _proj_names(self):
         if self.shared_kv:
@@ -127,27 +152,34 @@ class Attention(Mixer):
                 p.append(ParamSpec(self._norm_tensor("k"), (k_lanes,), init=("one_plus_normal", 0.1)))
         if s.sink:
             p.append(ParamSpec(f"{s.name}.sink", (s.n_heads,), init=("normal", 1.0)))
-        if s.out_gate:
+        if s.out_gate or s.head_gate:
             p.append(ParamSpec(f"{s.name}.g", (self.gate_size, s.hidden_size)))
+        if self.convolved:
+            p += [ParamSpec(f"{self._tensor('q_proj')}.conv", (self.q_size, s.conv), init=("normal", 0.5)),
+                  ParamSpec(f"{self._tensor('k_proj')}.conv", (self.kv_size, s.conv), init=("normal", 0.5))]
         return p
 
     def bind(self, tensors, rt):
         s, self.rt = self.spec, rt
-        if self.apart and rt.dtype == torch.bfloat16:
+        if (self.apart or self.convolved) and rt.dtype == torch.bfloat16:
             # rows of the sizes that the tensor-core attention kernels read; where they take none, the heads' own
             self.k_row, self.v_row = ops.attention_rows(s.head_dim, self.v_dim) or (s.head_dim, self.v_dim)
         names = self._proj_names()
         ws = [tensors.pop(self._tensor(n)) for n in names]
-        if s.out_gate:
+        if s.out_gate or s.head_gate:
             ws.append(tensors.pop(f"{s.name}.g"))       # the gate's logits come out of the same product
         self.w_qkv = ws[0] if len(ws) == 1 else torch.cat(ws, dim=0).contiguous()
         del ws
         self.b_qkv = None
         if s.qkv_bias:
             bs = [tensors.pop(self._tensor(n, bias=True)) for n in names]
-            if s.out_gate:
+            if s.out_gate or s.head_gate:
                 bs.append(torch.zeros(self.gate_size, dtype=bs[0].dtype, device=bs[0].device))   # the gate has no bias
             self.b_qkv = bs[0] if len(bs) == 1 else torch.cat(bs, dim=0).contiguous()
+        self.w_conv = None
+        if self.convolved:      # [taps, channels]: the kernels' lanes are channels
+            ws = [tensors.pop(f"{self._tensor(n)}.conv") for n in names]
+            self.w_conv = torch.cat(ws, dim=0).to(torch.float32).t().contiguous()
         # the sink logits enter 32-bit softmax arithmetic
         self.sinks = tensors[f"{s.name}.sink"].to(torch.float32).contiguous() if s.sink else None
         self.w_o = tensors[self._tensor("o_proj")]
@@ -200,12 +232,18 @@ class Attention(Mixer):
                                                       s.scale, self.span, n_splits, s.slope_base, self.q_temp,
                                                       sinks=self.sinks, values_are_keys=s.values_are_keys,
                                                       gated=s.out_gate, keep=s.keep_first, v_head_dim=self.v_dim,
-                                                      whole_norm=s.qk_norm_whole, rot_pairs=self.pairs)
+                                                      whole_norm=s.qk_norm_whole, rot_pairs=self.pairs, cap=s.score_cap,
+                                                      head_gated=s.head_gate,
+                                                      conv=(self.w_conv, cache.state, ctx.seq_slots) if self.convolved else None)
             else:
                 q = rt.empty(n, s.n_heads * self.k_row)
                 n_kv = 0 if self.shared_kv else s.n_kv_heads
                 with rt.phase("attn_rope"):
-                    if self.apart:
+                    if self.convolved:
+                        ops.qk_conv_norm_append(qkv, self.w_conv, cache.state, ctx.seq_slots, ctx.cu_seqlens, self.q_gamma,
+                                                self.k_gamma, eps, cos_sin, ctx.tok_seq, ctx.tok_pos, cache.block_table,
+                                                cache.k_pages, cache.v_pages, q, s.n_heads, n_kv, s.head_dim)
+                    elif self.apart:
                         ops.qk_whole_norm_append(qkv, self.q_gamma, self.k_gamma, eps, cos_sin, ctx.tok_seq, ctx.tok_pos,
                                                  cache.block_table, cache.k_pages, cache.v_pages, q, s.n_heads, n_kv,
                                                  s.head_dim, self.v_dim)
@@ -214,7 +252,7 @@ class Attention(Mixer):
                                                 cache.block_table, cache.k_pages, cache.v_pages, q, s.n_heads, n_kv,
                                                 s.head_dim, self.v_dim, self.q_temp, values_are_keys=s.values_are_keys)
                 with self._core_phase(ctx, cache):
-                    self._attend(ctx, q, cache, attn)
+                    self._attend(ctx, q, cache, attn, (qkv, self.gate_col) if s.head_gate else None)
                 if s.out_gate:      # (the decode kernel that starts from the projections applies the gate itself)
                     with rt.phase("attn_gate"):
                         ops.sigmoid_gate(attn, qkv, self.gate_col)
@@ -246,6 +284,8 @@ class Attention(Mixer):
     def _tensor_core_rows(self) -> bool:
         """Whether the heads lie in rows that the tensor-core attention kernels read."""
         s = self.spec
+        if s.score_cap > MAX_FAST_CAP or (s.score_cap > 0.0 and s.slope_base != 0.0):
+            return False
         return (not self.plain_core and ops.attention_mma_supported(s.n_heads, s.n_kv_heads, self.k_row)
                 and self.v_row in (64, self.k_row))
 
@@ -269,11 +309,12 @@ class Attention(Mixer):
                 and (self.position is None or (self.position.tables_by_pair and self.position.half * 2 == s.head_dim))
                 and ops.linear_tc_qkv_supported(x, s.n_heads, s.n_kv_heads, s.head_dim))
 
-    def _attend(self, ctx, q, cache, attn):
+    def _attend(self, ctx, q, cache, attn, head_gate=None):
         """bfloat16 with a head size the tensor-core kernels take: split-key
         decode, tcgen05 prefill for prompts, mma.sync prefill for a few tokens
         per sequence; everything else: the 32-bit kernel."""
-        s, extra = self.spec, {"keep": self.spec.keep_first, "v_lanes": self.v_dim}
+        s, extra = self.spec, {"keep": self.spec.keep_first, "v_lanes": self.v_dim, "cap": self.spec.score_cap,
+                               "head_gate": head_gate}
         if not (self._tensor_core_rows() and ops.attention_mma_supported(s.n_heads, s.n_kv_heads, self.k_row, q, cache.k_pages, attn)):
             ops.attention(q, cache.k_pages, cache.v_pages, cache.block_table, ctx.tok_seq, ctx.tok_pos, attn,
                           s.n_heads, s.n_kv_heads, self.k_row, s.scale, self.span, self.v_row, s.slope_base, self.sinks,

@@ -81,6 +81,18 @@ class NormRequest:
 
 
 @dataclass
+class SublayerClosing:
+    """How a block that norms its sublayers' outputs closes one: residual += post(branch), then (``then`` given) ``out`` =
+    then(residual).  Handed through ``ctx.closing`` to a part that says ``closes_sublayer``: where the part's last kernel holds
+    the branch's rows it does both and sets ``done``; the branch it was given is then not written."""
+    residual: torch.Tensor
+    post: "Norm"
+    then: Optional["Norm"] = None
+    out: Optional[torch.Tensor] = None
+    done: bool = False
+
+
+@dataclass
 class DeferredNorm:
     """A norm's output that is not finished: ``x_gamma`` [n, size] holds residual * gamma in the run's element
     type and ``bins`` the exact accumulators of the sums of squares of the residual's rows.  ``Runtime.linear`` takes

@@ -12,7 +12,7 @@ import torch
 from ..kernels import ops
 from ..weights.params import ParamSpec
 from . import base
-from .base import Block, NormRequest, register_block
+from .base import Block, NormRequest, SublayerClosing, register_block
 from .side import TokenSide
 
 
@@ -164,9 +164,13 @@ class SandwichBlock(Block):
             self.norm2_post = base.build("norm", spec.norm2_post)
         self._parts = tuple(p for p in (self.norm1, self.mixer, self.norm1_post, self.norm2, self.feed_forward,
                                         self.norm2_post) if p is not None)
+        # a layer without a feed-forward may still name the norms around it: their tensors are then optional and not used
+        self._spare = [] if self.feed_forward is not None else [
+            q for n in (spec.norm2, spec.norm2_post) if n is not None for q in base.build("norm", n).params()]
 
     def params(self):
-        return [p for part in self._parts for p in part.params()]
+        spare = [ParamSpec(p.name, p.shape, required=False, init=p.init) for p in self._spare]
+        return [p for part in self._parts for p in part.params()] + spare
 
     def bind(self, tensors, rt):
         self.rt = rt
@@ -183,12 +187,33 @@ class SandwichBlock(Block):
         n = self.norm1
         return NormRequest(n, residual, n.gamma, n.eps, n.size, wants_output=True)
 
+    @staticmethod
+    def _pairs(norm_post, residual, then, out) -> bool:
+        """Whether one pass can close a sublayer with ``norm_post`` and leave ``then``'s output in ``out``."""
+        return (then is not None and out is not None and hasattr(then, "offset") and then.size == norm_post.size
+                and then.gamma.dtype == norm_post.gamma.dtype and ops.rmsnorm_pair_supported(then.size)
+                and residual.dtype == torch.float32)
+
+    def _sublayer(self, ctx, part, run, x, residual, norm_post, then=None, out=None):
+        """residual += norm_post(part(x)), and ``out`` = then(residual) in the same pass where the sizes allow it (returned:
+        whether it was written).  A part that ``closes_sublayer`` may do the closing itself."""
+        closing = None
+        if getattr(part, "closes_sublayer", False) and hasattr(norm_post, "offset") and residual.dtype == torch.float32:
+            takes = self._pairs(norm_post, residual, then, out)
+            closing = SublayerClosing(residual, norm_post, then if takes else None, out if takes else None)
+        ctx.closing = closing
+        try:
+            branch = self._branch(ctx, residual, run, x)
+        finally:
+            ctx.closing = None
+        if closing is not None and closing.done:
+            return closing.out is not None
+        return self._close(ctx, norm_post, branch, residual, then, out)
+
     def _close(self, ctx, norm_post, branch, residual, then, out):
         """residual += norm_post(branch); and, in the same pass where the sizes allow it, ``out`` = then(residual), the
         norm that opens what follows.  Returns whether ``out`` was written."""
-        if (then is not None and out is not None and hasattr(then, "offset") and then.size == norm_post.size
-                and then.gamma.dtype == norm_post.gamma.dtype and ops.rmsnorm_pair_supported(then.size)
-                and residual.dtype == torch.float32):
+        if self._pairs(norm_post, residual, then, out):
             with self.rt.phase("norm"):
                 ops.rmsnorm_pair(branch, residual, norm_post.gamma, norm_post.offset, norm_post.eps, then.gamma,
                                  then.offset, then.eps, out)
@@ -231,22 +256,19 @@ class SandwichBlock(Block):
                     x = handed.output               # the block before left it with its closing norm
                 else:
                     x = self.norm1.forward(ctx, residual)
-                branch = self._branch(ctx, residual, lambda x, out: self.mixer.forward(ctx, x, out, caches[0]), x)
+                then, out = (self.norm2, x2) if ff is not None else (wanted.norm, nxt) if wanted is not None else (None, None)
+                wrote = self._sublayer(ctx, self.mixer, lambda x, o: self.mixer.forward(ctx, x, o, caches[0]), x, residual,
+                                       self.norm1_post, then, out)
                 if ff is not None:
-                    if not self._close(ctx, self.norm1_post, branch, residual, self.norm2, x2):
-                        x2 = None
-                elif wanted is not None and self._close(ctx, self.norm1_post, branch, residual, wanted.norm, nxt):
+                    x2 = x2 if wrote else None
+                elif wrote:
                     wanted.output = nxt
-                else:
-                    self._close(ctx, self.norm1_post, branch, residual, None, None)
             if ff is not None:
                 with rt.scope():
                     x = x2 if x2 is not None else self.norm2.forward(ctx, residual)
-                    branch = self._branch(ctx, residual, lambda x, out: ff.forward(ctx, x, out), x)
-                    if wanted is not None and self._close(ctx, self.norm2_post, branch, residual, wanted.norm, nxt):
+                    then, out = (wanted.norm, nxt) if wanted is not None else (None, None)
+                    if self._sublayer(ctx, ff, lambda x, o: ff.forward(ctx, x, o), x, residual, self.norm2_post, then, out):
                         wanted.output = nxt
-                    else:
-                        self._close(ctx, self.norm2_post, branch, residual, None, None)
         ctx.next_norm = after       # the block that follows finds its request there, fulfilled or not
 
 

@@ -106,17 +106,30 @@ class RoutedExperts(FeedForward):
     branch that the sum over a token's experts takes in, and that kernel, which holds the stream's new rows, leaves the norm
     that reads the stream next; in the form for few tokens the shared part runs in the experts' own two launches.
     ``out_scale`` (and the step's ``ctx.out_scale``) multiply what the part adds to the stream: they enter the
-    tokens' weights, so the sum over a token's experts is scaled at no cost."""
+    tokens' weights, so the sum over a token's experts is scaled at no cost.
+
+    ``scores`` "plain": the softmax over all outputs, the chosen scores as they are; with ``correction`` the choice (not the
+    weights) is by score + correction.  ``identity``: the router's last outputs stand for the input itself; a slot that
+    chose one takes no part in the products and is added where a token's experts are summed.  In a block that norms its
+    sublayers' outputs, the grouped form's sum stays in registers and the same kernel closes the sublayer."""
     scales_output = True
+    closes_sublayer = True
 
     def __init__(self, spec):
         if spec.activation not in GATED_ACTIVATIONS:
             raise UnsupportedModel(f"{spec.name}: activation {spec.activation!r} is not supported")
-        if not 0 < spec.top <= spec.n_experts:
-            raise UnsupportedModel(f"{spec.name}: the top {spec.top} of {spec.n_experts} experts")
-        if spec.scores not in ("chosen", "all", "sigmoid") or spec.weight_on not in ("output", "input"):
+        self.n_outputs = spec.n_experts + spec.identity       # of the router
+        if not 0 < spec.top <= self.n_outputs:
+            raise UnsupportedModel(f"{spec.name}: the top {spec.top} of {self.n_outputs} experts")
+        if spec.identity and (spec.weight_on != "output" or spec.n_groups > 1 or spec.shared_gate):
+            raise UnsupportedModel(f"{spec.name}: identity experts go with weights on the output, without groups and without a "
+                                   "gated shared feed-forward")
+        if spec.correction and spec.scores != "plain":
+            raise UnsupportedModel(f"{spec.name}: a correction of the choice goes with plain scores over all experts")
+        if spec.scores not in ("chosen", "all", "sigmoid", "plain") or spec.weight_on not in ("output", "input"):
             raise UnsupportedModel(f"{spec.name}: router scores of kind {spec.scores!r} on the {spec.weight_on!r}")
-        if spec.scores != "all" and (spec.n_groups > 1 or spec.weight_scale != 1.0 or spec.out_scale != 1.0):
+        if spec.scores not in ("all", "plain") and (spec.n_groups > 1 or spec.weight_scale != 1.0 or spec.out_scale != 1.0) \
+                or spec.scores == "plain" and spec.n_groups > 1:
             raise UnsupportedModel(f"{spec.name}: groups and scales go with scores over all experts")
         if spec.n_groups > 1 and (spec.n_experts % spec.n_groups or not 1 <= spec.keep_groups <= spec.n_groups
                                   or spec.keep_groups * (spec.n_experts // spec.n_groups) < spec.top):
@@ -137,9 +150,11 @@ class RoutedExperts(FeedForward):
             p += [ParamSpec(f"{s.name}.e{e}.gate", (s.intermediate_size, s.hidden_size)),
                   ParamSpec(f"{s.name}.e{e}.up", (s.intermediate_size, s.hidden_size)),
                   ParamSpec(f"{s.name}.e{e}.down", (s.hidden_size, s.intermediate_size))]
-        p.append(ParamSpec(f"{s.name}.router", (s.n_experts, s.hidden_size), init=("normal", 0.5)))
+        p.append(ParamSpec(f"{s.name}.router", (self.n_outputs, s.hidden_size), init=("normal", 0.5)))
         if s.router_bias:
-            p.append(ParamSpec(f"{s.name}.router.b", (s.n_experts,), init=("normal", 0.5)))
+            p.append(ParamSpec(f"{s.name}.router.b", (self.n_outputs,), init=("normal", 0.5)))
+        if s.correction:
+            p.append(ParamSpec(f"{s.name}.correction", (self.n_outputs,), init=("normal", 0.1)))
         if s.shared_gate:
             p.append(ParamSpec(f"{s.shared.name}.sg", (1, s.hidden_size), init=("normal", 0.5)))
         return p + (self.shared.params() if self.shared is not None else [])
@@ -163,6 +178,7 @@ class RoutedExperts(FeedForward):
             self.w_gate, self.w_up = gate, up
         del gate, up
         self.w_router, self.b_router = tensors[f"{s.name}.router"], tensors.get(f"{s.name}.router.b")
+        self.correction = tensors.get(f"{s.name}.correction") if s.correction else None
         if s.shared_gate:
             self.w_router = torch.cat([self.w_router, tensors.pop(f"{s.shared.name}.sg")], dim=0).contiguous()
         if self.shared is not None:
@@ -180,8 +196,10 @@ class RoutedExperts(FeedForward):
         if isinstance(x, DeferredNorm):
             x = x.finish(ctx)
         n = x.shape[0]
-        if getattr(ctx, "branch_is_fresh", False):
-            raise UnsupportedModel(f"{s.name}: routed experts add into the stream they are given")
+        # a branch of its own that is written, not added to (a block that norms its sublayers' outputs), and how it is closed
+        fresh, closing_pair = bool(getattr(ctx, "branch_is_fresh", False)), getattr(ctx, "closing", None)
+        if fresh and self.own_shared:
+            raise UnsupportedModel(f"{s.name}: routed experts with a gated shared feed-forward add into the stream they are given")
         ids = rt.empty(n, s.top, dtype=torch.int32)
         weights = rt.empty(n, s.top, dtype=torch.float32)
         out_scale = float(getattr(ctx, "out_scale", 1.0)) * s.out_scale
@@ -189,13 +207,15 @@ class RoutedExperts(FeedForward):
         gate = rt.empty(n, dtype=torch.float32) if s.shared_gate else None
         if s.scores == "all":
             scoring = ("all", s.n_groups, s.keep_groups, s.weight_scale * out_scale)
+        elif s.scores == "plain":
+            scoring = ("plain", self.correction, s.weight_scale * out_scale)
         elif s.scores == "sigmoid" and out_scale == 1.0:
             scoring = ("sigmoid",)
         elif out_scale != 1.0:
             raise UnsupportedModel(f"{s.name}: a scaled output goes with scores over all experts")
         with rt.phase("moe_route", self.w_router, n):
             many = n >= ROUTER_PRODUCT_FROM_TOKENS and rt.tensor_cores_take(x.dtype, self.w_router, s.hidden_size)
-            if not many and ops.moe_router_fits(s.n_experts, s.hidden_size):
+            if not many and ops.moe_router_fits(self.n_outputs, s.hidden_size):
                 ops.moe_router(x, self.w_router, self.b_router, s.top, ids, weights, scoring, gate)
             else:
                 # many tokens: the logits as a product of their own (bfloat16 operands are multiplied exactly and
@@ -210,6 +230,7 @@ class RoutedExperts(FeedForward):
         esize = self.w_gate.element_size()
         experts_read = min(S, s.n_experts)
         on_input = s.weight_on == "input"
+        identity_x = x if s.identity else None
         then = getattr(ctx, "next_norm", None)
         own = self.own_shared
         if self.grouped and S >= GROUPED_FROM_SLOTS and not (own and not ops.moe_combine_closes(h)):
@@ -241,8 +262,16 @@ class RoutedExperts(FeedForward):
                     and hasattr(then.norm, "closing_rms") and ops.moe_combine_closes(h):
                 then.output = norm_output_buffer(ctx, rt, residual.shape)
                 closing = then.norm.closing_rms(then.output)
+            if (closing_pair is not None and fresh and self.shared is None and not on_input and ops.moe_combine_closes(h)):
+                # the sublayer's closing norm, the stream's sum and the next norm in the pass that adds a token's experts up
+                c = closing_pair
+                with rt.phase("moe_combine", nbytes=4.0 * S * h + 10.0 * n * h):
+                    ops.moe_combine_pair(y, rows, weights, c.residual, (c.post.gamma, c.post.offset, c.post.eps),
+                                         None if c.then is None else (c.then.gamma, c.then.offset, c.then.eps, c.out), identity_x)
+                c.done = True
+                return
             with rt.phase("moe_combine", nbytes=4.0 * S * h + (12.0 if own else 8.0) * n * h + (2.0 * n * h if closing else 0.0)):
-                ops.moe_combine(y, rows, None if on_input else weights, residual, s.top, branch, gate, closing)
+                ops.moe_combine(y, rows, None if on_input else weights, residual, s.top, branch, gate, closing, identity_x, fresh)
         elif own:
             # few tokens: the shared feed-forward's rows in the experts' two launches
             sh = self.shared
@@ -256,11 +285,15 @@ class RoutedExperts(FeedForward):
             mid = rt.empty(S, f)
             with rt.phase("moe_experts", nbytes=experts_read * 3.0 * f * h * esize, flops=6.0 * S * f * h):
                 ops.moe_experts(x, self.w_gate, self.w_up, self.w_down, ids, weights, mid, residual, s.activation, s.limit,
-                                on_input)
+                                on_input, identity=bool(s.identity), fresh=fresh)
         if self.shared is not None and not own:
             if out_scale != 1.0:
                 raise UnsupportedModel(f"{s.name}: a shared expert under a scaled output")
-            self.shared.forward(ctx, x, residual)
+            ctx.branch_is_fresh = False         # the branch holds the experts' sum by now
+            try:
+                self.shared.forward(ctx, x, residual)
+            finally:
+                ctx.branch_is_fresh = fresh
 
 
 @register_feed_forward("dense_mlp")

@@ -16,6 +16,7 @@ class RMSNorm(Norm):
         self.size, self.eps, self.name = spec.size, spec.eps, spec.name
         self.tensor = spec.name + spec.suffix
         self.offset = float(spec.offset)
+        self.gain = float(spec.gain)
         self.gamma = None
 
     def params(self):
@@ -24,6 +25,9 @@ class RMSNorm(Norm):
     def bind(self, tensors, rt):
         self.rt = rt
         self.gamma = tensors[self.tensor]
+        if self.gain != 1.0:        # a factor on the output rides on the weight, in 32-bit
+            self.gamma = (self.gamma.to(torch.float32) + self.offset) * self.gain
+            self.offset = 0.0
         # what a product that carries this norm multiplies with: the weight with its offset, in 32-bit
         self.carried_gamma = self.gamma if self.offset == 0.0 else self.gamma.to(torch.float32) + self.offset
 
