@@ -18,7 +18,8 @@ with host token ids in and out.  The line also carries a prefill measurement (on
 layers of equal size: a 2 048-token prompt, decode at batch 8, and every phase's time and roofline fraction), and
 ``pikalorn`` (that design at two widths beside Zevivik and Romepel layers of equal size, measured the same way),
 ``vodalorn`` (that design at two widths beside Pikalorn and Zevivik layers of equal size, measured the same way), ``gekilix`` (that design at two widths beside Zevivik and Romepel layers
-of equal size, measured the same way).
+of equal size, measured the same way), ``vuvalorn`` (that design at two widths beside Zevivik and Pikalorn layers of equal
+size, measured the same way).
 """
 from __future__ import annotations
 
@@ -240,6 +241,7 @@ WORKLOADS = {
     "pikalorn": dict(model="8b"),
     "vodalorn": dict(model="8b"),
     "gekilix": dict(model="8b"),
+    "vuvalorn": dict(model="8b"),
 }
 
 # `--workload romepel`: the Romepel design (recurrent gla layers, windowed attention with a distance bias, sandwich
@@ -487,6 +489,42 @@ def gekilix_configs(z: dict):
     return gek, zev, rom
 
 
+# `--workload vuvalorn`: the Vuvalorn design (convolved keys that are the values, capped scores, a gate per head, sandwich
+# norms, clamped gated feed-forwards and experts some of which are the identity, a looped range of layers) at sizes that
+# resemble a real model's layers, beside the two closest existing designs at equal width, layer runs and head counts, every
+# key visible: Zevivik (the same feed-forwards and loop, experts without identities; a fused q/k/v epilogue) and Pikalorn
+# (values that are the keys and a gate, dense feed-forwards).
+VUVALORN_SIZES = {
+    "2048": dict(width=2048, heads=16, kv_heads=4, dim=128, conv=4, inter=6144, experts=16, identity=4, top=2, vocab=32768),
+    "4096": dict(width=4096, heads=32, kv_heads=8, dim=128, conv=4, inter=12288, experts=16, identity=4, top=2, vocab=65536),
+}
+
+
+def vuvalorn_configs(z: dict):
+    """(Vuvalorn configuration, Zevivik's and Pikalorn's of equal size).  Five layers of which the middle three run twice:
+    eight layer runs, four of them with routed experts."""
+    from nncpu_b200.config import config_from_dict
+    rot = {"base": 1000000.0, "dims": z["dim"]}
+    heads = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5, "rot": rot}
+    router = {"experts": z["experts"], "top": z["top"]}
+    loop = {"start": 1, "stop": 4, "times": 2}
+
+    def model(architecture, mixer, dense, moe, **more):
+        layers = [{"type": "attention", "mixer": mixer, "mlp": f} for f in (dense, moe, dense, moe, dense)]
+        return config_from_dict({"architecture": architecture, "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6},
+                                 "embedding": {"scale": 1.0}, "layers": layers, **more})
+
+    vuv = model("Vuvalorn", dict(heads, conv=z["conv"], softcap=30.0), {"kind": "dense", "ff": z["inter"], "limit": 7.0},
+                {"kind": "moe", "expert": {"ff": z["inter"] // 2}, "router": dict(router, identity=z["identity"])}, loop=loop,
+                logit_scale=0.5)
+    zev = model("Zevivik", dict(heads, mask={"size": CONTEXT}), {"kind": "dense", "ff": z["inter"]},
+                {"kind": "moe", "expert": {"ff": z["inter"] // 2, "limit": 7.0}, "router": router}, loop=loop)
+    pik = config_from_dict({"architecture": "Pikalorn", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6},
+                            "embedding": {"scale": 1.0},
+                            "layers": [{"type": "attention", "mixer": heads, "mlp": {"kind": "dense", "ff": z["inter"]}}] * 8})
+    return vuv, zev, pik
+
+
 def phase_table(totals: dict, calls: int, pk: dict) -> dict:
     """Per phase of the profiler: milliseconds per step and, where the phase states its bytes and operations, the
     fraction of the roofline (the slower of bytes / copy bandwidth and operations / tensor throughput, over the time)."""
@@ -613,6 +651,18 @@ def run_gekilix() -> dict:
         out["sizes"][name] = {"config": z, "gekilix": run_design_point(gek, z["vocab"], pk),
                               "zevivik_same_size": run_design_point(zev, z["vocab"], pk),
                               "romepel_same_size": run_design_point(rom, z["vocab"], pk)}
+    return out
+
+
+def run_vuvalorn() -> dict:
+    pk = peaks()
+    out = {"workload": "vuvalorn", "dtype": "bf16", "peaks": pk["source"], "prompt": PROMPT,
+           "data": "synthetic: random weights, uniform random token ids", "sizes": {}}
+    for name, z in VUVALORN_SIZES.items():
+        vuv, zev, pik = vuvalorn_configs(z)
+        out["sizes"][name] = {"config": z, "vuvalorn": run_design_point(vuv, z["vocab"], pk),
+                              "zevivik_same_size": run_design_point(zev, z["vocab"], pk),
+                              "pikalorn_same_size": run_design_point(pik, z["vocab"], pk)}
     return out
 
 
@@ -781,7 +831,7 @@ def main() -> int:
         return 0
     if args.workload:
         special = {"long-context": run_long_context, "romepel": run_romepel, "zevivik": run_zevivik,
-                   "pikalorn": run_pikalorn, "vodalorn": run_vodalorn, "gekilix": run_gekilix}
+                   "pikalorn": run_pikalorn, "vodalorn": run_vodalorn, "gekilix": run_gekilix, "vuvalorn": run_vuvalorn}
         print(json.dumps(special[args.workload]() if args.workload in special else run_workload(args.workload)))
         return 0
     model = Model.random(cfg, seed=0, dtype="bfloat16", device="cuda:0")

@@ -66,10 +66,12 @@ struct AttnParams {
     int vo;         // lanes of a head in the output (at most the value rows' VD)
     float slope_base;   // b != 0: head h takes 2^(-b (h + 1) / n_heads) * (query position - key position) off its scaled scores
     const float* sinks; // float32 [n_heads] or null: exp(sinks[h]) joins the denominator of head h's softmax, with no key and no value
-    // The weight of a key is 2^(u score_mul + score_add - m): without a cap u is the unscaled score, score_mul = scale2 and
-    // score_add = 0.  With a cap c (kCap) the score is c tanh(z / c) = c - 2 c / (1 + exp(2 z / c)), so
-    // u = -1 / (1 + 2^(cap_in * unscaled score)), score_mul = 2 c log2(e) and score_add = c log2(e).
-    float cap_in, score_mul, score_add;
+    // The weight of a key is 2^(u score_mul - m): without a cap u is the unscaled score and score_mul = scale2.  With a cap c
+    // (kCap) u = tanh(z / c), z the scaled score, and score_mul = c log2(e).  Where a warp's page holds no score beyond
+    // kTanhRange of the cap, u is a polynomial in x = cap_x * unscaled score (cap_x = scale / c): a matter of multiply-adds,
+    // two scores an instruction.  Elsewhere u = 1 - 2 / (1 + 2^(cap_in * unscaled score)): two more special-function
+    // results a score, which is what the softmax has least of.
+    float cap_in, cap_x, cap_small, score_mul;
     const float* head_gate;   // or null: row t (at t * gate_ld) holds a logit a head, whose sigmoid multiplies the head's output
     long gate_ld;
     int* status;
@@ -99,6 +101,26 @@ __device__ __forceinline__ float fast_exp2(float x) {
     float y;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
+}
+
+// tanh(x) = x P(x^2) for |x| <= kTanhRange, within 1.6e-6 (least squares over that range, reweighted towards equal
+// extremes).
+constexpr float kTanhRange = 1.2f;
+
+__device__ __forceinline__ uint64_t pair_of(float a, float b) {
+    uint64_t d;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(a), "f"(b));
+    return d;
+}
+__device__ __forceinline__ uint64_t fma_pair(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ uint64_t mul_pair(uint64_t a, uint64_t b) {
+    uint64_t d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
 }
 
 __device__ __forceinline__ float fast_rcp(float x) {
@@ -388,10 +410,30 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
                         u[c] = __float_as_uint(fmaf(bias_per_key, (float)c - far, __uint_as_float(u[c])));
                 }
                 if (kCap) {
+                    float big[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
-                    for (int c = 0; c < 64; ++c) {
-                        const float e = fast_exp2(__uint_as_float(u[c]) * p.cap_in);
-                        u[c] = __float_as_uint(fast_rcp(-1.0f - e));
+                    for (int c = 0; c < 64; ++c) big[c & 3] = fmaxf(big[c & 3], fabsf(__uint_as_float(u[c])));
+                    const float most = fmaxf(fmaxf(big[0], big[1]), fmaxf(big[2], big[3]));
+                    if (__all_sync(0xffffffffu, most <= p.cap_small)) {
+                        constexpr float kTanh[6] = {0.9999824762f, -0.3329640925f, 0.1310810596f, -0.0478774495f, 0.0132463686f,
+                                                    -0.0018748625f};
+                        const uint64_t k = pair_of(p.cap_x, p.cap_x);
+#pragma unroll
+                        for (int c = 0; c < 64; c += 2) {
+                            const uint64_t x = mul_pair(pair_of(__uint_as_float(u[c]), __uint_as_float(u[c + 1])), k);
+                            const uint64_t y = mul_pair(x, x);
+                            uint64_t t = fma_pair(y, pair_of(kTanh[5], kTanh[5]), pair_of(kTanh[4], kTanh[4]));
+#pragma unroll
+                            for (int i = 3; i >= 0; --i) t = fma_pair(y, t, pair_of(kTanh[i], kTanh[i]));
+                            t = mul_pair(x, t);
+                            asm("mov.b64 {%0, %1}, %2;" : "=r"(u[c]), "=r"(u[c + 1]) : "l"(t));
+                        }
+                    } else {
+#pragma unroll
+                        for (int c = 0; c < 64; ++c) {
+                            const float e = fast_exp2(__uint_as_float(u[c]) * p.cap_in);
+                            u[c] = __float_as_uint(fmaf(-2.0f, fast_rcp(1.0f + e), 1.0f));
+                        }
                     }
                 }
                 if (!((kb >= lim_lo || kb + 63 < p.keep) && kb + 63 <= lim_hi)) {
@@ -402,7 +444,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
                 }
             };
             auto weights = [&]() {
-                const float neg_m = m_ref == -INFINITY ? 0.0f : (kCap ? p.score_add : 0.0f) - m_ref;
+                const float neg_m = m_ref == -INFINITY ? 0.0f : 0.0f - m_ref;
                 float sm[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
                 for (int hf = 0; hf < 2; ++hf) {
@@ -434,8 +476,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
                         for (int c = 0; c < 64; ++c) mx[c & 3] = fmaxf(mx[c & 3], __uint_as_float(u[c]));
                     }
                 }
-                const float tmax = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * p.score_mul
-                                   + (kCap ? p.score_add : 0.0f);                                // the factor is positive
+                const float tmax = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * p.score_mul;   // the factor is positive
                 float alpha = 1.0f;
                 if (tmax > m_ref) {
                     alpha = fast_exp2(m_ref - tmax);    // 0 when nothing was seen yet
@@ -641,8 +682,9 @@ extern "C" int nncpu_attention_prefill_tc(const void* q, const void* k_pages, co
     p.sinks = sinks;
     const ScoreCap sc = score_cap(scale, cap);
     p.cap_in = sc.in;
-    p.score_mul = cap > 0.0f ? 2.0f * sc.out : p.scale2;
-    p.score_add = sc.out;
+    p.cap_x = cap > 0.0f ? scale / cap : 0.0f;
+    p.cap_small = cap > 0.0f ? kTanhRange * cap / scale : 0.0f;
+    p.score_mul = cap > 0.0f ? sc.out : p.scale2;
     p.head_gate = head_gate;
     p.gate_ld = gate_ld;
     p.status = status;

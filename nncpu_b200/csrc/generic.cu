@@ -798,6 +798,103 @@ qk_conv_norm_append_kernel(const float* __restrict__ proj, int ld, const ShortCo
     float g[kEpl];
 #pragma unroll
     for (int e = 0; e < kEpl; ++e) g[e] = gamma != nullptr && lane * kEpl + e < hd ? ld_f(gamma, lane * kEpl + e, g_dt) : 1.0f;
+    if (kTaps > 1 && t0 + kConvRun <= n_tok) {
+        const int s = tok_seq[t0];
+        if (s >= 0 && s == tok_seq[t0 + kConvRun - 1]) {
+            // the usual case of a prompt: all the run's tokens are one sequence's, at consecutive positions.  No branch
+            // between tokens, so that their sums and stores overlap.
+            const int first = cu_seqlens[s], end = cu_seqlens[s + 1], pos0 = tok_pos[t0];
+            if (t0 - (kTaps - 1) >= first) {
+#pragma unroll
+                for (int j = 0; j + 1 < kTaps; ++j)
+                    ld_lanes<kEpl, kVec>(proj + (size_t)(t0 - (kTaps - 1) + j) * ld + ch0, lane, hd, win[j]);
+            } else {
+                const int slot = cv.seq_slots[s];
+                const float* kept = conv_copy(cv, slot, conv_copy_in_use(cv, slot, tok_pos[first]));
+#pragma unroll
+                for (int j = 0; j + 1 < kTaps; ++j) {
+                    const int at = t0 - (kTaps - 1) + j;
+                    ld_lanes<kEpl, kVec>(at >= first ? proj + (size_t)at * ld + ch0
+                                                     : kept + (size_t)(kTaps - 1 + at - first) * cv.C + ch0, lane, hd, win[j]);
+                }
+            }
+            if (t0 + kConvRun > end - (kTaps - 1)) {        // the sequence's last inputs are among these (or all its tokens)
+                const int slot = cv.seq_slots[s], copy = conv_copy_in_use(cv, slot, tok_pos[first]);
+                float* next = conv_copy(cv, slot, 1 - copy);
+#pragma unroll
+                for (int i = 0; i < kConvRun; ++i)          // (a run has at least taps - 1 tokens: nothing older is kept)
+                    if (t0 + i >= end - (kTaps - 1))
+                        st_lanes<kEpl, kVec>(next + (size_t)(t0 + i - (end - (kTaps - 1))) * cv.C + ch0, lane, hd, u[kTaps > 0 ? i : 0]);
+                if (t0 + kConvRun == end && h == 0 && lane == 0) conv_mark(cv, slot, 1 - copy, pos0 + kConvRun);
+            }
+            const int* table = block_table + (size_t)s * bt_stride;
+            const int page0 = is_q ? 0 : table[pos0 / kPage], page1 = is_q ? 0 : table[(pos0 + kConvRun - 1) / kPage];
+            constexpr int kAtOnce = 4;
+#pragma unroll
+            for (int i0 = 0; i0 < kConvRun; i0 += kAtOnce) {
+                float x[kAtOnce][kEpl], ss[kAtOnce];
+                float2 c[kAtOnce][kEpl / 2];
+#pragma unroll
+                for (int i = 0; i < kAtOnce; ++i) {
+#pragma unroll
+                    for (int e = 0; e < kEpl; e += 2) {
+                        const int p = (lane * kEpl + e) >> 1;
+                        c[i][e / 2] = cs != nullptr && p < half ? cs[(size_t)(t0 + i0 + i) * half + p] : make_float2(1.0f, 0.0f);
+                    }
+                }
+#pragma unroll
+                for (int i = 0; i < kAtOnce; ++i) {
+                    ss[i] = 0.0f;
+#pragma unroll
+                    for (int e = 0; e < kEpl; ++e) {
+                        float a = 0.0f;
+#pragma unroll
+                        for (int j = 0; j < kTaps; ++j) {      // the oldest input first, as below
+                            const int back = kTaps - 1 - j, at = i0 + i - back;
+                            a = fmaf(w[j][e], at >= 0 ? u[kTaps > 0 && at >= 0 ? at : 0][e] : win[at + kKeep >= 0 && at < 0 ? at + kKeep : 0][e], a);
+                        }
+                        x[i][e] = a;
+                        ss[i] = fmaf(a, a, ss[i]);
+                    }
+                }
+                if (!is_q) {
+#pragma unroll
+                    for (int i = 0; i < kAtOnce; ++i) {
+                        const int pos = pos0 + i0 + i, page = pos / kPage == pos0 / kPage ? page0 : page1;
+                        if (page >= 0)
+                            st_row<kEpl>(v_pages, (((size_t)page * n_kv + (h - n_heads)) * kPage + pos % kPage) * vp, kv_dt, vp, lane, x[i]);
+                    }
+                }
+                if (gamma != nullptr) {
+#pragma unroll
+                    for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+                        for (int i = 0; i < kAtOnce; ++i) ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], o);
+#pragma unroll
+                    for (int i = 0; i < kAtOnce; ++i) {
+                        const float scale = 1.0f / sqrtf(ss[i] * (1.0f / (float)hd) + eps);
+#pragma unroll
+                        for (int e = 0; e < kEpl; ++e) x[i][e] = (x[i][e] * scale) * g[e];
+                    }
+                }
+#pragma unroll
+                for (int i = 0; i < kAtOnce; ++i) {
+#pragma unroll
+                    for (int e = 0; e < kEpl; e += 2) {
+                        const float a = x[i][e], b = x[i][e + 1];
+                        x[i][e] = fmaf(c[i][e / 2].x, a, 0.0f - c[i][e / 2].y * b);      // (the same roundings as below)
+                        x[i][e + 1] = fmaf(c[i][e / 2].y, a, c[i][e / 2].x * b);
+                    }
+                    const int pos = pos0 + i0 + i, page = pos / kPage == pos0 / kPage ? page0 : page1;
+                    if (is_q)
+                        st_row<kEpl>(q_out, ((size_t)(t0 + i0 + i) * n_heads + h) * qp, q_dt, qp, lane, x[i]);
+                    else if (page >= 0)
+                        st_row<kEpl>(k_pages, (((size_t)page * n_kv + (h - n_heads)) * kPage + pos % kPage) * qp, kv_dt, qp, lane, x[i]);
+                }
+            }
+            return;
+        }
+    }
     int seq = -1, first = 0, end = 0, slot = 0, copy = 0;
 #pragma unroll
     for (int i = 0; i < kConvRun; ++i) {
@@ -880,8 +977,8 @@ qk_conv_norm_append_kernel(const float* __restrict__ proj, int ld, const ShortCo
                 if (p < half) {
                     const float2 c = cs[(size_t)t * half + p];
                     const float a = x[e], b = x[e + 1];
-                    x[e] = c.x * a - c.y * b;
-                    x[e + 1] = c.y * a + c.x * b;
+                    x[e] = fmaf(c.x, a, 0.0f - c.y * b);
+                    x[e + 1] = fmaf(c.y, a, c.x * b);
                 }
             }
         }
@@ -956,7 +1053,7 @@ attention_kernel(const void* __restrict__ q, int q_dt, const void* __restrict__ 
                  int gate_ld) {
     extern __shared__ float smem[];
     float* qs = smem;                       // hd
-    float* p = smem + hd;                   // kAttnThreads
+    float* p = smem + ((hd + 1) & ~1);      // kAttnThreads (the offsets behind it are 8 bytes each)
     long long* row = (long long*)(p + kAttnThreads);  // kAttnThreads element offsets of the chunk's rows
     __shared__ float scratch[33];
 

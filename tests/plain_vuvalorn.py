@@ -149,10 +149,21 @@ def route(scores, correction, top):
     return ids, scores[ids]
 
 
-def routed_experts(h, f, w, name):
-    """The first ``experts`` outputs of the router are experts with tensors, the last ``identity`` hand the input on."""
+def margins(scores, correction, top):
+    """How far apart the last chosen and the first not chosen lie, per token (infinity where everything is chosen)."""
+    if top == scores.shape[1]:
+        return np.full(len(scores), np.inf)
+    key = np.sort(scores + correction, axis=1)[:, ::-1]
+    return key[:, top - 1] - key[:, top]
+
+
+def routed_experts(h, f, w, name, note=None):
+    """The first ``experts`` outputs of the router are experts with tensors, the last ``identity`` hand the input on.
+    ``note``: a list that receives the choices' margins."""
     n = f["router"]["experts"]
     s = softmax(h @ w[f"{name}.router"].T)
+    if note is not None:
+        note.append(margins(s, w[f"{name}.correction"], f["router"]["top"]))
     out = np.zeros_like(h)
     for t in range(h.shape[0]):
         for e, weight in zip(*route(s[t], w[f"{name}.correction"], f["router"]["top"])):
@@ -160,8 +171,8 @@ def routed_experts(h, f, w, name):
     return out
 
 
-def feed_forward(h, f, w, name):
-    return clamped_gated(h, w, name, f["limit"]) if f["kind"] == "dense" else routed_experts(h, f, w, name)
+def feed_forward(h, f, w, name, note=None):
+    return clamped_gated(h, w, name, f["limit"]) if f["kind"] == "dense" else routed_experts(h, f, w, name, note)
 
 
 # -- the model ------------------------------------------------------------------------------
@@ -176,8 +187,8 @@ def runs(cfg):
     return [(i, None) for i in range(a)] + body + [(i, None) for i in range(b, n)]
 
 
-def forward(cfg, w, tokens, with_streams=False):
-    """Logits [T, vocab] of a whole sequence (and the stream after every layer run)."""
+def forward(cfg, w, tokens, with_streams=False, note=None):
+    """Logits [T, vocab] of a whole sequence (and the stream after every layer run); ``note``: see ``routed_experts``."""
     eps = cfg["norm"]["eps"]
     x = w["embed"][np.asarray(tokens)] * (cfg.get("embedding") or {}).get("scale", 1.0)
     streams = []
@@ -188,7 +199,7 @@ def forward(cfg, w, tokens, with_streams=False):
         y = attention(norm(x, w[f"l{i}.norm1"], eps), layer["mixer"], w, f"l{i}.mix", eps)
         x = x + norm(y, w[f"l{i}.norm1b"], eps)
         if layer.get("mlp"):
-            y = feed_forward(norm(x, w[f"l{i}.norm2"], eps), layer["mlp"], w, f"l{i}.mlp")
+            y = feed_forward(norm(x, w[f"l{i}.norm2"], eps), layer["mlp"], w, f"l{i}.mlp", note)
             x = x + norm(y, w[f"l{i}.norm2b"], eps)
         streams.append(x.copy())
     logits = norm(x, w["final.norm"], eps) @ w["embed"].T * cfg.get("logit_scale", 1.0)
