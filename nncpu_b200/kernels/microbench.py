@@ -6,7 +6,8 @@ GFLOP/s for its row kernels and one attention block.
     python -m nncpu_b200.kernels.microbench linear M N K [--epilogue swiglu] [--accumulate] [--norm producer|consumer]
     python -m nncpu_b200.kernels.microbench linear-qkv TOKENS [--hidden K]
     python -m nncpu_b200.kernels.microbench attention-decode BATCH CONTEXT [--splits S] [--cluster] [--from-projections]
-    python -m nncpu_b200.kernels.microbench attention-prefill BATCH TOKENS
+    python -m nncpu_b200.kernels.microbench attention-prefill BATCH TOKENS [--cap C]
+    python -m nncpu_b200.kernels.microbench qk-conv BATCH TOKENS [--taps 4]
     python -m nncpu_b200.kernels.microbench rmsnorm ROWS DIM
     python -m nncpu_b200.kernels.microbench gla BATCH TOKENS [--columns 2|4]
     python -m nncpu_b200.kernels.microbench delta BATCH TOKENS [--lanes 4|8|16|32] [--columns 1|2] [--channel-decay]
@@ -169,16 +170,39 @@ def attention_prefill(args) -> None:
     q = torch.randn(b * t, nh * hd, device=DEV).bfloat16()
     out = torch.empty_like(q)
     if args.legacy:
-        run = lambda: ops.attention_prefill_mma(q, kp, vp, table, cu, pos, out, b, nh, nkv, hd, 1 / math.sqrt(hd), 0)
+        run = lambda: ops.attention_prefill_mma(q, kp, vp, table, cu, pos, out, b, nh, nkv, hd, 1 / math.sqrt(hd), 0, cap=args.cap)
     else:
         status = torch.zeros(1, dtype=torch.int32, device=DEV)
         run = lambda: ops.attention_prefill_tc(q, kp, vp, table, cu, pos, out, status, b, nh, nkv, hd,
-                                               1 / math.sqrt(hd), 0)
+                                               1 / math.sqrt(hd), 0, cap=args.cap)
     ms = _time([run] * 3, args.once)
     if not args.legacy and int(status.item()):
         raise SystemExit(f"the kernel gave up waiting (status {int(status.item())})")
     flops = 4.0 * nh * hd * b * t * (t + 1) / 2
-    print(f"attention-prefill batch={b} tokens={t}: {ms * 1e3:.1f} us, {flops / ms / 1e9:.0f} TFLOP/s (causal)")
+    print(f"attention-prefill batch={b} tokens={t}{f' cap={args.cap:g}' if args.cap else ''}: {ms * 1e3:.1f} us, {flops / ms / 1e9:.0f} TFLOP/s (causal)")
+
+
+def qk_conv(args) -> None:
+    """The stage between the q/k product and the attention of a layer with short convolutions: convolution, per-head norm,
+    rotation of half a head's lanes, queries, keys and values to their places, the state left advanced."""
+    nh, nkv, hd, b, t, taps = args.heads, args.kv_heads, args.head_dim, args.batch, args.tokens, args.taps
+    n, c = b * t, (nh + nkv) * hd
+    sets, table = _cache(b, t, nkv, hd, 1)
+    kp, vp = sets[0]
+    proj = torch.randn(n, c + nh, device=DEV)
+    w = torch.randn(taps, c, device=DEV)
+    state = torch.zeros(b + 1, ops.conv_state_floats(taps, c), device=DEV)
+    slots = torch.arange(b, dtype=torch.int32, device=DEV)
+    cu = torch.arange(0, n + 1, t, dtype=torch.int32, device=DEV)
+    pos = torch.arange(t, dtype=torch.int32, device=DEV).repeat(b)
+    seq = torch.arange(b, dtype=torch.int32, device=DEV).repeat_interleave(t)
+    gamma = torch.ones(hd, device=DEV).bfloat16()
+    cs = torch.randn(n, hd // 4, 2, device=DEV)
+    q = torch.empty(n, nh * hd, device=DEV, dtype=torch.bfloat16)
+    ms = _time([lambda: ops.qk_conv_norm_append(proj, w, state, slots, cu, gamma, gamma, 1e-6, cs, seq, pos, table, kp, vp, q, nh, nkv,
+                                                hd)] * 3, args.once)
+    nbytes = 4.0 * n * c + 2.0 * n * (nh + 2 * nkv) * hd + 4.0 * cs.numel()
+    print(f"qk-conv batch={b} tokens={t} heads={nh}/{nkv} taps={taps}: {ms * 1e3:.1f} us, {nbytes / ms / 1e6:.0f} GB/s of inputs and outputs")
 
 
 def rmsnorm(args) -> None:
@@ -297,10 +321,16 @@ def main(argv=None) -> int:
         p.add_argument("--heads", type=int, default=32); p.add_argument("--kv-heads", type=int, default=8)
         p.add_argument("--head-dim", type=int, default=128); p.add_argument("--splits", type=int, default=0)
         p.add_argument("--cluster", action="store_true", help="merge the splits inside a cluster (at most 8)")
+        p.add_argument("--cap", type=float, default=0.0, help="prefill: scores are capped, C tanh(z / C)")
         p.add_argument("--legacy", action="store_true", help="prefill: the mma.sync kernel instead of tcgen05")
         p.add_argument("--from-projections", action="store_true",
                        help="decode: start from the float32 q/k/v projections (norm, rotation, append inside), as a step does")
         p.set_defaults(fn=fn)
+    p = sub.add_parser("qk-conv")
+    p.add_argument("batch", type=int); p.add_argument("tokens", type=int)
+    p.add_argument("--heads", type=int, default=32); p.add_argument("--kv-heads", type=int, default=8)
+    p.add_argument("--head-dim", type=int, default=128); p.add_argument("--taps", type=int, default=4)
+    p.set_defaults(fn=qk_conv)
     p = sub.add_parser("linear-qkv")
     p.add_argument("tokens", type=int); p.add_argument("--hidden", type=int, default=4096)
     p.add_argument("--heads", type=int, default=32); p.add_argument("--kv-heads", type=int, default=8)
