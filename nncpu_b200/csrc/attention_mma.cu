@@ -505,7 +505,8 @@ __device__ __forceinline__ float row_squares(const float* __restrict__ src, int 
     return ss;
 }
 
-template <int HD, int VD, int NT, bool kCluster, bool kFused>
+// kMore: with a cap on the scores or a short convolution before the heads; kernels without either do not carry them.
+template <int HD, int VD, int NT, bool kCluster, bool kFused, bool kMore>
 __global__ void __launch_bounds__(128, 2)
 decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_pages,
                    const __nv_bfloat16* __restrict__ v_pages, const int* __restrict__ block_table, int bt_stride,
@@ -584,7 +585,7 @@ decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restri
         const float temp = f.temp_coef != 0.0f ? 1.0f + f.temp_coef * logf((float)((pos + 1) / f.temp_every) + 1.0f) : 1.0f;
         // A short convolution: every block reads the inputs kept from earlier steps; the first split's blocks leave those
         // of the queries advanced in the state's other copy, the owner those of its key.
-        const ShortConv* conv = f.conv.w != nullptr ? &f.conv : nullptr;
+        const ShortConv* conv = kMore && f.conv.w != nullptr ? &f.conv : nullptr;
         const float* kept = nullptr;
         float* next = nullptr;
         if (conv != nullptr) {
@@ -691,17 +692,17 @@ decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restri
                     b_hi[j] = slope2 * (float)(pos - (k0 + r + 8));
                 }
             }
-            if (cap.out > 0.0f) {
-#pragma unroll
-                for (int e = 0; e < 4; ++e) sv[e] = capped_score(sv[e], cap);
+            if (kMore && cap.out > 0.0f) {
+                sv[0] = lo_ok ? capped_score(sv[0], cap) - b_lo[0] : -INFINITY;
+                sv[1] = lo_ok ? capped_score(sv[1], cap) - b_lo[1] : -INFINITY;
+                sv[2] = hi_ok ? capped_score(sv[2], cap) - b_hi[0] : -INFINITY;
+                sv[3] = hi_ok ? capped_score(sv[3], cap) - b_hi[1] : -INFINITY;
             } else {
-#pragma unroll
-                for (int e = 0; e < 4; ++e) sv[e] *= scale2;
+                sv[0] = lo_ok ? sv[0] * scale2 - b_lo[0] : -INFINITY;
+                sv[1] = lo_ok ? sv[1] * scale2 - b_lo[1] : -INFINITY;
+                sv[2] = hi_ok ? sv[2] * scale2 - b_hi[0] : -INFINITY;
+                sv[3] = hi_ok ? sv[3] * scale2 - b_hi[1] : -INFINITY;
             }
-            sv[0] = lo_ok ? sv[0] - b_lo[0] : -INFINITY;
-            sv[1] = lo_ok ? sv[1] - b_lo[1] : -INFINITY;
-            sv[2] = hi_ok ? sv[2] - b_hi[0] : -INFINITY;
-            sv[3] = hi_ok ? sv[3] - b_hi[1] : -INFINITY;
             float mx0 = fmaxf(sv[0], sv[2]), mx1 = fmaxf(sv[1], sv[3]);
 #pragma unroll
             for (int sh = 4; sh <= 16; sh <<= 1) {
@@ -841,11 +842,11 @@ decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restri
     }
 }
 
-template <int HD, int VD>
-int launch_decode(const void* q, const void* k_pages, const void* v_pages, const int* block_table, int bt_stride,
+template <int HD, int VD, bool kMore>
+int launch_decode_one(const void* q, const void* k_pages, const void* v_pages, const int* block_table, int bt_stride,
                   const int* tok_seq, const int* tok_pos, void* out, float* scratch, int n_tok, int n_heads, int n_kv,
-                  float scale, int window, int keep, int vo, int n_splits, cudaStream_t stream, const FusedQK* fused = nullptr,
-                  float slope_base = 0.0f, const float* sinks = nullptr, float cap = 0.0f, const OutGate gate = OutGate{}) {
+                  float scale, int window, int keep, int vo, int n_splits, cudaStream_t stream, const FusedQK* fused,
+                  float slope_base, const float* sinks, float cap, const OutGate& gate) {
     using Kernel = void (*)(const __nv_bfloat16*, const __nv_bfloat16*, const __nv_bfloat16*, const int*, int, const int*,
                             const int*, __nv_bfloat16*, float*, float*, int, int, float, int, int, const FusedQK, const float*,
                             int, int, const ScoreCap, const OutGate);
@@ -858,10 +859,10 @@ int launch_decode(const void* q, const void* k_pages, const void* v_pages, const
     float* part_ml = scratch ? scratch + (size_t)n_tok * n_kv * n_splits * G * VD : nullptr;
     // without scratch the splits merge inside a cluster (the caller checked n_splits <= 8)
     const bool cluster = scratch == nullptr && n_splits > 1;
-    const Kernel plain = cluster ? (G <= 8 ? (Kernel)decode_kernel<HD, VD, 1, true, false> : (Kernel)decode_kernel<HD, VD, 2, true, false>)
-                                 : (G <= 8 ? (Kernel)decode_kernel<HD, VD, 1, false, false> : (Kernel)decode_kernel<HD, VD, 2, false, false>);
-    const Kernel from_qkv = cluster ? (G <= 8 ? (Kernel)decode_kernel<HD, VD, 1, true, true> : (Kernel)decode_kernel<HD, VD, 2, true, true>)
-                                    : (G <= 8 ? (Kernel)decode_kernel<HD, VD, 1, false, true> : (Kernel)decode_kernel<HD, VD, 2, false, true>);
+#define NN_PICK(CL, FU) (G <= 8 ? (Kernel)decode_kernel<HD, VD, 1, CL, FU, kMore> : (Kernel)decode_kernel<HD, VD, 2, CL, FU, kMore>)
+    const Kernel plain = cluster ? NN_PICK(true, false) : NN_PICK(false, false);
+    const Kernel from_qkv = cluster ? NN_PICK(true, true) : NN_PICK(false, true);
+#undef NN_PICK
     const Kernel kernel = fused ? from_qkv : plain;
     FusedQK f = fused ? *fused : FusedQK{};
     if (!fused) f.slope_base = slope_base;
@@ -898,6 +899,17 @@ int launch_decode(const void* q, const void* k_pages, const void* v_pages, const
         NN_LAUNCH_OK("attention merge");
     }
     return 0;
+}
+
+template <int HD, int VD>
+int launch_decode(const void* q, const void* k_pages, const void* v_pages, const int* block_table, int bt_stride,
+                  const int* tok_seq, const int* tok_pos, void* out, float* scratch, int n_tok, int n_heads, int n_kv,
+                  float scale, int window, int keep, int vo, int n_splits, cudaStream_t stream, const FusedQK* fused,
+                  float slope_base, const float* sinks, float cap, const OutGate& gate) {
+    const bool more = cap > 0.0f || (fused != nullptr && fused->conv.w != nullptr);
+    return (more ? launch_decode_one<HD, VD, true> : launch_decode_one<HD, VD, false>)(
+        q, k_pages, v_pages, block_table, bt_stride, tok_seq, tok_pos, out, scratch, n_tok, n_heads, n_kv, scale, window, keep, vo,
+        n_splits, stream, fused, slope_base, sinks, cap, gate);
 }
 
 template <int HD, int VD>
